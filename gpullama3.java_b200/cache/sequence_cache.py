@@ -13,7 +13,8 @@ sequence (inference/state/LlamaState.java:44-46,61-64 of the reference project).
   one page table per sequence (shared by the group's entries).  ``KVGroup`` is the paged group of
   attention: keys ``[entry][page][kv_head][64][head_dim]``, values transposed
   ``[entry][page][kv_head][head_dim][64]``; with a ``window`` it only keeps the pages a query can
-  still reach (and the pages of the first ``keep_first`` positions, if the need has any);
+  still reach (and the pages of the first ``keep_first`` positions, if the need has any), with a ``chunk`` those of the
+  run of positions the next query belongs to;
 * a *slot group* has a fixed size per sequence: ``StateGroup`` owns ``[entry][slot][...shape]``,
   zeroed when a slot is acquired;
 * a block that keeps several things per run (a mixer's cache and state of its own beside it) asks with ``EntryNeeds``,
@@ -35,11 +36,13 @@ from .pages import PAGE_TOKENS, CacheError, CacheFull, PagePool, SlotTable, page
 class KVCacheNeed:
     """Growing keys and values: one [kv_heads, head_dim] row per position; ``window`` = how many
     of the latest positions a query reads (None: all of them); with a window, the first ``keep_first``
-    positions of a sequence stay readable for good."""
+    positions of a sequence stay readable for good.  ``chunk`` (in place of a window): positions are cut into runs of
+    that many, counted from 0, and a query reads those of its own run."""
     n_kv_heads: int
     head_dim: int
     window: int | None = None
     keep_first: int = 0
+    chunk: int | None = None
 
 
 @dataclass(frozen=True)
@@ -101,13 +104,17 @@ class PagedGroup(CacheGroup):
     """Bookkeeping of a group that grows page by page; subclasses own the device storage and the view."""
     paged = True
 
-    def __init__(self, need, entries, sizes: CacheSizes, window: int | None = None, keep_first: int = 0):
+    def __init__(self, need, entries, sizes: CacheSizes, window: int | None = None, keep_first: int = 0,
+                 chunk: int | None = None):
         super().__init__(need, entries, sizes)
-        self.window = window
+        if window is not None and chunk is not None:
+            raise CacheError("a paged group has a window or runs of positions, not both")
+        self.window, self.chunk = window, chunk
         self.kept_pages = pages_for(keep_first) if window is not None else 0   # a sequence's first pages that are never let go
         n_pages = sizes.n_pages
-        if window is not None:   # a windowed group never holds more than this, whatever the promised total
-            per_seq = pages_for(window + max(sizes.window_slack, 1)) + 1 + self.kept_pages
+        reach = window if window is not None else chunk
+        if reach is not None:   # such a group never holds more than this, whatever the promised total
+            per_seq = pages_for(reach + max(sizes.window_slack, 1)) + 1 + self.kept_pages
             n_pages = min(n_pages, sizes.max_slots * per_seq)
         self.pool = PagePool(n_pages)
         # per live slot: logical page index -> physical page, -1 where a windowed group let go
@@ -129,9 +136,12 @@ class PagedGroup(CacheGroup):
 
     def commit(self, slot: int, new_length: int) -> None:
         """The sequence now holds ``new_length`` tokens: let go of pages no later query can reach."""
-        if self.window is None:
+        if self.window is not None:
+            first_needed = max(0, new_length - self.window + 1)  # the next query sits at position `new_length`
+        elif self.chunk is not None:
+            first_needed = new_length - new_length % self.chunk   # (in a run of its own when the last one is full)
+        else:
             return
-        first_needed = max(0, new_length - self.window + 1)  # the next query sits at position `new_length`
         dead = first_needed // PAGE_TOKENS
         row = self.rows[slot]
         drop = [p for p in row[self.kept_pages:dead] if p >= 0]
@@ -160,7 +170,7 @@ class KVView:
 
 class KVGroup(PagedGroup):
     def __init__(self, need: KVCacheNeed, entries, sizes: CacheSizes):
-        super().__init__(need, entries, sizes, window=need.window, keep_first=need.keep_first)
+        super().__init__(need, entries, sizes, window=need.window, keep_first=need.keep_first, chunk=need.chunk)
         n = self.pool.n_pages
         # keys: a row per position; values: transposed, a row per dimension (positions contiguous)
         self.k = torch.zeros((len(self.entries), n, need.n_kv_heads, PAGE_TOKENS, need.head_dim), dtype=sizes.dtype,

@@ -118,6 +118,11 @@ class ModelConfig:
         """What the embedding rows are multiplied with as they enter the residual stream."""
         return 1.0
 
+    def embedding_norm(self) -> PartSpec | None:
+        """A norm over the embedding rows whose result is the residual stream the first block is handed; None: the rows
+        themselves are.  Its parameter path is ``embedding_norm``."""
+        return None
+
     def output_scale(self) -> float:
         """What the logits are multiplied with as they leave the head."""
         return 1.0

@@ -32,6 +32,9 @@
 // exponential joins the denominator (the first warp of a sequence's first span starts its running maximum and sum
 // at (sinks[h], 1)); a gate per (sequence, head): the output is multiplied by sigmoid(gate).
 //
+// A further mask (DecodeTerms.chunk): positions are cut into runs of `chunk`, counted from position 0, and the token sees
+// the keys of its own run only.  It reaches the kernel as the window that ends at the token and starts with its run.
+//
 // Sizes: head_dim 32, 64, 96 or 128; group size (heads per kv head) <= 16.  Others are refused.
 #include "attention_decode_static.h"
 #include <cstdint>
@@ -80,6 +83,7 @@ __device__ __forceinline__ uint4 keep_first(uint4 v, int n) {
 // (n_seqs x n_splits of them at most; sequence i's are prefix_i .. prefix_i + count_i - 1 of span_plan).
 struct DecodeTerms {
     int keep_first;
+    int chunk;                     // 0: no runs
     const float* slopes;           // [n_heads] or null
     const float* sinks;            // [n_heads] or null
     const __nv_bfloat16* gate;     // [n_seqs][ld_gate], column h, or null
@@ -111,9 +115,15 @@ __device__ __forceinline__ float rotate_elem(const __nv_bfloat16* x, int d, int 
 // number, and the merge kernel evaluates the same plan.  Lengths are read before the dependency wait, like kv_lens[seq].
 constexpr int kSpanPlanMaxSeqs = 64;   // larger batches (whose grids fill the GPU with one or two spans) keep equal counts
 
+// how many of the latest positions the last of `kv_len` positions sees (0: all of them)
+__device__ __forceinline__ int reach_of(int kv_len, int window, int chunk) {
+    return chunk > 0 ? (kv_len - 1) % chunk + 1 : window;
+}
+
 __device__ __forceinline__ int cached_blocks(const int* __restrict__ kv_lens, int i, int window, bool own_key_apart,
-                                             int keep_first) {
+                                             int keep_first, int chunk) {
     const int kv_len = kv_lens[i];
+    window = reach_of(kv_len, window, chunk);
     const int lo = window > 0 ? max(0, kv_len - window) : 0;
     const int n_cached = own_key_apart ? kv_len - 1 : kv_len;
     const int n_keep = min(keep_first, lo);      // kept first positions the window no longer covers
@@ -123,12 +133,12 @@ __device__ __forceinline__ int cached_blocks(const int* __restrict__ kv_lens, in
 // prefix and count of sequence `seq` (find_cta < 0), or of the sequence that owns CTA number `find_cta`; false if that
 // CTA is left over (the counts are rounded down, so up to n_seqs CTAs of a kv head may be)
 __device__ __forceinline__ bool span_plan(const int* __restrict__ kv_lens, int n_seqs, int n_splits, int window,
-                                          bool own_key_apart, int keep_first, int seq, int find_cta, int& owner, int& prefix,
+                                          bool own_key_apart, int keep_first, int chunk, int seq, int find_cta, int& owner, int& prefix,
                                           int& count) {
     bool planned = n_splits > 1 && n_seqs <= kSpanPlanMaxSeqs;
     unsigned int total = 0;
     if (planned) {
-        for (int i = 0; i < n_seqs; ++i) total += (unsigned int)cached_blocks(kv_lens, i, window, own_key_apart, keep_first);
+        for (int i = 0; i < n_seqs; ++i) total += (unsigned int)cached_blocks(kv_lens, i, window, own_key_apart, keep_first, chunk);
         planned = total > 0 && total < (1u << 20);   // (the products below stay inside 32 bits)
     }
     if (!planned) {
@@ -141,7 +151,7 @@ __device__ __forceinline__ bool span_plan(const int* __restrict__ kv_lens, int n
     int at = 0;
     bool found = false;
     for (int i = 0; i < n_seqs; ++i) {
-        const int c = 1 + (int)((unsigned int)cached_blocks(kv_lens, i, window, own_key_apart, keep_first) * spare / total);
+        const int c = 1 + (int)((unsigned int)cached_blocks(kv_lens, i, window, own_key_apart, keep_first, chunk) * spare / total);
         if (find_cta < 0 ? i == seq : (find_cta >= at && find_cta < at + c)) {
             owner = i; prefix = at; count = c; found = true;
         }
@@ -161,7 +171,7 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_row_stride, _
                         float* __restrict__ part_o, float* __restrict__ part_ml, int n_heads, int n_kv_heads,
                         int window, int n_splits, RopeArgs rope, DecodeTerms given) {
     constexpr int D = KB * 32;
-    const DecodeTerms terms = TERMS ? given : DecodeTerms{0, nullptr, nullptr, nullptr, 0};
+    const DecodeTerms terms = TERMS ? given : DecodeTerms{0, 0, nullptr, nullptr, nullptr, 0};
     constexpr int NJ = D / 8;  // output tiles of 8 dims
     constexpr int SLOTS = kAttnDecodeWarps + (FUSED ? 1 : 0);  // partials merged per CTA: the warps, and the new key
     // Rows of the tiles that exist: 8 without the upper half.  (Shared memory is taken from the SM's L1, through which the
@@ -184,13 +194,14 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_row_stride, _
     // before the wait for the predecessor; the queries, the step's key and value and the cache are read after it.
     // Which sequence this CTA works for, as which of its spans, and how many spans that sequence has:
     int seq, span_first, span_count;
-    if (!span_plan(kv_lens, (int)gridDim.z, n_splits, window, FUSED && rope.write_cache, terms.keep_first, -1,
+    if (!span_plan(kv_lens, (int)gridDim.z, n_splits, window, FUSED && rope.write_cache, terms.keep_first, terms.chunk, -1,
                    (int)(blockIdx.z * gridDim.x + blockIdx.x), seq, span_first, span_count)) {
         pdl_wait();   // (a CTA that is left over; it still waits, so that this kernel's end implies its predecessor's)
         return;
     }
     const int split = (int)(blockIdx.z * gridDim.x + blockIdx.x) - span_first;
     const int kv_len = kv_lens[seq];
+    if (TERMS) window = reach_of(kv_len, window, terms.chunk);
     const int lo = window > 0 ? max(0, kv_len - window) : 0;
     // keys read from the cache: all of them, or all but the step's own when this kernel writes that one
     const int n_cached = (FUSED && rope.write_cache) ? kv_len - 1 : kv_len;
@@ -531,13 +542,13 @@ __device__ __forceinline__ void merge_spans_at_once(const float* __restrict__ pa
 // pays one round trip to L2 per span); they are added in span order, so the sum is the same.
 __global__ void attention_decode_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                               __nv_bfloat16* __restrict__ out, const int* __restrict__ kv_lens, int n_heads,
-                                              int n_splits, int D, int window, int own_key_apart, int keep_first,
+                                              int n_splits, int D, int window, int own_key_apart, int keep_first, int chunk,
                                               const __nv_bfloat16* __restrict__ gate, int ld_gate) {
     pdl_launch_dependents();
     const size_t row = blockIdx.x;  // seq * n_heads + head
     const int seq = (int)(blockIdx.x / n_heads), head = (int)(blockIdx.x % n_heads);
     int owner, span_first, count;
-    span_plan(kv_lens, (int)(gridDim.x / n_heads), n_splits, window, own_key_apart != 0, keep_first, seq, -1, owner, span_first, count);
+    span_plan(kv_lens, (int)(gridDim.x / n_heads), n_splits, window, own_key_apart != 0, keep_first, chunk, seq, -1, owner, span_first, count);
     pdl_wait();
     const float gv = gate ? 1.0f / (1.0f + expf(-__bfloat162float(gate[(size_t)seq * ld_gate + head]))) : 1.f;
     const size_t first = (size_t)span_first * n_heads + head, stride = (size_t)n_heads;
@@ -593,9 +604,10 @@ static int launch_attention_decode(const void* q, int q_row_stride, void* out, c
                                    int table_stride, void* k_pool, void* v_pool, float* scratch, long long scratch_floats,
                                    int n_seqs, int n_heads, int n_kv_heads, int head_dim, int window, int n_splits,
                                    bool fused, RopeArgs rope, bool early_start, cudaStream_t stream,
-                                   DecodeTerms terms = DecodeTerms{0, nullptr, nullptr, nullptr, 0}) {
+                                   DecodeTerms terms = DecodeTerms{0, 0, nullptr, nullptr, nullptr, 0}) {
     if (n_seqs <= 0) return 0;
     if (terms.keep_first < 0 || (terms.keep_first > 0 && window <= 0)) return kErrBadArgument;
+    if (terms.chunk < 0 || (terms.chunk > 0 && (window > 0 || terms.keep_first > 0))) return kErrBadArgument;
     if (n_kv_heads <= 0 || n_heads % n_kv_heads != 0 || n_splits < 1) return kErrBadArgument;
     const int group = n_heads / n_kv_heads;
     if (group > 16 || head_dim % 32 != 0 || head_dim < 32 || head_dim > 128 || q_row_stride % 8 != 0) return kErrUnsupportedSize;
@@ -616,7 +628,7 @@ static int launch_attention_decode(const void* q, int q_row_stride, void* out, c
     auto vv = (__nv_bfloat16*)v_pool;
     auto oo = (__nv_bfloat16*)out;
     int st = 0;
-    const bool any_term = terms.keep_first > 0 || terms.slopes || terms.sinks || terms.gate;
+    const bool any_term = terms.keep_first > 0 || terms.chunk > 0 || terms.slopes || terms.sinks || terms.gate;
     if (any_term && fused) return kErrBadArgument;   // (the fused variant is not built with the terms)
 #define B200_LAUNCH(KB, F) do { if (group > 8) B200_LAUNCH_T(KB, F, true); else B200_LAUNCH_T(KB, F, false); } while (0)
 #define B200_LAUNCH_T(KB, F, HI) do { if (!F && any_term) B200_LAUNCH_H(KB, F, HI, !F); else B200_LAUNCH_H(KB, F, HI, false); } while (0)
@@ -649,7 +661,7 @@ static int launch_attention_decode(const void* q, int q_row_stride, void* out, c
     if (st != 0 || n_splits == 1) return st;
     return launch_pdl(attention_decode_merge_kernel, dim3(n_seqs * n_heads), dim3(head_dim <= 64 ? 64 : 128), 0, stream,
                       (const float*)part_o, (const float*)part_ml, oo, kv_lens, n_heads, n_splits, head_dim, window,
-                      (fused && rope.write_cache) ? 1 : 0, terms.keep_first, terms.gate, terms.ld_gate);
+                      (fused && rope.write_cache) ? 1 : 0, terms.keep_first, terms.chunk, terms.gate, terms.ld_gate);
 }
 
 }  // namespace b200
@@ -702,13 +714,13 @@ extern "C" int b200_attention_decode(const void* q, int q_row_stride, void* out,
 extern "C" int b200_attention_decode_terms(const void* q, int q_row_stride, void* out, const int* kv_lens,
                                            const int* page_table, int table_stride, const void* k_pool, const void* v_pool,
                                            float* scratch, long long scratch_floats, int n_seqs, int n_heads, int n_kv_heads,
-                                           int head_dim, int window, int n_splits, int early_start, int keep_first,
+                                           int head_dim, int window, int n_splits, int early_start, int keep_first, int chunk,
                                            const float* slopes, const float* sinks, const void* gate, int ld_gate,
                                            cudaStream_t stream) {
     return b200::launch_attention_decode(q, q_row_stride, out, kv_lens, page_table, table_stride, const_cast<void*>(k_pool),
                                          const_cast<void*>(v_pool), scratch, scratch_floats, n_seqs, n_heads, n_kv_heads,
                                          head_dim, window, n_splits, false, b200::RopeArgs{nullptr, 0, 0}, early_start != 0, stream,
-                                         b200::DecodeTerms{keep_first, slopes, sinks, (const __nv_bfloat16*)gate, ld_gate});
+                                         b200::DecodeTerms{keep_first, chunk, slopes, sinks, (const __nv_bfloat16*)gate, ld_gate});
 }
 
 // The fused variant: `qkv` holds the step's raw projections [n_seqs, (n_heads + 2 n_kv_heads) head_dim]; queries

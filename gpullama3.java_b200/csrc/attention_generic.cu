@@ -11,6 +11,8 @@
 // tiles of 128 keys in 32-bit.  `window` > 0 keeps only the last `window` keys.
 //
 // Optional further terms (AttentionTerms; all off for the Llama 3 decoder):
+//   chunk       positions are cut into runs of `chunk`, counted from position 0: i sees j <= i of its own run only (in
+//               place of a window)
 //   keep_first  with a window, the first keep_first positions of a sequence stay visible to every later query
 //               (position i sees j when j <= i and (i - j < window or j < keep_first)); the keys a query reads are
 //               then two runs, [0, min(keep_first, first)) and [first, i], walked as one row of tiles
@@ -27,6 +29,7 @@ constexpr int kMaxDimBlocks = 16;   // head sizes up to 512, 32 dimensions per b
 
 struct AttentionTerms {
     int keep_first;
+    int chunk;             // 0: no runs
     const float* slopes;   // [n_heads] or null
     const float* sinks;    // [n_heads] or null
     const void* gate;      // [T][ld_gate] of the run's storage type, column h, or null
@@ -78,7 +81,7 @@ attention_paged_kernel(const T* __restrict__ q, int q_row_stride, T* __restrict_
     const int g = h / (n_heads / n_kv_heads);
     const int pos = positions[t];
     const int* pages = page_table + (size_t)seq_ids[t] * table_stride;
-    const int first = window > 0 ? max(0, pos - window + 1) : 0;
+    const int first = terms.chunk > 0 ? pos - pos % terms.chunk : window > 0 ? max(0, pos - window + 1) : 0;
     // With gridDim.z > 1 the keys first .. pos are cut into that many spans of whole tiles, one CTA each, which leave
     // unnormalised partial results (maximum, sum, output) for attention_paged_merge_kernel: a decode step has few
     // (token, head) pairs and long rows of keys.
@@ -222,11 +225,12 @@ __global__ void attention_paged_merge_kernel(const float* __restrict__ part_o, c
 extern "C" int b200_attention_paged(const void* q, int q_row_stride, void* out, int dtype, const int* positions,
                                     const int* seq_ids, const int* page_table, int table_stride, const void* k_pool,
                                     const void* v_pool, int n_tokens, int n_heads, int n_kv_heads, int head_dim,
-                                    int window, int n_splits, float* scratch, int keep_first, const float* slopes,
+                                    int window, int n_splits, float* scratch, int keep_first, int chunk, const float* slopes,
                                     const float* sinks, const void* gate, int ld_gate, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (keep_first < 0 || (keep_first > 0 && window <= 0)) return b200::kErrBadArgument;
-    const b200::AttentionTerms terms = {keep_first, slopes, sinks, gate, ld_gate};
+    if (chunk < 0 || (chunk > 0 && (window > 0 || keep_first > 0))) return b200::kErrBadArgument;
+    const b200::AttentionTerms terms = {keep_first, chunk, slopes, sinks, gate, ld_gate};
     if (n_splits < 1 || n_splits > 64 || (n_splits > 1 && scratch == nullptr)) return b200::kErrBadArgument;
     if (head_dim % 16 != 0 || head_dim < 16 || head_dim > 32 * b200::kMaxDimBlocks) return b200::kErrUnsupportedSize;
     if (n_kv_heads <= 0 || n_heads % n_kv_heads != 0) return b200::kErrBadArgument;

@@ -17,6 +17,9 @@
 // denominator (every row's running maximum and sum start at (sinks[h], 1)); a gate per (token, head): the output is
 // multiplied by sigmoid(gate).
 //
+// A further mask (PrefillTerms.chunk): positions are cut into runs of `chunk`, counted from position 0, and i sees j <= i
+// of its own run only.
+//
 // Sizes: head_dim 32, 64, 96, 128.  Each warp owns 32 query rows (head_dim <= 64) or 16.
 #include "common.cuh"
 
@@ -24,6 +27,7 @@ namespace b200 {
 
 struct PrefillTerms {
     int keep_first;
+    int chunk;                     // 0: no runs
     const float* slopes;           // [n_heads] or null
     const float* sinks;            // [n_heads] or null
     const __nv_bfloat16* gate;     // [T][ld_gate], column h, or null
@@ -122,7 +126,7 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_row_stride, 
 
     // keys this warp needs: from the window's start of its first row to its last row's position
     const int p_first = start + row0, p_last = start + min(row0 + MT * 16, q_len) - 1;
-    const int k_lo = window > 0 ? max(0, p_first - window + 1) : 0;
+    const int k_lo = terms.chunk > 0 ? p_first - p_first % terms.chunk : window > 0 ? max(0, p_first - window + 1) : 0;
     // blocks of kept first positions that lie wholly before the window's first block come first
     const int kept_blocks = min((terms.keep_first + 31) / 32, k_lo / 32), shift = k_lo / 32 - kept_blocks;
     for (int vblk = 0; vblk <= p_last / 32 - shift; ++vblk) {
@@ -145,7 +149,7 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_row_stride, 
         for (int j = 0; j < NJ; ++j)
             vf[j] = __ldg(reinterpret_cast<const uint4*>(vp + (size_t)(8 * j + g) * kPageTokens + in_page + t * 8));
         // no masking is needed when every key of the block is visible to every row of the warp
-        const bool full = base + 31 <= p_first && (window <= 0 || base >= p_last - window + 1 || base + 31 < terms.keep_first);
+        const bool full = base + 31 <= p_first && (terms.chunk <= 0 || base >= p_last - p_last % terms.chunk) && (window <= 0 || base >= p_last - window + 1 || base + 31 < terms.keep_first);
         const int n_valid = kv_len - (base + 8 * t);
         if (n_valid < 8) {
 #pragma unroll
@@ -167,6 +171,8 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_row_stride, 
             // scores stay in units of q.k; exp((s - m) / sqrt(d)) is evaluated as exp2((s - m) * scale_log2)
             float bm[2] = {-INFINITY, -INFINITY};
             if (!full) {
+                const int run_lo[2] = {terms.chunk > 0 ? pos[mt][0] - pos[mt][0] % terms.chunk : 0,
+                                       terms.chunk > 0 ? pos[mt][1] - pos[mt][1] % terms.chunk : 0};
 #pragma unroll
                 for (int i = 0; i < 4; ++i)
 #pragma unroll
@@ -174,7 +180,7 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_row_stride, 
                         const int key = base + 8 * t + 2 * i + e;
 #pragma unroll
                         for (int r = 0; r < 2; ++r) {
-                            const bool ok = key <= pos[mt][r] && (window <= 0 || key > pos[mt][r] - window || key < terms.keep_first);
+                            const bool ok = key <= pos[mt][r] && key >= run_lo[r] && (window <= 0 || key > pos[mt][r] - window || key < terms.keep_first);
                             if (!ok) s[i][2 * r + e] = -INFINITY;
                         }
                     }
@@ -258,12 +264,13 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_row_stride, 
 extern "C" int b200_attention_prefill(const void* q, int q_row_stride, void* out, const int* cu_seqlens,
                                       const int* kv_lens, const int* page_table, int table_stride, const void* k_pool,
                                       const void* v_pool, int n_seqs, int max_q_len, int n_heads, int n_kv_heads,
-                                      int head_dim, int window, int keep_first, const float* slopes, const float* sinks,
+                                      int head_dim, int window, int keep_first, int chunk, const float* slopes, const float* sinks,
                                       const void* gate, int ld_gate, cudaStream_t stream) {
     using namespace b200;
     if (n_seqs <= 0 || max_q_len <= 0) return 0;
     if (keep_first < 0 || (keep_first > 0 && window <= 0)) return kErrBadArgument;
-    const PrefillTerms terms = {keep_first, slopes, sinks, (const __nv_bfloat16*)gate, ld_gate};
+    if (chunk < 0 || (chunk > 0 && (window > 0 || keep_first > 0))) return kErrBadArgument;
+    const PrefillTerms terms = {keep_first, chunk, slopes, sinks, (const __nv_bfloat16*)gate, ld_gate};
     if (n_kv_heads <= 0 || n_heads % n_kv_heads != 0) return kErrBadArgument;
     if (head_dim % 32 != 0 || head_dim < 32 || head_dim > 128 || q_row_stride % 8 != 0) return kErrUnsupportedSize;
     if (n_seqs > 65535 || n_heads > 65535) return kErrUnsupportedSize;

@@ -14,6 +14,10 @@
 // saves most rescaling passes.  Q, K pages and V^T pages arrive by TMA (128-byte swizzle) through a
 // two-stage ring.  With head_dim 64 two CTAs fit on an SM, so one CTA's softmax overlaps the other's MMAs.
 //
+// The single-tile kernel takes a window, or `chunk` (positions cut into runs counted from position 0, i sees j <= i of its
+// own run), and a sink per head: a key without a value whose exponential joins the row's sum when the row is finished (the
+// running reference maximum is only a reference, so the sink need not take part in it).
+//
 // Roles (320 threads): warp 0 lane 0 issues TMA; warp 1 lane 0 issues MMAs (warp 1 owns the 256 TMEM
 // columns: S 128, O head_dim); warps 2-9 are the softmax (two threads per query row) and the epilogue.  Every mbarrier wait is bounded;
 // a wait that gives up sets a status word and all roles fall through to the common exit.
@@ -97,7 +101,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                             const __grid_constant__ CUtensorMap map_v, __nv_bfloat16* __restrict__ out,
                             const int* __restrict__ cu_seqlens, const int* __restrict__ kv_lens,
                             const int* __restrict__ page_table, int table_stride, int n_heads, int n_kv_heads,
-                            int window, int k_rows_total, int v_rows_total) {
+                            int window, int chunk, const float* __restrict__ sinks, int k_rows_total, int v_rows_total) {
     // Two CTAs share an SM only if each stays within 113 KB, which leaves no room for an alignment pad: the
     // dynamic shared memory of a kernel without static shared memory starts at the CTA's window, 1024-aligned;
     // if it ever does not, the kernel records that and leaves.
@@ -119,7 +123,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     const int q0 = tile * kFaRows;
     const int rows_here = min(kFaRows, q_len - q0);
     const int p_first = start + q0, p_last = start + q0 + rows_here - 1;  // positions of the first and last row
-    const int key_lo = window > 0 ? max(0, p_first - window + 1) : 0;
+    const int key_lo = chunk > 0 ? p_first - p_first % chunk : window > 0 ? max(0, p_first - window + 1) : 0;
     const int blk_begin = key_lo / kFaKeys, blk_end = p_last / kFaKeys + 1;  // key blocks [begin, end)
     const int* pages = page_table + (size_t)seq * table_stride;
     const int n_pages_seq = (kv_len + kPageTokens - 1) / kPageTokens;
@@ -224,8 +228,9 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             if (!ok) break;
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
             const int base = blk * kFaKeys + half * 64;  // first key of this thread's half
-            const bool masked = blk * kFaKeys + kFaKeys - 1 > p_first || (window > 0 && blk * kFaKeys < p_last - window + 1);
-            const int lo_key = window > 0 ? pos - window + 1 : 0;
+            const bool masked = blk * kFaKeys + kFaKeys - 1 > p_first || (window > 0 && blk * kFaKeys < p_last - window + 1) ||
+                                (chunk > 0 && blk * kFaKeys < p_last - p_last % chunk);
+            const int lo_key = chunk > 0 ? pos - pos % chunk : window > 0 ? pos - window + 1 : 0;
             // pass 1: the block's maximum of this row (this thread's 64 keys, then both halves together)
             float m_blk = -INFINITY;
 #pragma unroll
@@ -315,7 +320,11 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         asm volatile("bar.sync 1, 256;" ::: "memory");   // every thread is done with the maxima that share this memory
         if (half == 1) sm.row_sum[r] = l;
         asm volatile("bar.sync 1, 256;" ::: "memory");
-        if (half == 0) { l += sm.row_sum[r]; sm.row_sum[r] = l; }
+        if (half == 0) {
+            l += sm.row_sum[r];
+            if (sinks != nullptr) l += ex2(sinks[head] * 1.4426950408889634f - (m_ref == -INFINITY ? 0.f : m_ref * scale_log2));
+            sm.row_sum[r] = l;
+        }
         asm volatile("bar.sync 1, 256;" ::: "memory");
         if (ok) {
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
@@ -869,7 +878,7 @@ namespace b200 {
 template <int D>
 static int launch_fa(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, void* out, const int* cu_seqlens,
                      const int* kv_lens, const int* page_table, int table_stride, int n_seqs, int max_q_len, int n_heads,
-                     int n_kv_heads, int window, int k_rows, int v_rows, cudaStream_t stream) {
+                     int n_kv_heads, int window, int chunk, const float* sinks, int k_rows, int v_rows, cudaStream_t stream) {
     static_assert(D != 64 || sizeof(FaSmem<64>) <= 113 * 1024, "two CTAs per SM need at most 113 KB each");
     const size_t smem = sizeof(FaSmem<D>);
     static bool configured = false;
@@ -880,7 +889,7 @@ static int launch_fa(const CUtensorMap& mq, const CUtensorMap& mk, const CUtenso
     }
     dim3 grid((max_q_len + kFaRows - 1) / kFaRows, n_heads, n_seqs);
     return launch_pdl(attention_prefill_tc_kernel<D>, grid, dim3(kFaThreads), smem, stream, mq, mk, mv, (__nv_bfloat16*)out,
-                      cu_seqlens, kv_lens, page_table, table_stride, n_heads, n_kv_heads, window, k_rows, v_rows);
+                      cu_seqlens, kv_lens, page_table, table_stride, n_heads, n_kv_heads, window, chunk, sinks, k_rows, v_rows);
 }
 }  // namespace b200
 
@@ -913,14 +922,15 @@ static int launch_pair(const CUtensorMap& mq, const CUtensorMap& mk, const CUten
 
 // q: packed rows of q_row_stride elements whose first n_heads * head_dim are the rotated queries (n_rows of them);
 // k_pool [n_pages][n_kv_heads][64][head_dim], v_pool [n_pages][n_kv_heads][head_dim][64] (values transposed).
-// head_dim 64 or 128.
+// head_dim 64 or 128.  window, or chunk (not both; 0: none); sinks: float32 [n_heads] or null.
 extern "C" int b200_attention_prefill_tc(const void* q, int q_row_stride, int n_rows, void* out, const int* cu_seqlens,
                                          const int* kv_lens, const int* page_table, int table_stride,
                                          const void* k_pool, const void* v_pool, int n_pages, int n_seqs, int max_q_len,
-                                         int n_heads, int n_kv_heads, int head_dim, int window, cudaStream_t stream) {
+                                         int n_heads, int n_kv_heads, int head_dim, int window, int chunk, const float* sinks,
+                                         cudaStream_t stream) {
     using namespace b200;
     if (n_seqs <= 0 || max_q_len <= 0) return 0;
-    if (n_kv_heads <= 0 || n_heads % n_kv_heads != 0) return kErrBadArgument;
+    if (n_kv_heads <= 0 || n_heads % n_kv_heads != 0 || chunk < 0 || (chunk > 0 && window > 0)) return kErrBadArgument;
     if ((head_dim != 64 && head_dim != 128) || q_row_stride % 8 != 0 ||
         (((uintptr_t)q | (uintptr_t)k_pool | (uintptr_t)v_pool | (uintptr_t)out) & 15))
         return kErrUnsupportedSize;
@@ -932,7 +942,7 @@ extern "C" int b200_attention_prefill_tc(const void* q, int q_row_stride, int n_
         !make_map_2d(&mk, k_pool, k_rows, head_dim, head_dim, 64, 64) || !make_map_2d(&mv, v_pool, v_rows, 64, 64, 64, head_dim))
         return kErrUnsupportedSize;
     // tiles in pairs when there are enough pairs to give every SM one (fewer: the single-tile kernel fills more SMs)
-    if (window <= 0 && (long long)((max_q_len + 2 * kFaRows - 1) / (2 * kFaRows)) * n_heads * n_seqs >= device_sm_count()) {
+    if (window <= 0 && chunk <= 0 && sinks == nullptr && (long long)((max_q_len + 2 * kFaRows - 1) / (2 * kFaRows)) * n_heads * n_seqs >= device_sm_count()) {
         if (head_dim == 64)
             return launch_pair<64>(mq, mk, mv, out, cu_seqlens, kv_lens, page_table, table_stride, n_seqs, max_q_len, n_heads,
                                    n_kv_heads, (int)k_rows, (int)v_rows, stream);
@@ -941,7 +951,7 @@ extern "C" int b200_attention_prefill_tc(const void* q, int q_row_stride, int n_
     }
     if (head_dim == 64)
         return launch_fa<64>(mq, mk, mv, out, cu_seqlens, kv_lens, page_table, table_stride, n_seqs, max_q_len, n_heads,
-                             n_kv_heads, window, (int)k_rows, (int)v_rows, stream);
+                             n_kv_heads, window, chunk, sinks, (int)k_rows, (int)v_rows, stream);
     return launch_fa<128>(mq, mk, mv, out, cu_seqlens, kv_lens, page_table, table_stride, n_seqs, max_q_len, n_heads,
-                          n_kv_heads, window, (int)k_rows, (int)v_rows, stream);
+                          n_kv_heads, window, chunk, sinks, (int)k_rows, (int)v_rows, stream);
 }

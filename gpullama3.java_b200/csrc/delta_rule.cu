@@ -24,7 +24,8 @@
 // The same scan also runs the recurrences without the delta correction (linear_scan): S <- diag(g) S + k (beta v)^T,
 // o = S^T q + skip v, which is gated linear attention (a decay per key channel, g = sigmoid(.)^(1/tau), beta = 1) and the
 // state-space recurrence with a scalar decay per head (q = C, k = B, g = exp(-exp(A_log) dt), beta = dt = softplus(.),
-// skip = D); linear_scan_prepare makes their rows.  causal_conv is the convolution in its general form: input and output
+// skip = D), or a fixed decay per head (retention, lightning attention: g given, beta = 1, the keys and queries optionally
+// turned by their positions or passed through SiLU in 32 bits); linear_scan_prepare makes their rows.  causal_conv is the convolution in its general form: input and output
 // types of their own, an optional bias, SiLU or no activation, and optionally the input added to the result.
 #include "common.cuh"
 
@@ -380,7 +381,9 @@ delta_rule_prepare_kernel(PrepareArgs a) {
 // The rows of the recurrences without the delta correction, in the layout the scan reads: [q | k | g | v | beta | k . q |
 // skip].  q rows are scaled by q_scale; the decay is exp(-exp(A_log[h]) softplus(z + bias)) (kind 0) or
 // sigmoid(z + bias)^power (kind 1: exp(-softplus(-(z + bias)) power)), per key channel or per head; beta is 1, or the step
-// size softplus(z + bias) of a per-head decay of kind 0 (`step_scales_value`); skip is skip[h] or 0.
+// size softplus(z + bias) of a per-head decay of kind 0 (`step_scales_value`); skip is skip[h] or 0.  Kind 2: the decay is
+// a_log[h] as it stands (no projection).  `qk_silu`, `v_silu`: q and k (before the scale), v pass through SiLU; `pairs` > 0: the
+// pairs (i, i + pairs) of q and k, i < pairs, are turned by the token's position times inv_freq[i].
 struct LinearPrepareArgs {
     const void* q;          // [T, ld_q], head kvh of kv_heads at column kvh d_k
     int ld_q;
@@ -397,7 +400,12 @@ struct LinearPrepareArgs {
     int n_tokens, heads, kv_heads, d_k, d_v, d_pad, row;
     float q_scale, power;
     int decay_kind, decay_per_head, step_scales_value;
+    int qk_silu, v_silu, pairs;
+    const float* inv_freq;     // [pairs]
+    const int* positions;      // [T]
 };
+
+__device__ __forceinline__ float silu_of(float z) { return z / (1.0f + expf(-z)); }
 
 template <typename T>
 __global__ void __launch_bounds__(128)
@@ -411,7 +419,7 @@ linear_scan_prepare_kernel(LinearPrepareArgs a) {
     const T* kr = (const T*)a.k + t * a.ld_k + (size_t)kvh * a.d_k;
     const T* vr = (const T*)a.v + t * a.ld_v + (size_t)h * a.d_v;
     const size_t d_at = a.decay_per_head ? (size_t)h : (size_t)h * a.d_k;
-    const T* dr = (const T*)a.decay + t * a.ld_decay + d_at;
+    const T* dr = a.decay_kind == 2 ? nullptr : (const T*)a.decay + t * a.ld_decay + d_at;
     const float* br = a.decay_bias ? a.decay_bias + d_at : nullptr;
     float* out = a.rows + ((size_t)h * a.n_tokens + t) * a.row;
     const float neg_rate = a.decay_kind == 0 ? -expf(a.a_log[h]) : 0.f;
@@ -424,11 +432,22 @@ linear_scan_prepare_kernel(LinearPrepareArgs a) {
         return expf(-softplus(-z) * a.power);
     };
     float step_head = 1.f;
-    const float g_head = a.decay_per_head ? decay_of(to_f32<T>(dr[0]) + (br ? br[0] : 0.f), step_head) : 0.f;
+    const float g_head = a.decay_kind == 2 ? a.a_log[h] : a.decay_per_head ? decay_of(to_f32<T>(dr[0]) + (br ? br[0] : 0.f), step_head) : 0.f;
     float qk = 0.f;
     for (int i = lane; i < a.d_pad; i += 32) {
         const bool in = i < a.d_k;
-        const float qv = in ? to_f32<T>(qr[i]) * a.q_scale : 0.f, kv = in ? to_f32<T>(kr[i]) : 0.f;
+        float qv = in ? to_f32<T>(qr[i]) : 0.f, kv = in ? to_f32<T>(kr[i]) : 0.f;
+        if (a.qk_silu) { qv = silu_of(qv); kv = silu_of(kv); }
+        if (i < 2 * a.pairs) {
+            const bool first = i < a.pairs;
+            const int other = first ? i + a.pairs : i - a.pairs;
+            float sn, cs, qo = to_f32<T>(qr[other]), ko = to_f32<T>(kr[other]);
+            if (a.qk_silu) { qo = silu_of(qo); ko = silu_of(ko); }
+            sincosf((float)a.positions[t] * a.inv_freq[first ? i : other], &sn, &cs);
+            qv = first ? qv * cs - qo * sn : qv * cs + qo * sn;
+            kv = first ? kv * cs - ko * sn : kv * cs + ko * sn;
+        }
+        qv *= a.q_scale;
         qk += qv * kv;
         out[i] = qv;
         out[a.d_pad + i] = kv;
@@ -436,7 +455,10 @@ linear_scan_prepare_kernel(LinearPrepareArgs a) {
         out[2 * a.d_pad + i] = !in ? 0.f : a.decay_per_head ? g_head : decay_of(to_f32<T>(dr[i]) + (br ? br[i] : 0.f), unused);
     }
     qk = warp_sum(qk);
-    for (int j = lane; j < a.d_v; j += 32) out[3 * a.d_pad + j] = to_f32<T>(vr[j]);
+    for (int j = lane; j < a.d_v; j += 32) {
+        const float z = to_f32<T>(vr[j]);
+        out[3 * a.d_pad + j] = a.v_silu ? silu_of(z) : z;
+    }
     if (lane == 0) {
         out[3 * a.d_pad + a.d_v] = (a.step_scales_value && a.decay_per_head) ? step_head : 1.f;
         out[3 * a.d_pad + a.d_v + 1] = qk;
@@ -760,18 +782,21 @@ extern "C" int b200_linear_scan(const void* q, int ld_q, const void* k, int ld_k
                                 int ld_decay, const float* decay_bias, const float* a_log, const float* skip, float* state,
                                 long long slot_stride, const int* slots, const int* cu_seqlens, float* out, float* scratch,
                                 int dtype, int n_tokens, int n_seqs, int heads, int kv_heads, int d_k, int d_v, float q_scale,
-                                float power, int decay_kind, int decay_per_head, int step_scales_value, cudaStream_t stream) {
+                                float power, int decay_kind, int decay_per_head, int step_scales_value, int qk_silu, int v_silu,
+                                int pairs, const float* inv_freq, const int* positions, cudaStream_t stream) {
     if (n_seqs <= 0 || n_tokens <= 0) return 0;
     if (heads < 1 || kv_heads < 1 || heads % kv_heads || d_k < 1 || d_v < 1 || n_seqs > 65535 || heads > 65535 || !scratch)
         return b200::kErrBadArgument;
-    if ((decay_kind != 0 && decay_kind != 1) || (decay_kind == 0 && !a_log)) return b200::kErrBadArgument;
+    if (decay_kind < 0 || decay_kind > 2 || (decay_kind != 1 && !a_log) || (decay_kind != 2 && !decay)) return b200::kErrBadArgument;
+    if (decay_kind == 2 && !decay_per_head) return b200::kErrBadArgument;
+    if (pairs < 0 || 2 * pairs > d_k || (pairs > 0 && (!inv_freq || !positions))) return b200::kErrBadArgument;
     int rpt = 0, lanes = 0;
     if (!b200_delta_rule_plan(d_k, &rpt, &lanes)) return b200::kErrUnsupportedSize;
     const int row = b200_delta_rule_row(d_k, d_v);
     if ((uintptr_t)scratch % 16) return b200::kErrBadArgument;
     b200::LinearPrepareArgs p = {q, ld_q, k, ld_k, v, ld_v, decay, ld_decay, decay_bias, a_log, skip, scratch, n_tokens, heads,
                                  kv_heads, d_k, d_v, rpt * lanes, row, q_scale, power, decay_kind, decay_per_head ? 1 : 0,
-                                 step_scales_value ? 1 : 0};
+                                 step_scales_value ? 1 : 0, qk_silu, v_silu, pairs, inv_freq, positions};
     const long long units = (long long)n_tokens * heads;
     B200_DISPATCH_DTYPE(dtype, T,
         b200::linear_scan_prepare_kernel<T><<<(unsigned)((units + 3) / 4), 128, 0, stream>>>(p));

@@ -5,7 +5,11 @@
 //                      the row is multiplied by act(gate) first and the norm runs over the gated row; with
 //                      `weight_per_row` every row has weights of its own (w holds n_heads * d numbers), so that the rows
 //                      may be any equal parts of the mixer's output, not its heads; a warp per row, or a CTA per row
-//                      of 512 numbers and more
+//                      of 512 numbers and more; w may be absent, `mul` is a last factor, and the output's rows may be
+//                      columns of a wider buffer
+//   turn_back_rows     out[t, h, :d] = mul * (x[t, h, :d] turned by -position * inv_freq over the row's halves): the results of
+//                      attention over values that were cached turned by their own positions; x's heads are d_pad wide,
+//                      the output's rows may be columns of a wider buffer; a CTA per token, angles once per token
 //   gate_rows          x[t, :n] <- x[t, :n] * sigmoid(gate[t, :n]) (or SiLU), in place: a gate on a mixer's output
 //   scale_rows         x <- x * s, in place on 32-bit logits
 //   differential_heads out[t, h, :] = post * o / sqrt(mean(o^2) + eps) * sigmoid(gate[t, h, :]) with o = a1 - lambda a2, where
@@ -24,14 +28,15 @@ __global__ void softcap_kernel(float* __restrict__ x, size_t n, float cap) {
 template <typename T>
 __global__ void __launch_bounds__(128)
 gated_rmsnorm_kernel(const float* __restrict__ x, const float* __restrict__ w, const T* __restrict__ gate, int ld_gate,
-                     T* __restrict__ out, int n_heads, int d, int n_rows, float eps, int gate_act, int gate_first,
+                     T* __restrict__ out, int ld_out, float mul, int n_heads, int d, int n_rows, float eps, int gate_act, int gate_first,
                      int weight_per_row) {
     const int row = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
     if (row >= n_rows) return;
     const int t = row / n_heads, h = row % n_heads;
     const float* xr = x + (size_t)row * d;
     const T* g = gate + (size_t)t * ld_gate + (size_t)h * d;
-    const float* wr = w + (weight_per_row ? (size_t)h * d : 0);
+    const float* wr = w ? w + (weight_per_row ? (size_t)h * d : 0) : nullptr;
+    auto weight = [&](int e) { return wr ? wr[e] : 1.f; };
     auto act = [&](int e) {
         const float z = to_f32<T>(g[e]);
         const float sig = 1.0f / (1.0f + expf(-z));
@@ -43,10 +48,10 @@ gated_rmsnorm_kernel(const float* __restrict__ x, const float* __restrict__ w, c
         ss += v * v;
     }
     ss = warp_sum(ss);
-    const float scale = 1.0f / sqrtf(ss / (float)d + eps);
-    T* o = out + (size_t)row * d;
+    const float scale = mul / sqrtf(ss / (float)d + eps);
+    T* o = out + (size_t)t * ld_out + (size_t)h * d;
     for (int e = lane; e < d; e += 32)
-        o[e] = from_f32<T>(gate_first ? (xr[e] * act(e)) * scale * wr[e] : xr[e] * scale * wr[e] * act(e));
+        o[e] = from_f32<T>(gate_first ? (xr[e] * act(e)) * scale * weight(e) : xr[e] * scale * weight(e) * act(e));
 }
 
 // a CTA per row, for rows too long for one warp (a norm over a large part of the mixer's output); the gated values stay
@@ -55,13 +60,15 @@ constexpr int kWideThreads = 256, kWideKeep = 8;
 template <typename T>
 __global__ void __launch_bounds__(kWideThreads)
 gated_rmsnorm_wide_kernel(const float* __restrict__ x, const float* __restrict__ w, const T* __restrict__ gate, int ld_gate,
-                          T* __restrict__ out, int n_heads, int d, float eps, int gate_act, int gate_first, int weight_per_row) {
+                          T* __restrict__ out, int ld_out, float mul, int n_heads, int d, float eps, int gate_act, int gate_first,
+                          int weight_per_row) {
     __shared__ float scratch[33];
     const int row = blockIdx.x;
     const int t = row / n_heads, h = row % n_heads;
     const float* xr = x + (size_t)row * d;
     const T* g = gate + (size_t)t * ld_gate + (size_t)h * d;
-    const float* wr = w + (weight_per_row ? (size_t)h * d : 0);
+    const float* wr = w ? w + (weight_per_row ? (size_t)h * d : 0) : nullptr;
+    auto weight = [&](int e) { return wr ? wr[e] : 1.f; };
     auto act = [&](int e) {
         const float z = to_f32<T>(g[e]);
         const float sig = 1.0f / (1.0f + expf(-z));
@@ -79,15 +86,15 @@ gated_rmsnorm_wide_kernel(const float* __restrict__ x, const float* __restrict__
         ss += v * v;
     }
     ss = block_sum(ss, scratch);
-    const float scale = 1.0f / sqrtf(ss / (float)d + eps);
-    T* o = out + (size_t)row * d;
+    const float scale = mul / sqrtf(ss / (float)d + eps);
+    T* o = out + (size_t)t * ld_out + (size_t)h * d;
 #pragma unroll
     for (int i = 0; i < kWideKeep; ++i) {
         const int e = threadIdx.x + i * kWideThreads;
-        if (e < d) o[e] = from_f32<T>(gate_first ? keep[i] * scale * wr[e] : keep[i] * scale * wr[e] * act(e));
+        if (e < d) o[e] = from_f32<T>(gate_first ? keep[i] * scale * weight(e) : keep[i] * scale * weight(e) * act(e));
     }
     for (int e = threadIdx.x + kWideKeep * kWideThreads; e < d; e += kWideThreads)
-        o[e] = from_f32<T>(gate_first ? (xr[e] * act(e)) * scale * wr[e] : xr[e] * scale * wr[e] * act(e));
+        o[e] = from_f32<T>(gate_first ? (xr[e] * act(e)) * scale * weight(e) : xr[e] * scale * weight(e) * act(e));
 }
 
 template <typename T>
@@ -128,6 +135,35 @@ differential_heads_kernel(const T* __restrict__ maps, const T* __restrict__ gate
     }
 }
 
+constexpr int kTurnThreads = 128, kTurnPairs = 256;
+template <typename T>
+__global__ void __launch_bounds__(kTurnThreads)
+turn_back_rows_kernel(const T* __restrict__ x, const int* __restrict__ positions, const float* __restrict__ inv_freq,
+                      T* __restrict__ out, int ld_out, int n_heads, int d, int d_pad, float mul) {
+    __shared__ float cos_s[kTurnPairs], sin_s[kTurnPairs];
+    pdl_launch_dependents();
+    const int t = blockIdx.x, n = d / 2;
+    // positions were copied in before the step's first kernel: the angles are made before the wait
+    const float pos = inv_freq ? (float)positions[t] : 0.f;
+    for (int i = threadIdx.x; i < n && inv_freq; i += kTurnThreads) sincosf(pos * inv_freq[i], &sin_s[i], &cos_s[i]);
+    __syncthreads();
+    pdl_wait();
+    const T* xr = x + (size_t)t * n_heads * d_pad;
+    T* o = out + (size_t)t * ld_out;
+    if (!inv_freq) {
+        for (int u = blockIdx.y * kTurnThreads + threadIdx.x; u < n_heads * d; u += gridDim.y * kTurnThreads)
+            o[u] = from_f32<T>(to_f32<T>(xr[(size_t)(u / d) * d_pad + u % d]) * mul);
+        return;
+    }
+    for (int u = blockIdx.y * kTurnThreads + threadIdx.x; u < n_heads * n; u += gridDim.y * kTurnThreads) {
+        const int h = u / n, i = u % n;
+        const float a = to_f32<T>(xr[(size_t)h * d_pad + i]), b = to_f32<T>(xr[(size_t)h * d_pad + i + n]);
+        const float c = cos_s[i], s = sin_s[i];
+        o[(size_t)h * d + i] = from_f32<T>((a * c + b * s) * mul);
+        o[(size_t)h * d + i + n] = from_f32<T>((b * c - a * s) * mul);
+    }
+}
+
 __global__ void scale_kernel(float* __restrict__ x, size_t n, float s) {
     for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x) x[i] *= s;
 }
@@ -144,19 +180,19 @@ extern "C" int b200_softcap_rows(float* x, long long n, float cap, cudaStream_t 
 
 extern "C" int b200_gated_rmsnorm(const float* x, const float* w, const void* gate, int ld_gate, void* out, int dtype,
                                   int n_tokens, int n_heads, int d, float eps, int gate_act, int gate_first,
-                                  int weight_per_row, cudaStream_t stream) {
+                                  int weight_per_row, int ld_out, float mul, cudaStream_t stream) {
     if (gate_act != 0 && gate_act != 1) return b200::kErrBadArgument;   // 0 sigmoid, 1 SiLU
     if (n_tokens <= 0 || n_heads <= 0) return 0;
-    if (d < 1) return b200::kErrBadArgument;
+    if (d < 1 || ld_out < n_heads * d) return b200::kErrBadArgument;
     const long long rows = (long long)n_tokens * n_heads;
     if (rows > 0x7fffffffLL) return b200::kErrUnsupportedSize;
     B200_DISPATCH_DTYPE(dtype, T,
         if (d >= 512)      // (a warp would walk such a row in 16 or more rounds, twice)
-            b200::gated_rmsnorm_wide_kernel<T><<<(int)rows, b200::kWideThreads, 0, stream>>>(x, w, (const T*)gate, ld_gate, (T*)out,
+            b200::gated_rmsnorm_wide_kernel<T><<<(int)rows, b200::kWideThreads, 0, stream>>>(x, w, (const T*)gate, ld_gate, (T*)out, ld_out, mul,
                                                                                            n_heads, d, eps, gate_act, gate_first,
                                                                                            weight_per_row);
         else
-            b200::gated_rmsnorm_kernel<T><<<(int)((rows + 3) / 4), 128, 0, stream>>>(x, w, (const T*)gate, ld_gate, (T*)out,
+            b200::gated_rmsnorm_kernel<T><<<(int)((rows + 3) / 4), 128, 0, stream>>>(x, w, (const T*)gate, ld_gate, (T*)out, ld_out, mul,
                                                                                      n_heads, d, (int)rows, eps, gate_act, gate_first,
                                                                                      weight_per_row));
     return b200::launch_status();
@@ -191,5 +227,21 @@ extern "C" int b200_differential_heads(const void* maps, const void* gate, int l
     B200_DISPATCH_DTYPE(dtype, T,
         return b200::launch_pdl(b200::differential_heads_kernel<T>, dim3((int)((rows + 3) / 4)), dim3(128), 0, stream,
                                 (const T*)maps, (const T*)gate, ld_gate, (T*)out, n_heads, d, d_pad, (int)rows, lambda, post, eps));
+    return 0;
+}
+
+// x [T][n_heads d_pad], out [T][ld_out >= n_heads d] of the run's type; d even; inv_freq float32 [d / 2] (null: nothing is
+// turned, the heads are only moved and scaled)
+extern "C" int b200_turn_back_rows(const void* x, const int* positions, const float* inv_freq, void* out, int ld_out, int dtype,
+                                   int n_tokens, int n_heads, int d, int d_pad, float mul, cudaStream_t stream) {
+    if (n_tokens <= 0 || n_heads <= 0) return 0;
+    if (d < 1 || d_pad < d || ld_out < n_heads * d || (inv_freq && (d % 2 || !positions))) return b200::kErrBadArgument;
+    if (inv_freq && d / 2 > b200::kTurnPairs) return b200::kErrUnsupportedSize;
+    const int units = n_heads * (inv_freq ? d / 2 : d);
+    int ny = n_tokens >= 512 ? 1 : (units + b200::kTurnThreads - 1) / b200::kTurnThreads;   // few tokens: a token's heads over several CTAs
+    if (ny > 64) ny = 64;
+    B200_DISPATCH_DTYPE(dtype, T,
+        return b200::launch_pdl(b200::turn_back_rows_kernel<T>, dim3(n_tokens, ny), dim3(b200::kTurnThreads), 0, stream, (const T*)x,
+                                positions, inv_freq, (T*)out, ld_out, n_heads, d, d_pad, mul));
     return 0;
 }

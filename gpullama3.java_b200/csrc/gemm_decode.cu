@@ -21,7 +21,12 @@
 // x is w * x * r with r = rsqrt(mean(x^2) + eps) (inference/InferenceCore.java:47-56), and r, one number per
 // row, commutes with the next product.  The product that completes x (residual epilogue) also writes
 // bfloat16(x * w) and, per CTA, the sum of squares of the x it holds; the next product multiplies its
-// sums by r, which it gets by adding the partial sums in CTA order.  No kernel in between, no atomics.
+// sums by r, which it gets by adding the partial sums in CTA order.  No kernel in between, no atomics.  Two norms of the
+// same row that differ in their weights alone (a block whose two sublayers read the stream side by side) share the sums
+// of squares: the completing product then writes two copies, bfloat16(x * w) and bfloat16(x * w2).
+//
+// A bias (float32 [N], one number per output) joins every sum before the epilogue: before the activation of the gated
+// ones, once per element of the residual add.  It is a weight: it is fetched before the dependency wait.
 #include "common.cuh"
 
 namespace b200 {
@@ -59,6 +64,9 @@ struct NormLink {
     __nv_bfloat16* out_act;     // [M][ld_out_act]
     int ld_out_act;
     float* out_partials;        // [M][gridDim.x]
+    const void* out_weight2;    // [N] weights of a second norm of the same rows (of out_weight's type), or null
+    __nv_bfloat16* out_act2;    // [M][ld_out_act]
+    const float* bias;          // [N] or null
     // the gated epilogue's activation of the gate value: 0 SiLU, 1 GELU in its tanh form, 2 the clamped form
     // min(g, limit) sigmoid(slope min(g, limit)) (clamp(u, -limit, limit) + 1)
     int gate_act;
@@ -116,19 +124,25 @@ gemm_decode_kernel(const __nv_bfloat16* __restrict__ A, int lda, const __nv_bflo
     };
     // the first weights are on their way before the kernel that produces the activations has finished
     load_weights(warp * U);
+    __shared__ float bias_s[ROWS];
+    if (link.bias != nullptr && threadIdx.x < ROWS) bias_s[threadIdx.x] = row0 + (int)threadIdx.x < N ? link.bias[row0 + threadIdx.x] : 0.f;
     pdl_launch_dependents();
     pdl_wait();
     // What the epilogue will add to is asked for now, not at the CTA's tail (one element per thread when the
     // tile has no more elements than threads; a larger tile reads late).
     constexpr bool kEarlyC = EPI == 1 && NT * 8 * ROWS <= kDecodeThreads;
-    float c_early = 0.f, w_early = 0.f;
+    float c_early = 0.f, w_early = 0.f, w2_early = 0.f;
+    auto norm_weight = [&](const void* w, int n) {
+        return link.out_weight_f32 ? reinterpret_cast<const float*>(w)[n] : __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(w)[n]);
+    };
     if (kEarlyC && (int)threadIdx.x < NT * 8 * ROWS) {
         const int token = threadIdx.x / ROWS, row = threadIdx.x % ROWS;
         if (token < M && row0 + row < N) {
             c_early = to_f32<TC>(C[(size_t)token * ldc + row0 + row]);
-            if (LINK && NT <= 2 && link.out_weight != nullptr)
-                w_early = link.out_weight_f32 ? reinterpret_cast<const float*>(link.out_weight)[row0 + row]
-                                              : __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(link.out_weight)[row0 + row]);
+            if (LINK && NT <= 2 && link.out_weight != nullptr) {
+                w_early = norm_weight(link.out_weight, row0 + row);
+                if (link.out_weight2 != nullptr) w2_early = norm_weight(link.out_weight2, row0 + row);
+            }
         }
     }
     // The norm's factor of each row, made while the first weights are in flight: warp w adds the partial sums of
@@ -191,6 +205,7 @@ gemm_decode_kernel(const __nv_bfloat16* __restrict__ A, int lda, const __nv_bflo
 #pragma unroll
         for (int w = 0; w < kDecodeWarps; ++w) s += red[w][token][row];
         if (LINK && NT <= 2 && link.in_partials != nullptr) s *= row_factor[token];
+        if (link.bias != nullptr) s += bias_s[row];
         float square = 0.f;
         if (EPI == 2) {
             fin[token][row] = s;
@@ -200,10 +215,12 @@ gemm_decode_kernel(const __nv_bfloat16* __restrict__ A, int lda, const __nv_bflo
                 const float x = (kEarlyC ? c_early : to_f32<TC>(*c)) + s;
                 *c = from_f32<TC>(x);
                 if (LINK && NT <= 2 && link.out_weight != nullptr) {
-                    const float w = kEarlyC ? w_early
-                                  : link.out_weight_f32 ? reinterpret_cast<const float*>(link.out_weight)[row0 + row]
-                                                        : __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(link.out_weight)[row0 + row]);
+                    const float w = kEarlyC ? w_early : norm_weight(link.out_weight, row0 + row);
                     link.out_act[(size_t)token * link.ld_out_act + row0 + row] = __float2bfloat16_rn(x * w);
+                    if (link.out_weight2 != nullptr) {
+                        const float w2 = kEarlyC ? w2_early : norm_weight(link.out_weight2, row0 + row);
+                        link.out_act2[(size_t)token * link.ld_out_act + row0 + row] = __float2bfloat16_rn(x * w2);
+                    }
                     square = x * x;
                 }
             } else {
@@ -327,10 +344,12 @@ static int gemm_decode_launch(const void* A, int lda, const void* W, int ldw, vo
 }  // namespace b200
 
 // A, W bfloat16; C bfloat16 or float32 (c_dtype); epilogue 0 store, 1 residual add (C float32), 2 gated SiLU,
-// 3 gated GELU (tanh form), 4 gated and clamped (gate_limit, gate_slope).
+// 3 gated GELU (tanh form), 4 gated and clamped (gate_limit, gate_slope).  bias: float32 [N] or null.
 extern "C" int b200_gemm_decode(const void* A, int lda, const void* W, int ldw, void* C, int c_dtype, int ldc, int M,
-                                int N, int K, int epilogue, float gate_limit, float gate_slope, cudaStream_t stream) {
+                                int N, int K, int epilogue, float gate_limit, float gate_slope, const float* bias,
+                                cudaStream_t stream) {
     b200::NormLink link{};
+    link.bias = bias;
     link.gate_limit = gate_limit;
     link.gate_slope = gate_slope;
     return b200::gemm_decode_launch(A, lda, W, ldw, C, c_dtype, ldc, M, N, K, epilogue, link, stream);
@@ -348,17 +367,24 @@ extern "C" int b200_gemm_decode_ctas(int M, int N) {
 //       rsqrt(sum(in_partials[t]) / norm_dim + eps) before the epilogue.
 //   out_weight [N] (or null; epilogue 1 only): after the residual add, bfloat16(x * out_weight) goes to
 //       out_act [M][ld_out_act] and this CTA's sum of x^2 per row to out_partials [M][b200_gemm_decode_ctas(M, N)].
+//   out_weight2 [N] (or null): a second norm's weights over the same rows, bfloat16(x * out_weight2) to out_act2.
+//   bias [N] float32 (or null): joins every sum, behind the row factor and before the epilogue.
 extern "C" int b200_gemm_decode_linked(const void* A, int lda, const void* W, int ldw, void* C, int c_dtype, int ldc, int M,
                                        int N, int K, int epilogue, const float* in_partials, int n_in, float eps,
                                        int norm_dim, const void* out_weight, int out_weight_dtype, void* out_act,
-                                       int ld_out_act, float* out_partials, cudaStream_t stream) {
+                                       int ld_out_act, float* out_partials, const void* out_weight2, void* out_act2,
+                                       const float* bias, cudaStream_t stream) {
     using namespace b200;
     if (M > 16) return kErrUnsupportedSize;
     if (in_partials != nullptr && (n_in <= 0 || norm_dim <= 0)) return kErrBadArgument;
     if (out_weight != nullptr && (epilogue != 1 || out_act == nullptr || out_partials == nullptr || ld_out_act < N ||
                                   (out_weight_dtype != kF32 && out_weight_dtype != kBF16)))
         return kErrBadArgument;
+    if (out_weight2 != nullptr && (out_weight == nullptr || out_act2 == nullptr)) return kErrBadArgument;
     NormLink link{};
+    link.bias = bias;
+    link.out_weight2 = out_weight2;
+    link.out_act2 = (__nv_bfloat16*)out_act2;
     link.in_partials = in_partials;
     link.n_in = n_in;
     link.eps = eps;

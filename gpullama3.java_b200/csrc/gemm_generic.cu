@@ -13,6 +13,7 @@
 //   3  gated GELU    the same with gelu(g) = 0.5 g (1 + tanh(sqrt(2/pi) (g + 0.044715 g^3))), the tanh form
 //   4  gated, clamped  with g = min(acc[2j], limit), u = clamp(acc[2j+1], -limit, limit):
 //                    C[M, N/2] = g sigmoid(slope g) (u + 1); limit and slope are arguments
+// A bias (float32 [N]) joins every sum before the epilogue.
 #include "common.cuh"
 
 namespace b200 {
@@ -32,7 +33,9 @@ __device__ __forceinline__ float gated_pair(float gate, float up, int epilogue, 
 struct ProductExtras {
     long long a, w, c;
     float gate_limit, gate_slope;   // epilogue 4 alone reads these
+    const float* bias;              // [N] or null
 };
+__device__ __forceinline__ float bias_of(const ProductExtras& x, int n) { return x.bias ? x.bias[n] : 0.f; }
 
 constexpr int kTileM = 64, kTileN = 64, kTileK = 16, kGemmThreads = 256;
 
@@ -83,7 +86,7 @@ gemm_generic_kernel(const TA* __restrict__ A, int lda, const TW* __restrict__ W,
             for (int j = 0; j < 4; j += 2) {
                 const int n = n0 + tx * 4 + j;
                 if (n + 1 < N) {
-                    const float gate = acc[i][j], up = acc[i][j + 1];
+                    const float gate = acc[i][j] + bias_of(batch, n), up = acc[i][j + 1] + bias_of(batch, n + 1);
                     C[(size_t)m * ldc + n / 2] = from_f32<TC>(gated_pair(gate, up, epilogue, batch.gate_limit, batch.gate_slope));
                 }
             }
@@ -93,8 +96,9 @@ gemm_generic_kernel(const TA* __restrict__ A, int lda, const TW* __restrict__ W,
                 const int n = n0 + tx * 4 + j;
                 if (n >= N) continue;
                 TC* c = C + (size_t)m * ldc + n;
-                if (epilogue == 1) *c = from_f32<TC>(to_f32<TC>(*c) + acc[i][j]);
-                else *c = from_f32<TC>(acc[i][j]);
+                const float sum = acc[i][j] + bias_of(batch, n);
+                if (epilogue == 1) *c = from_f32<TC>(to_f32<TC>(*c) + sum);
+                else *c = from_f32<TC>(sum);
             }
         }
     }
@@ -160,7 +164,7 @@ gemm_generic_big_kernel(const TA* __restrict__ A, int lda, const TW* __restrict_
             for (int j = 0; j < 8; j += 2) {
                 const int n = n0 + tx * 8 + j;
                 if (n + 1 < N) {
-                    const float gate = acc[i][j], up = acc[i][j + 1];
+                    const float gate = acc[i][j] + bias_of(batch, n), up = acc[i][j + 1] + bias_of(batch, n + 1);
                     C[(size_t)m * ldc + n / 2] = from_f32<TC>(gated_pair(gate, up, epilogue, batch.gate_limit, batch.gate_slope));
                 }
             }
@@ -170,8 +174,9 @@ gemm_generic_big_kernel(const TA* __restrict__ A, int lda, const TW* __restrict_
                 const int n = n0 + tx * 8 + j;
                 if (n >= N) continue;
                 TC* c = C + (size_t)m * ldc + n;
-                if (epilogue == 1) *c = from_f32<TC>(to_f32<TC>(*c) + acc[i][j]);
-                else *c = from_f32<TC>(acc[i][j]);
+                const float sum = acc[i][j] + bias_of(batch, n);
+                if (epilogue == 1) *c = from_f32<TC>(to_f32<TC>(*c) + sum);
+                else *c = from_f32<TC>(sum);
             }
         }
     }
@@ -258,11 +263,13 @@ gemm_fewrows_kernel(const TA* __restrict__ A, int lda, const TW* __restrict__ W,
     float sum = 0.f;
 #pragma unroll
     for (int wp = 0; wp < kFewWarps; ++wp) sum += part[wp][i];
+    if (batch.bias && n < N) sum += batch.bias[n];
     if (epilogue >= 2) {
         float up = 0.f;   // the gate row's thread also adds up the up row (the next row of the CTA)
         if ((r & 1) == 0) {
 #pragma unroll
             for (int wp = 0; wp < kFewWarps; ++wp) up += part[wp][i + MT];
+            if (batch.bias && n + 1 < N) up += batch.bias[n + 1];
             if (m < M && n + 1 < N) C[(size_t)m * ldc + n / 2] = from_f32<TC>(gated_pair(sum, up, epilogue, batch.gate_limit, batch.gate_slope));
         }
     } else if (m < M && n < N) {
@@ -316,9 +323,9 @@ static int gemm_generic_launch(const void* A, int a_dtype, int lda, const void* 
 
 extern "C" int b200_gemm_generic(const void* A, int a_dtype, int lda, const void* W, int w_dtype, int ldw, void* C,
                                  int c_dtype, int ldc, int M, int N, int K, int epilogue, float gate_limit,
-                                 float gate_slope, cudaStream_t stream) {
+                                 float gate_slope, const float* bias, cudaStream_t stream) {
     return gemm_generic_launch(A, a_dtype, lda, W, w_dtype, ldw, C, c_dtype, ldc, M, N, K, epilogue, 1,
-                               b200::ProductExtras{0, 0, 0, gate_limit, gate_slope}, stream);
+                               b200::ProductExtras{0, 0, 0, gate_limit, gate_slope, bias}, stream);
 }
 
 // n_batch products of the same shape: product z uses A + z a_step, W + z w_step, C + z c_step (steps in elements).
@@ -326,5 +333,5 @@ extern "C" int b200_gemm_generic_batched(const void* A, int a_dtype, int lda, lo
                                          int ldw, long long w_step, void* C, int c_dtype, int ldc, long long c_step, int M,
                                          int N, int K, int n_batch, cudaStream_t stream) {
     return gemm_generic_launch(A, a_dtype, lda, W, w_dtype, ldw, C, c_dtype, ldc, M, N, K, 0, n_batch,
-                               b200::ProductExtras{a_step, w_step, c_step, 0.f, 0.f}, stream);
+                               b200::ProductExtras{a_step, w_step, c_step, 0.f, 0.f, nullptr}, stream);
 }

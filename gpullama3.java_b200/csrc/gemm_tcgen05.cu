@@ -88,6 +88,7 @@ struct RopeEpilogue {
     int gate_act;              // the gated epilogue (EPI 2) alone reads this: 0 SiLU, 1 GELU in its tanh form, of the gate value;
                                // 2 the clamped form g' sigmoid(slope g') (u' + 1), g' = min(g, limit), u' = clamp(u, -limit, limit)
     float gate_limit, gate_slope;
+    const float* bias;         // [N] float32 or null: joins every sum before the store, residual and gated epilogues (not EPI 3)
 };
 
 __device__ __forceinline__ float gated_clamped(float gate, float up, float limit, float slope) {
@@ -208,6 +209,19 @@ __device__ __forceinline__ void epilogue_tile(uint32_t acc, int quarter, int lan
         if (n0 + c0 >= N) break;  // uniform: whole chunk beyond the matrix
         float v[32];
         tmem_ld32(acc + ((uint32_t)(quarter * 32) << 16) + c0, v);
+        if (rope.bias != nullptr) {   // (the same 32 numbers for every row: one broadcast read per column)
+            if (n0 + c0 + 32 <= N && ((uintptr_t)(rope.bias + n0 + c0) & 15) == 0) {
+                const float4* b4 = reinterpret_cast<const float4*>(rope.bias + n0 + c0);
+#pragma unroll
+                for (int j = 0; j < 8; ++j) {
+                    const float4 b = __ldg(b4 + j);
+                    v[4 * j] += b.x; v[4 * j + 1] += b.y; v[4 * j + 2] += b.z; v[4 * j + 3] += b.w;
+                }
+            } else {
+#pragma unroll
+                for (int j = 0; j < 32; ++j) if (n0 + c0 + j < N) v[j] += rope.bias[n0 + c0 + j];
+            }
+        }
         if (EPI == 1 && reduce_c) {
             // the box is free once the reduction before has read it; row `lane` of the box, its eight
             // 16-byte pieces at piece ^ (row % 8): the layout the tensor map's 128-byte swizzle expects
@@ -764,7 +778,7 @@ __device__ __forceinline__ float4 cluster_load_f32x4(uint32_t addr) {
 template <int EPI, typename TC>
 __global__ void __launch_bounds__(kGemmTcThreads, 1)
 gemm_tcgen05_spans_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_w,
-                          TC* __restrict__ C, int ldc, int M, int N, int K, int blocks_per_span) {
+                          TC* __restrict__ C, int ldc, int M, int N, int K, int blocks_per_span, const float* __restrict__ bias) {
     constexpr int BN = kSplitBN, STAGES = kSplitStages;
     using Smem = GemmSmem<BN, STAGES>;
     static_assert(sizeof(float) * BM * kSplitPitch <= sizeof(Smem::a), "the partial tile fits in the stages of A");
@@ -871,6 +885,12 @@ gemm_tcgen05_spans_kernel(const __grid_constant__ CUtensorMap map_a, const __gri
                 }
             }
             if (row >= M || col >= N) continue;
+            if (bias != nullptr) {
+                acc.x += bias[col];
+                if (col + 1 < N) acc.y += bias[col + 1];
+                if (col + 2 < N) acc.z += bias[col + 2];
+                if (col + 3 < N) acc.w += bias[col + 3];
+            }
             const float v[4] = {acc.x, acc.y, acc.z, acc.w};
             if (EPI == 2) {  // columns are gate, up, gate, up
                 TC* dst = C + (size_t)row * ldc + (col >> 1);
@@ -980,17 +1000,16 @@ static int launch_tc(const void* A, int lda, const void* W, int ldw, void* C, in
 
 template <int BN, int STAGES>
 static int launch_width(const void* A, int lda, const void* W, int ldw, void* C, int c_dtype, int ldc, int M, int N, int K,
-                        int epilogue, cudaStream_t stream, int gate_act = 0, float gate_limit = 0.f, float gate_slope = 0.f) {
-    if (epilogue == 2) {
-        RopeEpilogue gated = {};
-        gated.gate_act = gate_act;
-        gated.gate_limit = gate_limit;
-        gated.gate_slope = gate_slope;
-        return launch_tc<BN, STAGES, 2, __nv_bfloat16>(A, lda, W, ldw, C, ldc, M, N, K, stream, gated);
-    }
-    if (epilogue == 1) return launch_tc<BN, STAGES, 1, float>(A, lda, W, ldw, C, ldc, M, N, K, stream);
-    if (c_dtype == kF32) return launch_tc<BN, STAGES, 0, float>(A, lda, W, ldw, C, ldc, M, N, K, stream);
-    return launch_tc<BN, STAGES, 0, __nv_bfloat16>(A, lda, W, ldw, C, ldc, M, N, K, stream);
+                        int epilogue, cudaStream_t stream, int gate_act, float gate_limit, float gate_slope, const float* bias) {
+    RopeEpilogue more = {};
+    more.gate_act = gate_act;
+    more.gate_limit = gate_limit;
+    more.gate_slope = gate_slope;
+    more.bias = bias;
+    if (epilogue == 2) return launch_tc<BN, STAGES, 2, __nv_bfloat16>(A, lda, W, ldw, C, ldc, M, N, K, stream, more);
+    if (epilogue == 1) return launch_tc<BN, STAGES, 1, float>(A, lda, W, ldw, C, ldc, M, N, K, stream, more);
+    if (c_dtype == kF32) return launch_tc<BN, STAGES, 0, float>(A, lda, W, ldw, C, ldc, M, N, K, stream, more);
+    return launch_tc<BN, STAGES, 0, __nv_bfloat16>(A, lda, W, ldw, C, ldc, M, N, K, stream, more);
 }
 
 // How many CTA pairs can run at once (a pair needs two SMs that can form a cluster; each CTA fills its SM).
@@ -1033,17 +1052,16 @@ static int launch_pair(const void* A, int lda, const void* W, int ldw, void* C, 
 
 template <int BN, int STAGES>
 static int launch_pair_width(const void* A, int lda, const void* W, int ldw, void* C, int c_dtype, int ldc, int M, int N, int K,
-                             int epilogue, cudaStream_t stream, int gate_act = 0, float gate_limit = 0.f, float gate_slope = 0.f) {
-    if (epilogue == 2) {
-        RopeEpilogue gated = {};
-        gated.gate_act = gate_act;
-        gated.gate_limit = gate_limit;
-        gated.gate_slope = gate_slope;
-        return launch_pair<BN, STAGES, 2, __nv_bfloat16>(A, lda, W, ldw, C, ldc, M, N, K, stream, gated);
-    }
-    if (epilogue == 1) return launch_pair<BN, STAGES, 1, float>(A, lda, W, ldw, C, ldc, M, N, K, stream);
-    if (c_dtype == kF32) return launch_pair<BN, STAGES, 0, float>(A, lda, W, ldw, C, ldc, M, N, K, stream);
-    return launch_pair<BN, STAGES, 0, __nv_bfloat16>(A, lda, W, ldw, C, ldc, M, N, K, stream);
+                             int epilogue, cudaStream_t stream, int gate_act, float gate_limit, float gate_slope, const float* bias) {
+    RopeEpilogue more = {};
+    more.gate_act = gate_act;
+    more.gate_limit = gate_limit;
+    more.gate_slope = gate_slope;
+    more.bias = bias;
+    if (epilogue == 2) return launch_pair<BN, STAGES, 2, __nv_bfloat16>(A, lda, W, ldw, C, ldc, M, N, K, stream, more);
+    if (epilogue == 1) return launch_pair<BN, STAGES, 1, float>(A, lda, W, ldw, C, ldc, M, N, K, stream, more);
+    if (c_dtype == kF32) return launch_pair<BN, STAGES, 0, float>(A, lda, W, ldw, C, ldc, M, N, K, stream, more);
+    return launch_pair<BN, STAGES, 0, __nv_bfloat16>(A, lda, W, ldw, C, ldc, M, N, K, stream, more);
 }
 
 // Spans of K per tile for the cluster kernel (1: the plain kernel).  Worth it when the 128 x 128 tiles times the spans
@@ -1068,7 +1086,7 @@ static int k_spans_for(int M, int N, int K) {
 
 template <int EPI, typename TC>
 static int launch_spans(const void* A, int lda, const void* W, int ldw, void* C, int ldc, int M, int N, int K, int spans,
-                        cudaStream_t stream) {
+                        cudaStream_t stream, const float* bias) {
     CUtensorMap ma, mw;
     if (!make_map(&ma, A, M, K, lda, BM) || !make_map(&mw, W, N, K, ldw, kSplitBN)) return kErrUnsupportedSize;
     const size_t smem = sizeof(GemmSmem<kSplitBN, kSplitStages>) + 1024;
@@ -1082,7 +1100,7 @@ static int launch_spans(const void* A, int lda, const void* W, int ldw, void* C,
     const int kb = (K + BK - 1) / BK;
     const int tiles = ((N + kSplitBN - 1) / kSplitBN) * ((M + BM - 1) / BM);
     return launch_pdl_cluster(kernel, dim3(tiles, spans), dim3(kGemmTcThreads), smem, stream, dim3(1, spans, 1), true,
-                              ma, mw, (TC*)C, ldc, M, N, K, (kb + spans - 1) / spans);
+                              ma, mw, (TC*)C, ldc, M, N, K, (kb + spans - 1) / spans, bias);
 }
 
 template <int BN, int STAGES, int EPI, typename TC>
@@ -1150,10 +1168,11 @@ extern "C" int b200_gemm_tcgen05_k_spans(int M, int N, int K) {
 // tile_width: 256, 128 or 64 output columns per tile; 0 lets the product's shape decide.
 // k_spans: 2 or 4 cuts K among the CTAs of a cluster (128-column tiles; tile_width is then ignored), 1 never does,
 // 0 lets the shape decide.
+// bias: float32 [N] or null, joins every sum before the epilogue.
 // cta_pair: 1 computes 256-row tiles by pairs of CTAs (tile_width 256 or 128), -1 never does, 0 lets the shape decide.
 extern "C" int b200_gemm_tcgen05(const void* A, int lda, const void* W, int ldw, void* C, int c_dtype, int ldc, int M,
                                  int N, int K, int epilogue, int tile_width, int k_spans, int cta_pair, float gate_limit,
-                                 float gate_slope, cudaStream_t stream) {
+                                 float gate_slope, const float* bias, cudaStream_t stream) {
     using namespace b200;
     if (M <= 0 || N <= 0) return 0;
     if (K < 8 || K % 8 != 0 || lda % 8 != 0 || ldw % 8 != 0 || (((uintptr_t)A | (uintptr_t)W) & 15)) return kErrUnsupportedSize;
@@ -1169,8 +1188,8 @@ extern "C" int b200_gemm_tcgen05(const void* A, int lda, const void* W, int ldw,
     if (c_dtype != kF32 && c_dtype != kBF16) return kErrBadArgument;
     if (k_spans != 0 && k_spans != 1 && k_spans != 2 && k_spans != 4) return kErrBadArgument;
     if (cta_pair > 0) {
-        if (tile_width == 128) return launch_pair_width<128, 8>(A, lda, W, ldw, C, c_dtype, ldc, M, N, K, epilogue, stream, gate_act, gate_limit, gate_slope);
-        if (tile_width == 256 || tile_width == 0) return launch_pair_width<256, 6>(A, lda, W, ldw, C, c_dtype, ldc, M, N, K, epilogue, stream, gate_act, gate_limit, gate_slope);
+        if (tile_width == 128) return launch_pair_width<128, 8>(A, lda, W, ldw, C, c_dtype, ldc, M, N, K, epilogue, stream, gate_act, gate_limit, gate_slope, bias);
+        if (tile_width == 256 || tile_width == 0) return launch_pair_width<256, 6>(A, lda, W, ldw, C, c_dtype, ldc, M, N, K, epilogue, stream, gate_act, gate_limit, gate_slope, bias);
         return kErrBadArgument;
     }
     // left the choice: pairs of CTAs as soon as their 256 x 256 tiles occupy two thirds of the SMs (measured: from there on
@@ -1178,23 +1197,23 @@ extern "C" int b200_gemm_tcgen05(const void* A, int lda, const void* W, int ldw,
     if (cta_pair == 0 && tile_width == 0 && (k_spans == 0 || gate_act != 0)) {
         const long long pair_tiles = (long long)((M + 2 * BM - 1) / (2 * BM)) * ((N + 255) / 256);
         if (pair_tiles * 3 >= (long long)(sm_count() / 2) * 2) {
-            const int st = launch_pair_width<256, 6>(A, lda, W, ldw, C, c_dtype, ldc, M, N, K, epilogue, stream, gate_act, gate_limit, gate_slope);
+            const int st = launch_pair_width<256, 6>(A, lda, W, ldw, C, c_dtype, ldc, M, N, K, epilogue, stream, gate_act, gate_limit, gate_slope, bias);
             if (st != kErrUnsupportedSize) return st;   // (no two SMs that can form a pair: the single-CTA kernels below)
         }
     }
     const int spans = k_spans > 0 ? k_spans : (tile_width > 0 ? 1 : k_spans_for(M, N, K));
     if (spans > 1) {
         if ((K + BK - 1) / BK < spans) return kErrBadArgument;
-        if (epilogue == 2) return launch_spans<2, __nv_bfloat16>(A, lda, W, ldw, C, ldc, M, N, K, spans, stream);
-        if (epilogue == 1) return launch_spans<1, float>(A, lda, W, ldw, C, ldc, M, N, K, spans, stream);
-        if (c_dtype == kF32) return launch_spans<0, float>(A, lda, W, ldw, C, ldc, M, N, K, spans, stream);
-        return launch_spans<0, __nv_bfloat16>(A, lda, W, ldw, C, ldc, M, N, K, spans, stream);
+        if (epilogue == 2) return launch_spans<2, __nv_bfloat16>(A, lda, W, ldw, C, ldc, M, N, K, spans, stream, bias);
+        if (epilogue == 1) return launch_spans<1, float>(A, lda, W, ldw, C, ldc, M, N, K, spans, stream, bias);
+        if (c_dtype == kF32) return launch_spans<0, float>(A, lda, W, ldw, C, ldc, M, N, K, spans, stream, bias);
+        return launch_spans<0, __nv_bfloat16>(A, lda, W, ldw, C, ldc, M, N, K, spans, stream, bias);
     }
     // a stage holds 16 KB of A and BN / 8 KB of W: the narrower the tile, the deeper the ring
     const int width = tile_width > 0 ? tile_width : tile_width_for(M, N);
-    if (width == 256) return launch_width<256, 4>(A, lda, W, ldw, C, c_dtype, ldc, M, N, K, epilogue, stream, gate_act, gate_limit, gate_slope);
-    if (width == 128) return launch_width<128, 6>(A, lda, W, ldw, C, c_dtype, ldc, M, N, K, epilogue, stream, gate_act, gate_limit, gate_slope);
-    if (width == 64) return launch_width<64, 8>(A, lda, W, ldw, C, c_dtype, ldc, M, N, K, epilogue, stream, gate_act, gate_limit, gate_slope);
+    if (width == 256) return launch_width<256, 4>(A, lda, W, ldw, C, c_dtype, ldc, M, N, K, epilogue, stream, gate_act, gate_limit, gate_slope, bias);
+    if (width == 128) return launch_width<128, 6>(A, lda, W, ldw, C, c_dtype, ldc, M, N, K, epilogue, stream, gate_act, gate_limit, gate_slope, bias);
+    if (width == 64) return launch_width<64, 8>(A, lda, W, ldw, C, c_dtype, ldc, M, N, K, epilogue, stream, gate_act, gate_limit, gate_slope, bias);
     return kErrBadArgument;
 }
 
@@ -1216,7 +1235,7 @@ extern "C" int b200_gemm_tcgen05_qkv_rope(const void* A, int lda, const void* W,
         return kErrUnsupportedSize;
     if (write_cache && (k_pool == nullptr || v_pool == nullptr)) return kErrBadArgument;
     const int N = (n_heads + 2 * n_kv_heads) * head_dim;
-    RopeEpilogue rope;
+    RopeEpilogue rope = {};
     rope.positions = positions; rope.seq_ids = seq_ids; rope.page_table = page_table; rope.table_stride = table_stride;
     rope.angles = reinterpret_cast<const float2*>(angles);
     rope.n_tokens = M;

@@ -14,6 +14,8 @@
 //     (z[2i], z[2i+1]) <- turned by position * inv_freq[i]   (optional: rotary position encoding over the row's interleaved
 //                                                   pairs, the angle, its cosine and sine in 32 bits; `mul` then also carries
 //                                                   a factor on cosine and sine)
+//     or, over halves: (z[i], z[i + n]) <- turned by position * inv_freq[f + i] for i < n, the columns from 2 n on as they
+//                                                   are; every segment with frequencies (f) and pairs (n) of its own
 // A segment's rows need not lie back to back (`src_stride`: a part of every head of a wider projection; 0 as a stride:
 // every row reads the same numbers, one row shared by all heads) nor be written back to back (`dst_stride`), and a row may
 // fill only some columns of a cache row (`dst_off` columns in, `cache_dim` the cache's row size), so that two segments can
@@ -29,7 +31,7 @@
 namespace b200 {
 
 constexpr int kRowSegments = 6;
-constexpr int kSegmentWords = 20;   // 32-bit words of one segment record at the C interface (17 used)
+constexpr int kSegmentWords = 20;   // 32-bit words of one segment record at the C interface (19 used)
 constexpr int kRowThreads = 128;
 
 struct RowSegment {
@@ -41,10 +43,12 @@ struct RowSegment {
     int target;       // 0: dst; 1: key rows of the cache; 2: value rows of the cache
     int weight_per_row;  // 1: the weight has n_rows * d entries (one per element of the segment), 0: d (shared by the rows)
     int mix_off;      // column of `other` where this segment's counterpart starts, -1: no mixing
-    int rotate;       // 1: the row's pairs (2i, 2i + 1) are turned by position * inv_freq[i] (d even, no mixing)
+    int rotate;       // 1: the row's pairs (2i, 2i + 1) are turned by position * inv_freq[i] (d even, no mixing);
+                      // 2: its pairs (i, i + pairs), i < pairs, by position * inv_freq[freq_off + i]
     int src_stride;   // numbers between two rows of the source (-1: d)
     int dst_stride;   // numbers between two rows written to dst (-1: d_pad)
     int cache_dim;    // row size of the cache the segment goes into (-1: d_pad); the segment starts dst_off columns in
+    int pairs, freq_off;   // rotate 2 alone reads these
     int lead;         // zeros written in front of the row: of the d_pad numbers the first `lead` are zero, then the d, then zeros
 };
 struct MixSource {
@@ -110,6 +114,20 @@ __device__ __forceinline__ void head_row(const T* __restrict__ src, int ld_src, 
         for (int e = lane; e < g.lead; e += 32) o[(size_t)e * step] = from_f32<T>(0.f);
         o += (size_t)g.lead * step;
         d_pad -= g.lead;
+    }
+    if (g.rotate == 2) {
+        const float pos = (float)cache.positions[t];
+        const int n = g.pairs;
+        auto value = [&](int e) { return (to_f32<T>(x[e]) + (b ? b[e] : 0.f)) * factor * (w ? w[e] : 1.f); };
+        for (int i = lane; i < n; i += 32) {
+            const float u = value(i), v = value(i + n);
+            float sn, cs;
+            sincosf(pos * cache.inv_freq[g.freq_off + i], &sn, &cs);
+            o[(size_t)i * step] = from_f32<T>(u * cs - v * sn);
+            o[(size_t)(i + n) * step] = from_f32<T>(v * cs + u * sn);
+        }
+        for (int e = 2 * n + lane; e < d_pad; e += 32) o[(size_t)e * step] = from_f32<T>(e < g.d ? value(e) : 0.f);
+        return;
     }
     if (g.rotate) {
         const float pos = (float)cache.positions[t];
@@ -197,7 +215,7 @@ head_rows_token_kernel(const T* __restrict__ src, int ld_src, T* __restrict__ ds
 }  // namespace b200
 
 // `segments`: n_segments records of twenty 32-bit words each (src_off, n_rows, d, dst_off, d_pad, bias_off, norm,
-// weight_off, mul as float bits, target, weight_per_row, mix_off, rotate, src_stride, dst_stride, cache_dim, lead; the rest
+// weight_off, mul as float bits, target, weight_per_row, mix_off, rotate, src_stride, dst_stride, cache_dim, lead, pairs, freq_off; the rest
 // unused), read on the host.  Segments with a cache target need positions, seq_ids,
 // page_table and the pools; their n_rows is the number of kv heads of the cache entry and d_pad its head size.
 extern "C" int b200_head_rows(const void* src, int ld_src, void* dst, int ld_dst, int dtype, const float* bias,
@@ -221,8 +239,12 @@ extern "C" int b200_head_rows(const void* src, int ld_src, void* dst, int ld_dst
         g.weight_per_row = p[10];
         g.mix_off = p[11];
         g.rotate = p[12]; g.src_stride = p[13]; g.dst_stride = p[14]; g.cache_dim = p[15]; g.lead = p[16];
+        g.pairs = p[17]; g.freq_off = p[18];
         if (g.lead < 0 || g.lead + g.d > g.d_pad) return b200::kErrBadArgument;
-        if (g.rotate && (!inv_freq || !positions || g.d % 2 || g.mix_off >= 0)) return b200::kErrBadArgument;
+        if (g.rotate && (!inv_freq || !positions || g.mix_off >= 0)) return b200::kErrBadArgument;
+        if (g.rotate == 1 && g.d % 2) return b200::kErrBadArgument;
+        if (g.rotate == 2 && (g.pairs < 0 || 2 * g.pairs > g.d || g.freq_off < 0)) return b200::kErrBadArgument;
+        if (g.rotate < 0 || g.rotate > 2) return b200::kErrBadArgument;
         if (g.cache_dim >= 0 && (g.target == 0 || g.dst_off < 0 || g.dst_off + g.d_pad > g.cache_dim)) return b200::kErrBadArgument;
         if (g.norm < 0 || g.norm > 2) return b200::kErrBadArgument;
         if (g.mix_off >= 0 && (other == nullptr || lambda == nullptr)) return b200::kErrBadArgument;

@@ -3,7 +3,8 @@
 // as inference/InferenceCore.java:47-56 of the reference project computes it (eps inside the root,
 // added after the mean; the weight multiplies plainly).  The sum of squares and the scale are
 // 32-bit whatever the storage types.  `rows` (optional) selects which rows of x are normalised,
-// so that only the positions whose logits are wanted reach the output head.
+// so that only the positions whose logits are wanted reach the output head.  rmsnorm_pair: two norms of the same rows
+// that differ in their weights alone (a block whose two sublayers read the stream side by side), one read of the row.
 #include "common.cuh"
 
 namespace b200 {
@@ -131,6 +132,80 @@ template <typename TW, typename TO, int KEEP>
 static int launch_norm_warp(const float* x, const void* w, void* out, const int* rows, int n_rows, float eps, cudaStream_t stream) {
     return launch_pdl(rmsnorm_warp_kernel<TW, TO, KEEP>, dim3((n_rows + kNormWarps - 1) / kNormWarps), dim3(kNormWarps * 32), 0,
                       stream, x, (const TW*)w, (TO*)out, rows, n_rows, eps);
+}
+
+// Two norms of the same rows: out1 = w1 x r and out2 = w2 x r with the one r = 1 / sqrt(mean(x^2) + eps).  Weights are 32-bit.
+// KEEP > 0: a warp per row of 128 * KEEP numbers held in registers; KEEP = 0: a CTA per row of any length.
+template <typename TO, int KEEP>
+__global__ void __launch_bounds__(kNormThreads)
+rmsnorm_pair_kernel(const float* __restrict__ x, const float* __restrict__ w1, const float* __restrict__ w2, TO* __restrict__ out1,
+                    TO* __restrict__ out2, int n_rows, int dim, float eps) {
+    pdl_launch_dependents();
+    pdl_wait();
+    if constexpr (KEEP > 0) {
+        const int lane = threadIdx.x & 31, r = blockIdx.x * (kNormThreads / 32) + (threadIdx.x >> 5);
+        if (r >= n_rows) return;
+        const float* xr = x + (size_t)r * dim;
+        float keep[KEEP > 0 ? KEEP : 1][4], ss = 0.f;
+#pragma unroll
+        for (int k = 0; k < KEEP; ++k) load4<float>(xr + (k * 32 + lane) * 4, keep[k]);
+#pragma unroll
+        for (int k = 0; k < KEEP; ++k)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) ss += keep[k][e] * keep[k][e];
+        ss = warp_sum(ss);
+        const float scale = 1.0f / sqrtf(ss / (float)dim + eps);
+#pragma unroll
+        for (int which = 0; which < 2; ++which) {
+            const float* w = which ? w2 : w1;
+            TO* o = (which ? out2 : out1) + (size_t)r * dim;
+#pragma unroll
+            for (int k = 0; k < KEEP; ++k) {
+                float wv[4], y[4];
+                load4<float>(w + (k * 32 + lane) * 4, wv);
+#pragma unroll
+                for (int e = 0; e < 4; ++e) y[e] = wv[e] * (scale * keep[k][e]);
+                store4<TO>(o + (k * 32 + lane) * 4, y);
+            }
+        }
+    } else {
+        __shared__ float scratch[33];
+        const float* xr = x + (size_t)blockIdx.x * dim;
+        constexpr int kKeep = 8;    // numbers a thread keeps between the two passes
+        float keep[kKeep], ss = 0.f;
+#pragma unroll
+        for (int k = 0; k < kKeep; ++k) {
+            const int i = k * kNormThreads + threadIdx.x;
+            keep[k] = i < dim ? xr[i] : 0.f;
+            ss += keep[k] * keep[k];
+        }
+        for (int i = kKeep * kNormThreads + threadIdx.x; i < dim; i += kNormThreads) ss += xr[i] * xr[i];
+        ss = block_sum(ss, scratch);
+        const float scale = 1.0f / sqrtf(ss / (float)dim + eps);
+        TO* o1 = out1 + (size_t)blockIdx.x * dim;
+        TO* o2 = out2 + (size_t)blockIdx.x * dim;
+#pragma unroll
+        for (int k = 0; k < kKeep; ++k) {
+            const int i = k * kNormThreads + threadIdx.x;
+            if (i < dim) {
+                o1[i] = from_f32<TO>(w1[i] * (scale * keep[k]));
+                o2[i] = from_f32<TO>(w2[i] * (scale * keep[k]));
+            }
+        }
+        for (int i = kKeep * kNormThreads + threadIdx.x; i < dim; i += kNormThreads) {
+            const float v = scale * xr[i];
+            o1[i] = from_f32<TO>(w1[i] * v);
+            o2[i] = from_f32<TO>(w2[i] * v);
+        }
+    }
+}
+
+template <typename TO, int KEEP>
+static int launch_norm_pair(const float* x, const float* w1, const float* w2, void* out1, void* out2, int n_rows, int dim, float eps,
+                            cudaStream_t stream) {
+    const int per_cta = KEEP > 0 ? kNormThreads / 32 : 1;
+    return launch_pdl(rmsnorm_pair_kernel<TO, KEEP>, dim3((n_rows + per_cta - 1) / per_cta), dim3(kNormThreads), 0, stream, x, w1, w2,
+                      (TO*)out1, (TO*)out2, n_rows, dim, eps);
 }
 
 // Layer norm with weight and bias over rows of the 32-bit residual stream:
@@ -301,5 +376,25 @@ extern "C" int b200_layernorm(const float* x, const float* w, const float* b, vo
                                       (TO*)out, rows, dim, eps)
                    : b200::launch_pdl(b200::layernorm_kernel<TO, false>, dim3(n_rows), dim3(b200::kNormThreads), 0, stream, x, w, b,
                                       (TO*)out, rows, dim, eps));
+    return b200::launch_status();
+}
+
+// out1 and out2 (of one type) receive the rows under the two weights (32-bit, [dim] each).
+extern "C" int b200_rmsnorm_pair(const float* x, const float* w1, const float* w2, void* out1, void* out2, int out_dtype, int n_rows,
+                                 int dim, float eps, cudaStream_t stream) {
+    if (n_rows <= 0) return 0;
+    if (dim < 1 || !w1 || !w2) return b200::kErrBadArgument;
+    const bool vec = ((((uintptr_t)x) | ((uintptr_t)w1) | ((uintptr_t)w2) | ((uintptr_t)out1) | ((uintptr_t)out2)) & 15) == 0;
+    if (vec && n_rows >= 1024 && dim % 1024 == 0 && dim <= 4096) {
+        B200_DISPATCH_DTYPE(out_dtype, TO,
+            switch (dim / 1024) {
+                case 1: return b200::launch_norm_pair<TO, 8>(x, w1, w2, out1, out2, n_rows, dim, eps, stream);
+                case 2: return b200::launch_norm_pair<TO, 16>(x, w1, w2, out1, out2, n_rows, dim, eps, stream);
+                case 3: return b200::launch_norm_pair<TO, 24>(x, w1, w2, out1, out2, n_rows, dim, eps, stream);
+                default: return b200::launch_norm_pair<TO, 32>(x, w1, w2, out1, out2, n_rows, dim, eps, stream);
+            });
+    }
+    B200_DISPATCH_DTYPE(out_dtype, TO,
+        return b200::launch_norm_pair<TO, 0>(x, w1, w2, out1, out2, n_rows, dim, eps, stream));
     return b200::launch_status();
 }

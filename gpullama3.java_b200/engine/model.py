@@ -26,6 +26,8 @@ class CausalLM:
             raise ConfigError(f"the engine runs in float32 or bfloat16, not {dtype}")
         self.config, self.dtype, self.device = config, dtype, torch.device(device)
         self.embedding = TokenEmbedding(config.vocab_size, config.hidden_size, scale=config.embedding_scale())
+        norm = config.embedding_norm()
+        self.embedding_norm = build_part(norm) if norm is not None else None
         self.blocks: list[Block] = [build_block(s) for s in config.layer_specs()]
         self.final_norm = build_part(config.final_norm())
         self.head = OutputHead(config.vocab_size, config.hidden_size,
@@ -89,6 +91,9 @@ class CausalLM:
         """Every part by its path: ``embedding``, ``layers.3.mixer``, ``layers.3.mixer.position``, ..."""
         parts: dict[str, Part] = {"embedding": self.embedding}
         parts.update(all_parts(self.embedding, "embedding."))
+        if self.embedding_norm is not None:
+            parts["embedding_norm"] = self.embedding_norm
+            parts.update(all_parts(self.embedding_norm, "embedding_norm."))
         for i, b in enumerate(self.blocks):
             if b.parameters():      # a block with parameters of its own (``layers.3.<name>``), beside those of its parts
                 parts[f"layers.{i}"] = b
@@ -131,7 +136,7 @@ class CausalLM:
             for pname in part.parameters():
                 local[pname] = by_checkpoint_name[names[f"{path}.{pname}"]]
             part.load(local, self.dtype, self.device)
-        self.loaded = True
+        self._after_load()
 
     def load_folder(self, model_dir: str | Path) -> None:
         expected = {name: spec.shape for name, spec in self.checkpoint_specs().items()}
@@ -152,6 +157,15 @@ class CausalLM:
                 local[pname] = random_tensor(cname, specs[cname], seed, self.config.init_std(), norm_std, store_dtype,
                                              self.device)
             part.load(local, self.dtype, self.device)
+        self._after_load()
+
+    def _after_load(self) -> None:
+        """Every part has its weights: parts may now join theirs with those of the parts they were built with."""
+        seen: set[int] = set()
+        for part in [*reversed(self.named_parts().values()), *self.blocks]:   # (children come before their parents)
+            if id(part) not in seen:
+                seen.add(id(part))
+                part.after_load()
         self.loaded = True
 
     # ---- one forward pass over a packed batch
@@ -162,6 +176,8 @@ class CausalLM:
             raise WeightError("the model has no weights yet (load_folder / load_random / load_tensors)")
         ws = ctx.workspace
         residual = self.embedding.forward(ctx.tokens, ctx.empty)  # float32 [T, hidden]; lives for the whole pass
+        if self.embedding_norm is not None:
+            residual = self.embedding_norm.forward(residual, torch.float32, alloc=ctx.empty)
         if self.streams is not None:
             residual = open_streams(residual, self.streams, ctx.empty)   # [T, streams, hidden]
         # a block may leave the first norm of the block that runs next to that block's first product

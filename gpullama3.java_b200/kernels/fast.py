@@ -11,12 +11,20 @@ import torch
 from . import ops
 
 
-def try_gemm(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, epilogue: int, gate_args=(0.0, 0.0)) -> bool:
+def try_gemm(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, epilogue: int, gate_args=(0.0, 0.0), bias=None) -> bool:
     if a.dtype != torch.bfloat16 or w.dtype != torch.bfloat16:
         return False
     M = a.shape[0]
     if M <= 16:
-        return ops.gemm_decode(a, w, c, epilogue, gate_args)
+        return ops.gemm_decode(a, w, c, epilogue, gate_args, bias)
+    if bias is not None:
+        # (the few-token tensor-core kernel has no bias: what it adds to the residual stream gets the bias behind it)
+        if M <= 128 and epilogue == ops.EPILOGUE_RESIDUAL_ADD and c.is_contiguous() and ops.gemm_skinny(a, w, c, epilogue):
+            ops.add_row(c, bias)
+            return True
+        if M <= 64 and ops.gemm_decode(a, w, c, epilogue, gate_args, bias):
+            return True
+        return ops.gemm_tcgen05(a, w, c, epilogue, gate_args=gate_args, bias=bias)
     # (the few-token tensor-core kernel has the gated epilogue with SiLU only; the other activations' sizes go to the other two)
     if M <= 128 and epilogue in (ops.EPILOGUE_STORE, ops.EPILOGUE_RESIDUAL_ADD, ops.EPILOGUE_GATED_SILU) and ops.gemm_skinny(a, w, c, epilogue):
         return True
@@ -55,9 +63,10 @@ def try_decode_attention_with_rope(qkv, out, ctx, page_table, cache, mixer, writ
 
 def try_attention(qkv, out, ctx, page_table, cache, mixer, gate=None) -> bool:
     if getattr(mixer, "has_terms", False):
-        # kept first positions, distance penalty, sink, output gate: the span kernel for decode steps, the flash kernel
-        # for prompts (the tcgen05 prompt kernel does not have these terms)
-        terms = dict(keep_first=mixer.keep_first, slopes=mixer.slopes, sinks=mixer.sinks, gate=gate)
+        # kept first positions, runs of positions, distance penalty, sink, output gate: the span kernel for decode steps, for
+        # prompts the tcgen05 kernel where runs and sink are all there is (heads of 64 and 128), else the flash kernel
+        chunk = getattr(mixer, "chunk", None) or 0
+        terms = dict(keep_first=mixer.keep_first, chunk=chunk, slopes=mixer.slopes, sinks=mixer.sinks, gate=gate)
         if qkv.dtype != torch.bfloat16 or mixer.head_dim not in (32, 64, 96, 128):
             return False
         if ctx.all_decode and ops.attention_decode_supported(qkv.dtype, mixer.n_heads, mixer.n_kv_heads, mixer.head_dim):
@@ -67,6 +76,10 @@ def try_attention(qkv, out, ctx, page_table, cache, mixer, gate=None) -> bool:
             return True
         if qkv.shape[1] % 8 or (qkv.data_ptr() & 15):
             return False
+        if not mixer.keep_first and mixer.slopes is None and gate is None and ops.attention_prefill_tc(
+                qkv, qkv.shape[1], out, ctx.cu_seqlens, ctx.kv_lens, page_table, cache.k, cache.v, ctx.n_seqs, ctx.max_q_len,
+                mixer.n_heads, mixer.n_kv_heads, mixer.head_dim, mixer.window or 0, chunk=chunk, sinks=mixer.sinks):
+            return True
         ops.attention_prefill(qkv, qkv.shape[1], out, ctx.cu_seqlens, ctx.kv_lens, page_table, cache.k, cache.v,
                               ctx.n_seqs, ctx.max_q_len, mixer.n_heads, mixer.n_kv_heads, mixer.head_dim,
                               mixer.window or 0, **terms)

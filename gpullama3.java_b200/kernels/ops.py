@@ -40,19 +40,19 @@ _SIGNATURES = {
                                              c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int]),
     "b200_attention_paged": ("attention_generic", [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
                                                    c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
-                                                   c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int]),
+                                                   c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int]),
     "b200_gemm_generic": ("gemm_generic", [c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_void_p, c_int, c_int,
-                                           c_int, c_int, c_int, c_int, c_float, c_float]),
+                                           c_int, c_int, c_int, c_int, c_float, c_float, c_void_p]),
     "b200_gemm_generic_batched": ("gemm_generic", [c_void_p, c_int, c_int, ctypes.c_longlong, c_void_p, c_int, c_int,
                                                    ctypes.c_longlong, c_void_p, c_int, c_int, ctypes.c_longlong, c_int, c_int,
                                                    c_int, c_int]),
     "b200_gemm_decode": ("gemm_decode", [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int,
-                                         c_int, c_float, c_float]),
+                                         c_int, c_float, c_float, c_void_p]),
     "b200_gemm_decode_linked": ("gemm_decode", [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int,
                                                 c_int, c_int, c_void_p, c_int, c_float, c_int, c_void_p, c_int, c_void_p,
-                                                c_int, c_void_p]),
+                                                c_int, c_void_p, c_void_p, c_void_p, c_void_p]),
     "b200_gemm_tcgen05": ("gemm_tcgen05", [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int,
-                                           c_int, c_int, c_int, c_int, c_float, c_float]),
+                                           c_int, c_int, c_int, c_int, c_float, c_float, c_void_p]),
     "b200_gemm_tcgen05_grouped": ("gemm_tcgen05", [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
                                                    c_void_p, c_int, c_float, c_float]),
     "b200_gemm_tcgen05_qkv_rope": ("gemm_tcgen05", [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p,
@@ -66,16 +66,16 @@ _SIGNATURES = {
                                                    c_int, c_int, c_int]),
     "b200_attention_decode_terms": ("attention_decode", [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
                                                          c_void_p, c_void_p, ctypes.c_longlong, c_int, c_int, c_int, c_int,
-                                                         c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int]),
+                                                         c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int]),
     "b200_attention_prefill": ("attention_prefill", [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
                                                      c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
-                                                     c_void_p, c_void_p, c_void_p, c_int]),
+                                                     c_int, c_void_p, c_void_p, c_void_p, c_int]),
     "b200_attention_decode_rope": ("attention_decode", [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
                                                         c_void_p, c_void_p, ctypes.c_longlong, c_int, c_int, c_int,
                                                         c_int, c_int, c_int, c_void_p, c_int, c_int, c_int]),
     "b200_attention_prefill_tc": ("attention_prefill_tcgen05", [c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p,
                                                                 c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int,
-                                                                c_int, c_int, c_int, c_int]),
+                                                                c_int, c_int, c_int, c_int, c_int, c_void_p]),
     "b200_random_fill": ("random_init", [c_void_p, c_int, ctypes.c_longlong, ctypes.c_ulonglong, c_float, c_float]),
     "b200_streams_combine": ("streams", [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int]),
     "b200_streams_read_norm": ("streams", [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int,
@@ -87,7 +87,10 @@ _SIGNATURES = {
                                      c_void_p, c_void_p]),
     "b200_softcap_rows": ("elementwise", [c_void_p, ctypes.c_longlong, c_float]),
     "b200_gated_rmsnorm": ("elementwise", [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int,
-                                           c_float, c_int, c_int, c_int]),
+                                           c_float, c_int, c_int, c_int, c_int, c_float]),
+    "b200_turn_back_rows": ("elementwise", [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
+                                            c_float]),
+    "b200_rmsnorm_pair": ("norm", [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_float]),
     "b200_gate_rows": ("elementwise", [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int]),
     "b200_scale_rows": ("elementwise", [c_void_p, ctypes.c_longlong, c_float]),
     "b200_group_rmsnorm": ("sandwich", [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_float]),
@@ -102,7 +105,8 @@ _SIGNATURES = {
                                         c_int]),
     "b200_linear_scan": ("delta_rule", [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p,
                                         c_void_p, c_void_p, ctypes.c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
-                                        c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_int, c_int]),
+                                        c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_int, c_int, c_int, c_int,
+                                        c_int, c_void_p, c_void_p]),
     "b200_moe_table_route": ("moe", [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int]),
     "b200_layernorm": ("norm", [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_float]),
     "b200_causal_conv_silu": ("delta_rule", [c_void_p, c_int, c_void_p, c_void_p, ctypes.c_longlong, c_void_p, c_void_p,
@@ -260,6 +264,17 @@ def rmsnorm(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, eps: float
                                float(eps), _stream()), "rmsnorm")
 
 
+def rmsnorm_pair(x: torch.Tensor, weights, outs, eps: float) -> None:
+    """outs[i] = weights[i] * x / sqrt(mean(x^2) + eps) for i = 0, 1: two norms of the same rows in one read.  x [T, dim] and
+    the weights float32, the results of one type."""
+    (w1, w2), (o1, o2) = weights, outs
+    _dev(x, w1, w2, o1, o2)
+    assert x.dtype == w1.dtype == w2.dtype == torch.float32 and x.is_contiguous() and o1.is_contiguous() and o2.is_contiguous()
+    assert o1.dtype == o2.dtype and o1.shape == o2.shape == x.shape and w1.numel() == w2.numel() == x.shape[1]
+    _check(_fn("b200_rmsnorm_pair")(x.data_ptr(), w1.data_ptr(), w2.data_ptr(), o1.data_ptr(), o2.data_ptr(), dtype_code(o1.dtype),
+                                    x.shape[0], x.shape[1], float(eps), _stream()), "rmsnorm_pair")
+
+
 def layernorm(x: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor, out: torch.Tensor, eps: float,
               rows: torch.Tensor | None = None) -> None:
     """out[r] = (x[rows[r]] - mean) / sqrt(mean((x - mean)^2) + eps) * weight + bias.  x, weight, bias float32."""
@@ -301,14 +316,15 @@ def rope_cache_write(qkv: torch.Tensor, positions: torch.Tensor, seq_ids: torch.
 def attention_paged(q: torch.Tensor, q_row_stride: int, out: torch.Tensor, positions: torch.Tensor,
                     seq_ids: torch.Tensor, page_table: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor,
                     n_heads: int, n_kv_heads: int, head_dim: int, window: int = 0, n_splits: int = 1, *,
-                    keep_first: int = 0, slopes: torch.Tensor | None = None, sinks: torch.Tensor | None = None,
-                    gate: torch.Tensor | None = None) -> None:
+                    keep_first: int = 0, chunk: int = 0, slopes: torch.Tensor | None = None,
+                    sinks: torch.Tensor | None = None, gate: torch.Tensor | None = None) -> None:
     """Causal grouped-query attention of every token of ``q`` over the cached keys 0..position of
     its sequence.  q: rows of ``q_row_stride`` elements whose first H*D are the rotated queries.
     ``n_splits`` > 1 cuts every token's keys into that many spans, one CTA each, merged by a second kernel (a decode
     step: few tokens, long rows of keys).  ``keep_first``: positions below it stay visible behind the window;
     ``slopes`` float32 [H]: score -= slopes[h] * distance; ``sinks`` float32 [H]: exp(sinks[h]) joins the softmax's
-    denominator; ``gate`` [T, >= H] of q's dtype: head outputs are multiplied by sigmoid(gate[t, h])."""
+    denominator; ``gate`` [T, >= H] of q's dtype: head outputs are multiplied by sigmoid(gate[t, h]).  ``chunk`` (in place of a
+    window): positions are cut into runs of that many, counted from 0, and a query sees the keys of its own run."""
     _dev(q, out, positions, seq_ids, page_table, k_pool, v_pool)
     assert out.is_contiguous() and out.shape[1] == n_heads * head_dim and out.dtype == q.dtype == k_pool.dtype
     assert tuple(k_pool.shape[1:]) == (n_kv_heads, PAGE_TOKENS, head_dim)
@@ -325,7 +341,7 @@ def attention_paged(q: torch.Tensor, q_row_stride: int, out: torch.Tensor, posit
         q.data_ptr(), q_row_stride, out.data_ptr(), dtype_code(q.dtype), positions.data_ptr(), seq_ids.data_ptr(),
         page_table.data_ptr(), page_table.shape[1], k_pool.data_ptr(), v_pool.data_ptr(), out.shape[0], n_heads,
         n_kv_heads, head_dim, int(window), int(n_splits), scratch.data_ptr() if scratch is not None else None,
-        int(keep_first), ptr(slopes), ptr(sinks), ptr(gate), gate.stride(0) if gate is not None else 0, _stream()),
+        int(keep_first), int(chunk), ptr(slopes), ptr(sinks), ptr(gate), gate.stride(0) if gate is not None else 0, _stream()),
         "attention_paged")
 
 
@@ -338,10 +354,19 @@ ACTIVATION_CODES = {"silu": 0, "gelu_tanh": 1, "clamped_sigmoid": 2}
 GATED_EPILOGUE_OF = {"silu": EPILOGUE_GATED_SILU, "gelu_tanh": EPILOGUE_GATED_GELU_TANH, "clamped_sigmoid": EPILOGUE_GATED_CLAMPED}
 
 
+def _bias_ptr(bias: torch.Tensor | None, n: int):
+    """A product's bias: float32, one number per output row of the weight, joined before the epilogue."""
+    if bias is None:
+        return None
+    assert bias.is_cuda and bias.dtype == torch.float32 and bias.is_contiguous() and bias.numel() == n
+    return bias.data_ptr()
+
+
 def gemm_generic(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, epilogue: int = EPILOGUE_STORE,
-                 gate_args: tuple[float, float] = (0.0, 0.0)) -> None:
+                 gate_args: tuple[float, float] = (0.0, 0.0), bias: torch.Tensor | None = None) -> None:
     """c = a @ w.T (store), c += a @ w.T (residual add, c float32) or c = act(gate) * up with
-    gate/up rows interleaved in w (act: SiLU, or GELU in its tanh form).  32-bit FMA accumulation, no tensor cores."""
+    gate/up rows interleaved in w (act: SiLU, or GELU in its tanh form).  32-bit FMA accumulation, no tensor cores.
+    ``bias`` float32 [w.shape[0]] joins every sum before the epilogue."""
     _dev(a, w, c)
     M, K = a.shape
     N = w.shape[0]
@@ -349,8 +374,8 @@ def gemm_generic(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, epilogue: in
     assert c.shape[0] == M and c.shape[1] == (N // 2 if epilogue in GATED_EPILOGUES else N)
     _check(_fn("b200_gemm_generic")(
         a.data_ptr(), dtype_code(a.dtype), a.stride(0), w.data_ptr(), dtype_code(w.dtype), w.stride(0), c.data_ptr(),
-        dtype_code(c.dtype), c.stride(0), M, N, K, epilogue, float(gate_args[0]), float(gate_args[1]), _stream()),
-        "gemm_generic")
+        dtype_code(c.dtype), c.stride(0), M, N, K, epilogue, float(gate_args[0]), float(gate_args[1]),
+        _bias_ptr(bias, N), _stream()), "gemm_generic")
 
 
 def gemm_per_head(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor) -> None:
@@ -367,7 +392,7 @@ def gemm_per_head(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor) -> None:
 
 
 def gemm_decode(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, epilogue: int = EPILOGUE_STORE,
-                gate_args: tuple[float, float] = (0.0, 0.0)) -> bool:
+                gate_args: tuple[float, float] = (0.0, 0.0), bias: torch.Tensor | None = None) -> bool:
     """The decode-step matrix product (bfloat16 operands, at most 64 tokens, K a multiple of 32).
     Returns False, having done nothing, for operands it does not take."""
     M, K = a.shape
@@ -380,7 +405,7 @@ def gemm_decode(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, epilogue: int
     assert c.shape[1] == (N // 2 if epilogue in GATED_EPILOGUES else N)
     _check(_fn("b200_gemm_decode")(a.data_ptr(), a.stride(0), w.data_ptr(), w.stride(0), c.data_ptr(),
                                    dtype_code(c.dtype), c.stride(0), M, N, K, epilogue, float(gate_args[0]),
-                                   float(gate_args[1]), _stream()), "gemm_decode")
+                                   float(gate_args[1]), _bias_ptr(bias, N), _stream()), "gemm_decode")
     return True
 
 
@@ -397,14 +422,15 @@ def gemm_decode_partials(n_rows: int, n_out: int) -> int:
 
 
 def gemm_decode_linked(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, epilogue: int, *, row_factors=None,
-                       emit=None) -> None:
+                       emit=None, emit_second=None, bias: torch.Tensor | None = None) -> None:
     """``gemm_decode`` as one half, or both, of an RMSNorm split between two products (at most 16 rows).
 
     ``row_factors = (partials [M, P] float32, eps, dim)``: the rows of ``a`` are x * w of a norm; every
     sum of row t is multiplied by rsqrt(sum(partials[t]) / dim + eps) before the epilogue.
     ``emit = (norm_weight [N], act [M, N] bfloat16, partials [M, gemm_decode_partials(M, N)] float32)``
     (residual epilogue only): after c += a w^T, act = bfloat16(c * norm_weight) and partials hold each
-    CTA's sum of c^2 per row."""
+    CTA's sum of c^2 per row.  ``emit_second = (norm_weight, act)``: a second norm's weights (of the same type) over the same
+    rows, its copy of them beside the first.  ``bias`` float32 [N] joins every sum before the epilogue."""
     M, K = a.shape
     N = w.shape[0]
     _dev(a, w, c)
@@ -424,15 +450,21 @@ def gemm_decode_linked(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, epilog
         assert part_out.dtype == torch.float32 and part_out.is_contiguous()
         assert tuple(part_out.shape) == (M, gemm_decode_partials(M, N))
         out_w, out_w_dtype, out_act, ld_act, out_p = nw.data_ptr(), dtype_code(nw.dtype), act.data_ptr(), act.stride(0), part_out.data_ptr()
+    out_w2, out_act2 = None, None
+    if emit_second is not None:
+        nw2, act2 = emit_second
+        assert emit is not None and nw2.dtype == emit[0].dtype and nw2.numel() == N and nw2.is_contiguous()
+        assert act2.dtype == torch.bfloat16 and act2.shape == (M, N) and act2.stride() == emit[1].stride()
+        out_w2, out_act2 = nw2.data_ptr(), act2.data_ptr()
     _check(_fn("b200_gemm_decode_linked")(
         a.data_ptr(), a.stride(0), w.data_ptr(), w.stride(0), c.data_ptr(), dtype_code(c.dtype), c.stride(0), M, N, K,
-        epilogue, in_p, n_in, float(eps), int(dim), out_w, out_w_dtype, out_act, ld_act, out_p, _stream()),
-        "gemm_decode_linked")
+        epilogue, in_p, n_in, float(eps), int(dim), out_w, out_w_dtype, out_act, ld_act, out_p, out_w2, out_act2,
+        _bias_ptr(bias, N), _stream()), "gemm_decode_linked")
 
 
 def gemm_tcgen05(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, epilogue: int = EPILOGUE_STORE,
                  tile_width: int = 0, k_spans: int = 0, cta_pair: int = 0,
-                 gate_args: tuple[float, float] = (0.0, 0.0)) -> bool:
+                 gate_args: tuple[float, float] = (0.0, 0.0), bias: torch.Tensor | None = None) -> bool:
     """The prefill matrix product on tcgen05 tensor cores (bfloat16 operands, rows 16-byte aligned).
     ``tile_width``: 256, 128 or 64 output columns per tile; 0 lets the shape decide (narrower tiles when the
     widest would leave SMs without one).  ``k_spans``: 2 or 4 cuts K among the CTAs of a cluster, which add their
@@ -454,8 +486,8 @@ def gemm_tcgen05(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, epilogue: in
     ldc, c_inner = c.stride()
     assert Kw == K and c_inner == 1 and c.shape == (M, N // 2 if epilogue in GATED_EPILOGUES else N)
     _check(_fn("b200_gemm_tcgen05")(pa, lda, pw, ldw, c.data_ptr(), dtype_code(c.dtype), ldc, M, N, K, epilogue,
-                                    tile_width, k_spans, cta_pair, float(gate_args[0]), float(gate_args[1]), _stream()),
-           "gemm_tcgen05")
+                                    tile_width, k_spans, cta_pair, float(gate_args[0]), float(gate_args[1]),
+                                    _bias_ptr(bias, N), _stream()), "gemm_tcgen05")
     return True
 
 
@@ -667,13 +699,13 @@ def attention_decode_rope(qkv: torch.Tensor, out: torch.Tensor, kv_lens: torch.T
 def attention_decode(q: torch.Tensor, q_row_stride: int, out: torch.Tensor, kv_lens: torch.Tensor,
                      page_table: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, n_heads: int,
                      n_kv_heads: int, head_dim: int, window: int, n_splits: int,
-                     scratch: torch.Tensor | None = None, early_start: bool = True, *, keep_first: int = 0,
+                     scratch: torch.Tensor | None = None, early_start: bool = True, *, keep_first: int = 0, chunk: int = 0,
                      slopes: torch.Tensor | None = None, sinks: torch.Tensor | None = None,
                      gate: torch.Tensor | None = None) -> None:
     """One query token per sequence (row i of q belongs to sequence i) over kv_lens[i] cached keys.
     ``scratch``: float32 workspace for the spans' partial results (allocated here when absent).
-    ``early_start``: see ``attention_decode_early_start``.  ``keep_first``, ``slopes``, ``sinks``, ``gate``: as for
-    ``attention_paged``."""
+    ``early_start``: see ``attention_decode_early_start``.  ``keep_first``, ``chunk``, ``slopes``, ``sinks``, ``gate``:
+    as for ``attention_paged``."""
     _dev(q, out, kv_lens, page_table, k_pool, v_pool)
     n_seqs = out.shape[0]
     assert q.dtype == out.dtype == k_pool.dtype == torch.bfloat16 and out.is_contiguous()
@@ -682,7 +714,7 @@ def attention_decode(q: torch.Tensor, q_row_stride: int, out: torch.Tensor, kv_l
     need = n_seqs * n_heads * n_splits * (head_dim + 2) if n_splits > 1 else 0
     if need and (scratch is None or scratch.numel() < need):
         scratch = torch.empty(need, dtype=torch.float32, device=q.device)
-    if keep_first or slopes is not None or sinks is not None or gate is not None:
+    if keep_first or chunk or slopes is not None or sinks is not None or gate is not None:
         _dev(slopes, sinks, gate)
         for t in (slopes, sinks):
             assert t is None or (t.dtype == torch.float32 and t.is_contiguous() and t.numel() == n_heads)
@@ -691,7 +723,7 @@ def attention_decode(q: torch.Tensor, q_row_stride: int, out: torch.Tensor, kv_l
         _check(_fn("b200_attention_decode_terms")(
             q.data_ptr(), q_row_stride, out.data_ptr(), kv_lens.data_ptr(), page_table.data_ptr(), page_table.shape[1],
             k_pool.data_ptr(), v_pool.data_ptr(), scratch.data_ptr() if need else None, scratch.numel() if need else 0,
-            n_seqs, n_heads, n_kv_heads, head_dim, int(window), n_splits, 1 if early_start else 0, int(keep_first),
+            n_seqs, n_heads, n_kv_heads, head_dim, int(window), n_splits, 1 if early_start else 0, int(keep_first), int(chunk),
             ptr(slopes), ptr(sinks), ptr(gate), gate.stride(0) if gate is not None else 0, _stream()),
             "attention_decode_terms" if early_start else "attention_decode_terms:late")
         return
@@ -705,11 +737,11 @@ def attention_decode(q: torch.Tensor, q_row_stride: int, out: torch.Tensor, kv_l
 def attention_prefill(q: torch.Tensor, q_row_stride: int, out: torch.Tensor, cu_seqlens: torch.Tensor,
                       kv_lens: torch.Tensor, page_table: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor,
                       n_seqs: int, max_q_len: int, n_heads: int, n_kv_heads: int, head_dim: int, window: int, *,
-                      keep_first: int = 0, slopes: torch.Tensor | None = None, sinks: torch.Tensor | None = None,
+                      keep_first: int = 0, chunk: int = 0, slopes: torch.Tensor | None = None, sinks: torch.Tensor | None = None,
                       gate: torch.Tensor | None = None) -> None:
     """Causal attention of packed query tokens: sequence i owns rows cu_seqlens[i]..cu_seqlens[i+1],
     which are its last positions (kv_lens[i] - q_len .. kv_lens[i] - 1); keys come from the cache.
-    ``keep_first``, ``slopes``, ``sinks``, ``gate``: as for ``attention_paged``."""
+    ``keep_first``, ``chunk``, ``slopes``, ``sinks``, ``gate``: as for ``attention_paged``."""
     _dev(q, out, cu_seqlens, kv_lens, page_table, k_pool, v_pool, slopes, sinks, gate)
     for t in (slopes, sinks):
         assert t is None or (t.dtype == torch.float32 and t.is_contiguous() and t.numel() == n_heads)
@@ -721,25 +753,29 @@ def attention_prefill(q: torch.Tensor, q_row_stride: int, out: torch.Tensor, cu_
     _check(_fn("b200_attention_prefill")(
         q.data_ptr(), q_row_stride, out.data_ptr(), cu_seqlens.data_ptr(), kv_lens.data_ptr(), page_table.data_ptr(),
         page_table.shape[1], k_pool.data_ptr(), v_pool.data_ptr(), n_seqs, max_q_len, n_heads, n_kv_heads, head_dim,
-        int(window), int(keep_first), ptr(slopes), ptr(sinks), ptr(gate), gate.stride(0) if gate is not None else 0,
-        _stream()), "attention_prefill")
+        int(window), int(keep_first), int(chunk), ptr(slopes), ptr(sinks), ptr(gate),
+        gate.stride(0) if gate is not None else 0, _stream()), "attention_prefill")
 
 
 def attention_prefill_tc(q: torch.Tensor, q_row_stride: int, out: torch.Tensor, cu_seqlens: torch.Tensor,
                          kv_lens: torch.Tensor, page_table: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor,
-                         n_seqs: int, max_q_len: int, n_heads: int, n_kv_heads: int, head_dim: int, window: int) -> bool:
-    """``attention_prefill`` on tcgen05 tensor cores (head_dim 64 or 128).  Returns False, having done
+                         n_seqs: int, max_q_len: int, n_heads: int, n_kv_heads: int, head_dim: int, window: int, *,
+                         chunk: int = 0, sinks: torch.Tensor | None = None) -> bool:
+    """``attention_prefill`` on tcgen05 tensor cores (head_dim 64 or 128), with ``chunk`` and ``sinks`` but none of the other
+    terms.  Returns False, having done
     nothing, for sizes it does not take."""
     if head_dim not in (64, 128) or q.dtype != torch.bfloat16 or q_row_stride % 8 or (q.data_ptr() | out.data_ptr()) & 15:
         return False
-    _dev(q, out, cu_seqlens, kv_lens, page_table, k_pool, v_pool)
+    _dev(q, out, cu_seqlens, kv_lens, page_table, k_pool, v_pool, sinks)
+    assert sinks is None or (sinks.dtype == torch.float32 and sinks.is_contiguous() and sinks.numel() == n_heads)
     assert out.dtype == k_pool.dtype == torch.bfloat16 and out.is_contiguous() and k_pool.is_contiguous()
     assert tuple(k_pool.shape[1:]) == (n_kv_heads, PAGE_TOKENS, head_dim)
     assert tuple(v_pool.shape[1:]) == (n_kv_heads, head_dim, PAGE_TOKENS)
     _check(_fn("b200_attention_prefill_tc")(
         q.data_ptr(), q_row_stride, out.shape[0], out.data_ptr(), cu_seqlens.data_ptr(), kv_lens.data_ptr(),
         page_table.data_ptr(), page_table.shape[1], k_pool.data_ptr(), v_pool.data_ptr(), k_pool.shape[0], n_seqs,
-        max_q_len, n_heads, n_kv_heads, head_dim, int(window), _stream()), "attention_prefill_tc")
+        max_q_len, n_heads, n_kv_heads, head_dim, int(window), int(chunk), sinks.data_ptr() if sinks is not None else None,
+        _stream()), "attention_prefill_tc")
     return True
 
 
@@ -850,7 +886,8 @@ ROW_WORDS = 20   # 32-bit words of one segment record (head_rows.cu: kSegmentWor
 def head_row_segment(src_off: int, n_rows: int, d: int, dst_off: int, d_pad: int | None = None, bias_off: int = -1,
                      norm: bool | int = False, weight_off: int = -1, mul: float = 1.0, target: int = TO_ROWS,
                      weight_per_row: bool = False, mix_off: int = -1, rotate: bool = False, src_stride: int = -1,
-                     dst_stride: int = -1, cache_dim: int = -1, lead: int = 0) -> list[int]:
+                     dst_stride: int = -1, cache_dim: int = -1, lead: int = 0, half_pairs: int | None = None,
+                     freq_off: int = 0) -> list[int]:
     """One segment of ``head_rows``: ``n_rows`` rows of ``d`` numbers from column ``src_off`` on, each (+ bias)
     (normalised) (* weight) * mul, written ``d_pad`` wide (zeros behind the ``d``) from column ``dst_off`` on, or with
     ``target`` TO_CACHE_KEYS / TO_CACHE_VALUES into the cache page of the token's position (``n_rows`` = the cache
@@ -861,12 +898,14 @@ def head_row_segment(src_off: int, n_rows: int, d: int, dst_off: int, d_pad: int
     ``src_stride`` / ``dst_stride``: numbers between two rows read / written when they do not lie back to back (a source
     stride of 0: all rows read the same numbers).  ``cache_dim``: the row size of the cache, when the segment fills only
     the ``d_pad`` columns from ``dst_off`` on of every cache row.  ``lead``: how many of the ``d_pad`` numbers written are
-    zeros in front of the row's ``d`` (the rest of the zeros follow it)."""
+    zeros in front of the row's ``d`` (the rest of the zeros follow it).  ``half_pairs`` n (in place of ``rotate``): the
+    row's pairs (i, i + n), i < n, are turned by the token's position times the frequencies from ``freq_off`` on; the columns
+    from 2 n on pass."""
     import struct
 
     return [src_off, n_rows, d, dst_off, d if d_pad is None else d_pad, bias_off, int(norm), weight_off,
             struct.unpack("<i", struct.pack("<f", float(mul)))[0], target, 1 if weight_per_row else 0, mix_off,
-            1 if rotate else 0, src_stride, dst_stride, cache_dim, int(lead), 0, 0, 0]
+            2 if half_pairs else 1 if rotate else 0, src_stride, dst_stride, cache_dim, int(lead), int(half_pairs or 0), int(freq_off), 0]
 
 
 def head_rows(src: torch.Tensor, dst: torch.Tensor | None, segments, eps: float = 0.0, bias: torch.Tensor | None = None,
@@ -924,20 +963,34 @@ def softcap_rows(logits: torch.Tensor, cap: float) -> None:
 GATE_ACTIVATIONS = {"sigmoid": 0, "silu": 1}
 
 
-def gated_rmsnorm(x: torch.Tensor, weight: torch.Tensor, gate: torch.Tensor, out: torch.Tensor, n_heads: int, d: int,
-                  eps: float, activation: str = "sigmoid", gate_first: bool = False) -> None:
+def gated_rmsnorm(x: torch.Tensor, weight: torch.Tensor | None, gate: torch.Tensor, out: torch.Tensor, n_heads: int, d: int,
+                  eps: float, activation: str = "sigmoid", gate_first: bool = False, mul: float = 1.0) -> None:
     """Per (token, head) row of float32 x [T, n_heads d]: x / sqrt(mean(x^2) + eps) * weight[d] * act(gate), act the
     sigmoid or SiLU.  ``gate_first``: the row is multiplied by act(gate) first and the norm runs over the gated row.
-    A weight of n_heads * d numbers gives every row weights of its own (the rows are then any equal parts of x's rows)."""
+    A weight of n_heads * d numbers gives every row weights of its own (the rows are then any equal parts of x's rows); None:
+    no weight.  ``mul``: a last factor, in 32 bits.  ``out`` may be columns of a wider buffer."""
     _dev(x, weight, gate, out)
-    assert x.dtype == weight.dtype == torch.float32 and x.is_contiguous() and out.is_contiguous() and gate.stride(1) == 1
-    assert x.shape[1] == n_heads * d == out.shape[1] and gate.shape[1] >= n_heads * d and weight.numel() in (d, n_heads * d)
-    assert gate.dtype == out.dtype and weight.is_contiguous()
-    per_row = weight.numel() != d
-    _check(_fn("b200_gated_rmsnorm")(x.data_ptr(), weight.data_ptr(), gate.data_ptr(), gate.stride(0), out.data_ptr(),
+    assert x.dtype == torch.float32 and x.is_contiguous() and out.stride(1) == 1 and gate.stride(1) == 1
+    assert x.shape[1] == n_heads * d == out.shape[1] and gate.shape[1] >= n_heads * d and gate.dtype == out.dtype
+    assert weight is None or (weight.dtype == torch.float32 and weight.is_contiguous() and weight.numel() in (d, n_heads * d))
+    per_row = weight is not None and weight.numel() != d
+    _check(_fn("b200_gated_rmsnorm")(x.data_ptr(), weight.data_ptr() if weight is not None else None, gate.data_ptr(), gate.stride(0), out.data_ptr(),
                                      dtype_code(out.dtype), x.shape[0], n_heads, d, float(eps),
-                                     GATE_ACTIVATIONS[activation], 1 if gate_first else 0, 1 if per_row else 0, _stream()),
-           "gated_rmsnorm")
+                                     GATE_ACTIVATIONS[activation], 1 if gate_first else 0, 1 if per_row else 0, out.stride(0),
+                                     float(mul), _stream()), "gated_rmsnorm")
+
+
+def turn_back_rows(x: torch.Tensor, positions: torch.Tensor, inv_freq: torch.Tensor | None, out: torch.Tensor, n_heads: int,
+                   d: int, d_pad: int, mul: float = 1.0) -> None:
+    """out[t, h] = mul * (the first ``d`` numbers of head h of x [T, n_heads d_pad], their pairs (i, i + d / 2) turned by
+    -positions[t] * inv_freq[i]); ``inv_freq`` None: nothing is turned.  ``out`` [T, n_heads d] may be columns of a wider buffer."""
+    _dev(x, positions, inv_freq, out)
+    assert x.is_contiguous() and out.stride(1) == 1 and x.dtype == out.dtype and x.shape[0] == out.shape[0] == positions.numel()
+    assert x.shape[1] == n_heads * d_pad and out.shape[1] == n_heads * d and positions.dtype == torch.int32
+    assert inv_freq is None or (inv_freq.dtype == torch.float32 and inv_freq.is_contiguous() and inv_freq.numel() >= d // 2)
+    _check(_fn("b200_turn_back_rows")(x.data_ptr(), positions.data_ptr(), inv_freq.data_ptr() if inv_freq is not None else None,
+                                      out.data_ptr(), out.stride(0), dtype_code(x.dtype), x.shape[0], n_heads, int(d), int(d_pad),
+                                      float(mul), _stream()), "turn_back_rows")
 
 
 def gate_rows(x: torch.Tensor, gate: torch.Tensor, activation: str = "sigmoid") -> None:
@@ -1175,25 +1228,36 @@ def causal_conv(x: torch.Tensor, weight: torch.Tensor, state: torch.Tensor, slot
            "causal_conv")
 
 
-DECAY_SOFTPLUS_RATE, DECAY_SIGMOID_POWER = 0, 1
+DECAY_SOFTPLUS_RATE, DECAY_SIGMOID_POWER, DECAY_FIXED = 0, 1, 2
 
 
-def linear_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, state: torch.Tensor,
+def linear_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor | None, state: torch.Tensor,
                 slots: torch.Tensor, cu_seqlens: torch.Tensor, out: torch.Tensor, heads: int, kv_heads: int, d_k: int,
                 d_v: int, *, decay_kind: int, decay_per_head: bool = False, decay_bias: torch.Tensor | None = None,
                 a_log: torch.Tensor | None = None, power: float = 1.0, q_scale: float = 1.0,
-                step_scales_value: bool = False, skip: torch.Tensor | None = None, alloc=None) -> None:
+                step_scales_value: bool = False, skip: torch.Tensor | None = None, qk_silu: bool = False,
+                v_silu: bool = False, rotary=None, alloc=None) -> None:
     """The recurrence S <- diag(g) S + k (beta v)^T, o = S^T q + skip v per head over a packed step (no delta correction).
     q, k [T, >= kv_heads d_k] (head h reads head h // (heads // kv_heads)), v [T, >= heads d_v], decay [T, >= heads d_k]
     (or [T, >= heads] with ``decay_per_head``) before its bias and activation, all of one type; g =
     exp(-exp(a_log[h]) softplus(decay + bias)) (``DECAY_SOFTPLUS_RATE``) or sigmoid(decay + bias)^power
     (``DECAY_SIGMOID_POWER``); beta = 1, or the step size softplus(decay + bias) with ``step_scales_value``.  state float32
-    [slots, >= heads d_k d_v], updated in place; out float32 [T, heads d_v]; everything but the operands' storage is 32-bit."""
+    [slots, >= heads d_k d_v], updated in place; out float32 [T, heads d_v]; everything but the operands' storage is 32-bit.
+    ``DECAY_FIXED``: g = a_log[h] as it stands and ``decay`` is None.  ``qk_silu`` / ``v_silu``: q and k / v pass through SiLU;
+    ``rotary`` = (positions int32 [T], inverse frequencies float32 [n]): the pairs (i, i + n), i < n, of q and k are turned."""
     _dev(q, k, v, decay, state, slots, cu_seqlens, out, decay_bias, a_log, skip)
-    assert q.dtype == k.dtype == v.dtype == decay.dtype and q.stride(1) == k.stride(1) == v.stride(1) == decay.stride(1) == 1
+    fixed = decay_kind == DECAY_FIXED
+    assert (decay is None) == fixed and (not fixed or (decay_per_head and a_log is not None))
+    assert q.dtype == k.dtype == v.dtype and q.stride(1) == k.stride(1) == v.stride(1) == 1
+    assert fixed or (decay.dtype == q.dtype and decay.stride(1) == 1)
     assert state.dtype == out.dtype == torch.float32 and out.is_contiguous() and state.stride(1) == 1
     n_decay = heads if decay_per_head else heads * d_k
-    assert q.shape[1] >= kv_heads * d_k and k.shape[1] >= kv_heads * d_k and v.shape[1] >= heads * d_v and decay.shape[1] >= n_decay
+    assert q.shape[1] >= kv_heads * d_k and k.shape[1] >= kv_heads * d_k and v.shape[1] >= heads * d_v
+    assert fixed or decay.shape[1] >= n_decay
+    rot_pos, inv_freq = rotary if rotary is not None else (None, None)
+    if rotary is not None:
+        _dev(rot_pos, inv_freq)
+        assert rot_pos.dtype == torch.int32 and rot_pos.numel() == q.shape[0] and inv_freq.dtype == torch.float32 and 2 * inv_freq.numel() <= d_k
     for t, n in ((decay_bias, n_decay), (a_log, heads), (skip, heads)):
         assert t is None or (t.dtype == torch.float32 and t.is_contiguous() and t.numel() == n)
     assert decay_kind != DECAY_SOFTPLUS_RATE or a_log is not None
@@ -1204,11 +1268,12 @@ def linear_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.
     scratch = alloc(shape, torch.float32) if alloc is not None else torch.empty(shape, dtype=torch.float32, device=q.device)
     ptr = lambda t: t.data_ptr() if t is not None else None
     _check(_fn("b200_linear_scan")(q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0),
-                                   decay.data_ptr(), decay.stride(0), ptr(decay_bias), ptr(a_log), ptr(skip), state.data_ptr(),
+                                   ptr(decay), 0 if fixed else decay.stride(0), ptr(decay_bias), ptr(a_log), ptr(skip), state.data_ptr(),
                                    state.stride(0), slots.data_ptr(), cu_seqlens.data_ptr(), out.data_ptr(), scratch.data_ptr(),
                                    dtype_code(q.dtype), q.shape[0], slots.numel(), heads, kv_heads, d_k, d_v, float(q_scale),
                                    float(power), int(decay_kind), 1 if decay_per_head else 0, 1 if step_scales_value else 0,
-                                   _stream()), "linear_scan")
+                                   1 if qk_silu else 0, 1 if v_silu else 0, inv_freq.numel() if inv_freq is not None else 0,
+                                   ptr(inv_freq), ptr(rot_pos), _stream()), "linear_scan")
 
 
 def delta_rule_supported(d_k: int) -> bool:

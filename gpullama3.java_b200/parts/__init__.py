@@ -20,6 +20,9 @@ from .position import YarnRotaryPositionEncoding
 from .feed_forward import DenseFeedForward
 from .differential_attention import DifferentialAttention
 from .gated_residual import GatedResidualBlock
+from .linear_recurrence import FixedDecayAttention
+from .chunked_attention import ChunkedAttention
+from .parallel import ParallelBlock, ParallelMixers
 
 __all__ = ["Block", "FeedForward", "Mixer", "Norm", "Part", "PartRegistryError", "PositionEncoding", "ScaledRows",
            "StepContext", "all_parts", "build_block", "build_part", "register_block", "register_feed_forward",
@@ -28,4 +31,5 @@ __all__ = ["Block", "FeedForward", "Mixer", "Norm", "Part", "PartRegistryError",
            "PreNormBlock", "OutputHead", "TokenEmbedding", "ConnectedBlock", "StreamConnection", "LatentAttention",
            "ChannelDeltaRule", "HeadDeltaRule", "LayerNorm", "RoutedFeedForward", "GatedLinearAttention",
            "StateSpaceDuality", "SandwichBlock", "YarnRotaryPositionEncoding", "DenseFeedForward",
-           "DifferentialAttention", "GatedResidualBlock"]
+           "DifferentialAttention", "GatedResidualBlock", "FixedDecayAttention", "ChunkedAttention", "ParallelBlock",
+           "ParallelMixers"]

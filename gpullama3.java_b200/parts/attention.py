@@ -232,13 +232,20 @@ def plan_decode_attention(shape, ctx: StepContext, cache: KVView) -> tuple[int, 
     whether the kernel may be scheduled while its predecessor still runs.  Both follow from the number of
     sequences, the mixer's own kv heads and the longest sequence the step must be right for (its cache
     group's ``kv_capacity``: a recorded step is replayed until its page tables are outgrown).  ``shape``: whatever
-    has ``n_heads``, ``n_kv_heads``, ``head_dim``, ``window`` and ``keep_first`` as the attention kernels are to see them."""
+    has ``n_heads``, ``n_kv_heads``, ``head_dim``, ``window`` and ``keep_first`` (and ``chunk``) as the attention kernels are to see
+    them."""
     capacity = ctx.capacity(cache.group)
-    if shape.window:
-        capacity = min(capacity, shape.window + shape.keep_first)
+    capacity = min(capacity, _reach(shape) or capacity)
     resident = ops.resident_ctas(ctx.device, shape.head_dim, shape.n_heads // shape.n_kv_heads)
     splits = ops.attention_decode_splits(ctx.n_seqs, shape.n_kv_heads, capacity, resident)
     return splits, ops.attention_decode_early_start(ctx.n_seqs, shape.n_kv_heads, capacity, splits)
+
+
+def _reach(shape) -> int | None:
+    """The most keys one query sees; None: all of them."""
+    if shape.window:
+        return shape.window + shape.keep_first
+    return getattr(shape, "chunk", None)
 
 
 def attend(shape, qkv: torch.Tensor, out: torch.Tensor, ctx: StepContext, table: torch.Tensor, cache: KVView, gate=None) -> None:
@@ -249,11 +256,11 @@ def attend(shape, qkv: torch.Tensor, out: torch.Tensor, ctx: StepContext, table:
     if fast.try_attention(qkv, out, ctx, table, cache, shape, gate):
         return
     rows = qkv.shape[0] * shape.n_heads
-    reach = ctx.capacity(cache.group) if not shape.window else min(ctx.capacity(cache.group), shape.window + shape.keep_first)
+    reach = min(ctx.capacity(cache.group), _reach(shape) or ctx.capacity(cache.group))
     splits = 1 if rows >= 1024 else max(1, min(16, 1024 // rows, reach // 512))
     ops.attention_paged(qkv, qkv.shape[1], out, ctx.positions, ctx.seq_ids, table, cache.k, cache.v,
                         shape.n_heads, shape.n_kv_heads, shape.head_dim, shape.window or 0, n_splits=splits,
-                        keep_first=shape.keep_first, slopes=getattr(shape, "slopes", None), sinks=getattr(shape, "sinks", None),
+                        keep_first=shape.keep_first, chunk=getattr(shape, "chunk", None) or 0, slopes=getattr(shape, "slopes", None), sinks=getattr(shape, "sinks", None),
                         gate=gate)
 
 

@@ -105,10 +105,44 @@ class Part:
         """Take the parameters (CPU or device tensors by local name), move and re-lay them out for
         the kernels.  ``dtype`` is the run's precision."""
 
+    def after_load(self) -> None:
+        """Called once when every part of the model has been loaded, on the parts this one was built with before it: where
+        a part joins its matrices with theirs."""
+
     def children(self) -> dict[str, "Part"]:
         """Parts this part was built with, by the names it gives them.  Their parameters are declared and
         loaded under ``<this part's path>.<name>``; the part itself only declares its own."""
         return {}
+
+
+class OpenEnded:
+    """A mixer or feed-forward whose result is one last product over rows it makes: result = W rows (+ b).  Whoever
+    arranges such parts side by side may take their last products over (``take_output``), let each write its rows into
+    neighbouring columns of one buffer (``rows_into``) and multiply once; where a part is used alone, its own ``forward`` does
+    both.  Mixers that also start with one product over their input can give that away too (``take_input``) and be handed
+    its result (``rows_from``)."""
+
+    def open_columns(self) -> int:
+        """Numbers per token of the rows before the last product."""
+        raise NotImplementedError
+
+    def take_output(self) -> tuple[torch.Tensor, torch.Tensor | None]:
+        """The last product's weight [hidden, open_columns] and bias (or None); the part keeps neither."""
+        raise NotImplementedError
+
+    def rows_into(self, x, ctx: "StepContext", cache, rows: torch.Tensor, writes_cache: bool = True, mul: float = 1.0) -> None:
+        """The rows of input x (a tensor, or ScaledRows where ``takes_scaled_rows``) into ``rows`` [T, open_columns], columns of
+        a wider buffer; ``mul``: a factor on them, applied in 32 bits before they are rounded."""
+        raise NotImplementedError
+
+    def take_input(self) -> torch.Tensor:
+        """The first product's weight [columns, hidden], columns a multiple of 8; the part keeps none."""
+        raise NotImplementedError
+
+    def rows_from(self, raw: torch.Tensor, ctx: "StepContext", cache, rows: torch.Tensor, writes_cache: bool = True,
+                  mul: float = 1.0) -> None:
+        """``rows_into`` behind the first product: ``raw`` [T, columns] is its result, columns of a wider buffer."""
+        raise NotImplementedError
 
 
 class Norm(Part):

@@ -12,18 +12,22 @@ from .base import ScaledRows
 
 
 class Linear:
-    def __init__(self, weight: torch.Tensor):
+    def __init__(self, weight: torch.Tensor, bias: torch.Tensor | None = None):
+        """``bias``: one number per row of the weight, kept in 32 bits; it joins the sums before whatever the product's
+        epilogue does with them."""
         assert weight.dim() == 2 and weight.is_contiguous()
         self.weight = weight
+        self.bias = bias.to(device=weight.device, dtype=torch.float32).contiguous() if bias is not None else None
         self.out_features, self.in_features = weight.shape
 
     def _run(self, a, c: torch.Tensor, epilogue: int, gate_args=(0.0, 0.0)) -> None:
         if isinstance(a, ScaledRows):  # only handed to a product that said it links (links_with)
-            ops.gemm_decode_linked(a.data, self.weight, c, epilogue, row_factors=(a.partials, a.eps, a.dim))
+            ops.gemm_decode_linked(a.data, self.weight, c, epilogue, row_factors=(a.partials, a.eps, a.dim),
+                                   bias=self.bias)
             return
-        if fast.try_gemm(a, self.weight, c, epilogue, gate_args):
+        if fast.try_gemm(a, self.weight, c, epilogue, gate_args, self.bias):
             return
-        ops.gemm_generic(a, self.weight, c, epilogue, gate_args)
+        ops.gemm_generic(a, self.weight, c, epilogue, gate_args, self.bias)
 
     def links_with(self, n_rows: int, dtype: torch.dtype) -> bool:
         """Whether this product can be one half of a split norm for ``n_rows`` rows of ``dtype``."""
@@ -42,16 +46,21 @@ class Linear:
 
     def add_to(self, a: torch.Tensor, residual: torch.Tensor, then_norm=None) -> ScaledRows | None:
         """residual += a @ W.T, the sum kept in float32.  With ``then_norm`` (a norm that has a row-factor form)
-        and a product that links, the same kernel also leaves that norm of the new residual as ScaledRows."""
+        and a product that links, the same kernel also leaves that norm of the new residual as ScaledRows; a ``then_norm``
+        that stands for two norms of the same rows (``second_form``) gets the rows under both weights."""
         form = then_norm.row_factor_form() if then_norm is not None else None
+        second = getattr(then_norm, "second_form", None)
         if (form is not None and a.dtype == torch.bfloat16 and self.links_with(a.shape[0], a.dtype)
                 and form[2] == self.out_features and a.stride(1) == 1 and a.stride(0) % 8 == 0 and a.data_ptr() % 16 == 0):
             weight, eps, dim = form
             n = a.shape[0]
             act = torch.empty((n, dim), dtype=torch.bfloat16, device=a.device)
             partials = torch.empty((n, ops.gemm_decode_partials(n, self.out_features)), dtype=torch.float32, device=a.device)
-            ops.gemm_decode_linked(a, self.weight, residual, ops.EPILOGUE_RESIDUAL_ADD, emit=(weight, act, partials))
-            return ScaledRows(act, partials, eps, dim)
+            act2 = torch.empty_like(act) if second is not None else None
+            ops.gemm_decode_linked(a, self.weight, residual, ops.EPILOGUE_RESIDUAL_ADD, emit=(weight, act, partials),
+                                   emit_second=(second(), act2) if second is not None else None, bias=self.bias)
+            rows = ScaledRows(act, partials, eps, dim)
+            return (rows, ScaledRows(act2, partials, eps, dim)) if second is not None else rows
         self._run(a, residual, ops.EPILOGUE_RESIDUAL_ADD)
         return None
 

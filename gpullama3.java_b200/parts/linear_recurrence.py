@@ -1,5 +1,5 @@
 """Recurrent mixers whose memory is one matrix per head that decays and gains an outer product per token, without the
-delta rule's correction:  S_t = diag(g_t) S_(t-1) + k_t (b_t v_t)^T,  o_t = S_t^T q_t.  Two of them:
+delta rule's correction:  S_t = diag(g_t) S_(t-1) + k_t (b_t v_t)^T,  o_t = S_t^T q_t.  Three of them:
 
 ``GatedLinearAttention`` (``gla``): a decay per key channel from a low-rank projection,
 
@@ -14,7 +14,13 @@ delta rule's correction:  S_t = diag(g_t) S_(t-1) + k_t (b_t v_t)^T,  o_t = S_t^
     k = B, q = C  [groups, state] (head h reads group h / (heads / groups)) ;  v = x  [heads, d_v]
     o_t += D_h x_t ;  y = W_o ( norm( o * silu(z) ) )       the gate first, then an RMS norm in ``norm_groups`` equal parts
 
-Both keep, per sequence, S of every head in 32 bits (and the convolution's last inputs) in one row of their cache slot,
+``FixedDecayAttention`` (``fixed_decay``): a decay per head that the configuration gives, b = 1 (retention, lightning attention),
+
+    q, k = act(W_q x), act(W_k x)  [heads, d_k] ;  v = act(W_v x)  [heads, d_v] ;  act: SiLU or none
+    q and k turned by the token's position (halves; optional) ;  q times ``scale`` (it stands for a factor on the keys as well)
+    y = W_o ( norm(o) * gate(W_g x) )      norm over each head's numbers or over all heads together, with a weight or none
+
+All keep, per sequence, S of every head in 32 bits (and the convolution's last inputs) in one row of their cache slot,
 starting from zero.  Decays, step sizes, the recurrence and the output norms are 32-bit in both precisions; projections
 and the convolution are computed in the run's precision.  The scan is the kernel of the delta rule, told to leave out
 the correction."""
@@ -26,8 +32,9 @@ from ..cache.sequence_cache import StateNeed, StateView
 from ..config.base import ConfigError
 from ..kernels import ops
 from ..weights.loader import ParamSpec
-from .base import Mixer, StepContext, register_mixer
+from .base import Mixer, OpenEnded, PositionEncoding, StepContext, register_mixer
 from .linear import Linear
+from .position import PAIRING_CODES
 
 
 def _pad8(n: int) -> int:
@@ -162,5 +169,91 @@ class StateSpaceDuality(Mixer):
         return self.o.add_to(gated, residual, then_norm)
 
 
+class FixedDecayAttention(Mixer, OpenEnded):
+    graph_safe = True
+    pad_safe = False
+
+    def __init__(self, hidden_size: int, n_heads: int, head_dim: int, value_dim: int, decay, norm_eps: float, *,
+                 activation: str | None = None, position: PositionEncoding | None = None, scale: float = 1.0,
+                 norm_over: str = "head", norm_weight: bool = False, gate: str = "silu"):
+        """``decay``: one number per head.  ``norm_over``: ``head`` (every head by its own root mean square) or ``all`` (all heads
+        together).  ``norm_weight``: the norm has a weight per number.  ``gate``: the activation of the output gate."""
+        if min(n_heads, head_dim, value_dim) < 1 or head_dim > 512:
+            raise ConfigError(f"fixed-decay attention: key size {head_dim} must be between 1 and 512, heads and value size positive")
+        if len(decay) != n_heads or not all(0.0 <= float(g) <= 1.0 for g in decay):
+            raise ConfigError(f"fixed-decay attention: {n_heads} heads need as many decays between 0 and 1, got {list(decay)}")
+        if activation not in (None, "silu") or norm_over not in ("head", "all") or gate not in ops.GATE_ACTIVATIONS:
+            raise ConfigError(f"fixed-decay attention: activation {activation!r}, norm over {norm_over!r}, gate {gate!r}")
+        if position is not None and position.rotary_dim:
+            if position.rotary_dim > head_dim or position.pairing != PAIRING_CODES["half"]:
+                raise ConfigError(f"fixed-decay attention turns pairs over halves of at most {head_dim} numbers")
+        self.hidden_size, self.n_heads, self.key_dim, self.value_dim = int(hidden_size), int(n_heads), int(head_dim), int(value_dim)
+        self.decay, self.norm_eps, self.scale = [float(g) for g in decay], float(norm_eps), float(scale)
+        self.silu, self.position, self.norm_over = activation == "silu", position, norm_over
+        self.norm_weight, self.gate = bool(norm_weight), gate
+        self.state_floats = self.n_heads * self.key_dim * self.value_dim
+        self.inputs: Linear | None = None
+        self.o: Linear | None = None
+
+    def parameters(self):
+        H, dk, dv, h = self.n_heads, self.key_dim, self.value_dim, self.hidden_size
+        p = {"q": ParamSpec((H * dk, h)), "k": ParamSpec((H * dk, h)), "v": ParamSpec((H * dv, h)), "g": ParamSpec((H * dv, h)),
+             "o": ParamSpec((h, H * dv))}
+        if self.norm_weight:
+            p["norm"] = ParamSpec((H * dv if self.norm_over == "all" else dv,), "norm")
+        return p
+
+    def children(self):
+        return {"position": self.position} if self.position is not None else {}
+
+    def cache_need(self):
+        return StateNeed((self.state_floats,), torch.float32)
+
+    def load(self, tensors, dtype, device):
+        run = lambda t: t.to(device).to(torch.float32 if dtype == torch.float32 else t.dtype)
+        self.inputs, (self.q_off, self.k_off, self.v_off, self.g_off) = _stacked([run(tensors[n]) for n in ("q", "k", "v", "g")], device)
+        self.o = Linear(run(tensors["o"]).contiguous())
+        self.weight = tensors["norm"].to(device=device, dtype=torch.float32).contiguous() if self.norm_weight else None
+        self.decays = torch.tensor(self.decay, dtype=torch.float64).to(torch.float32).to(device)
+        self.inv_freq = None
+        if self.position is not None and self.position.rotary_dim:
+            self.inv_freq = self.position.inverse_frequencies(device)[:self.position.rotary_dim // 2].contiguous()
+        if device.type == "cuda" and not ops.delta_rule_supported(self.key_dim):
+            raise ConfigError(f"fixed-decay attention: no kernel holds a state column of {self.key_dim} rows")
+
+    def open_columns(self):
+        return self.n_heads * self.value_dim
+
+    def take_output(self):
+        weight, self.o = self.o.weight, None
+        return weight, None
+
+    def take_input(self):
+        weight, self.inputs = self.inputs.weight, None
+        return weight
+
+    def takes_scaled_rows(self, ctx: StepContext) -> bool:
+        return ctx.all_decode and self.inputs is not None and self.inputs.links_with(ctx.n_tokens, ctx.dtype)
+
+    def rows_into(self, x, ctx: StepContext, cache: StateView, rows, writes_cache=True, mul=1.0):
+        self.rows_from(self.inputs.store(x, ctx.dtype, ctx.empty), ctx, cache, rows, writes_cache, mul)
+
+    def rows_from(self, raw, ctx: StepContext, cache: StateView, rows, writes_cache=True, mul=1.0):
+        H, dk, dv, T = self.n_heads, self.key_dim, self.value_dim, raw.shape[0]
+        o = ctx.empty((T, H * dv), torch.float32)
+        ops.linear_scan(raw[:, self.q_off:], raw[:, self.k_off:], raw[:, self.v_off:], None, cache.data, ctx.slots_dev,
+                        ctx.cu_seqlens, o, H, H, dk, dv, decay_kind=ops.DECAY_FIXED, decay_per_head=True, a_log=self.decays,
+                        q_scale=self.scale, qk_silu=self.silu, v_silu=self.silu,
+                        rotary=(ctx.positions, self.inv_freq) if self.inv_freq is not None else None, alloc=ctx.empty)
+        parts, d = (H, dv) if self.norm_over == "head" else (1, H * dv)
+        ops.gated_rmsnorm(o, self.weight, raw[:, self.g_off:], rows, parts, d, self.norm_eps, self.gate, mul=mul)
+
+    def forward(self, x, ctx: StepContext, cache: StateView, residual, writes_cache=True, then_norm=None):
+        rows = ctx.empty((x.shape[0], self.open_columns()), ctx.dtype)
+        self.rows_into(x, ctx, cache, rows, writes_cache)
+        return self.o.add_to(rows, residual, then_norm)
+
+
+register_mixer("fixed_decay", FixedDecayAttention)
 register_mixer("gla", GatedLinearAttention)
 register_mixer("ssd", StateSpaceDuality)
