@@ -30,6 +30,8 @@ __global__ void __launch_bounds__(128)
 gated_rmsnorm_kernel(const float* __restrict__ x, const float* __restrict__ w, const T* __restrict__ gate, int ld_gate,
                      T* __restrict__ out, int ld_out, float mul, int n_heads, int d, int n_rows, float eps, int gate_act, int gate_first,
                      int weight_per_row) {
+    pdl_launch_dependents();
+    pdl_wait();
     const int row = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
     if (row >= n_rows) return;
     const int t = row / n_heads, h = row % n_heads;
@@ -63,6 +65,8 @@ gated_rmsnorm_wide_kernel(const float* __restrict__ x, const float* __restrict__
                           T* __restrict__ out, int ld_out, float mul, int n_heads, int d, float eps, int gate_act, int gate_first,
                           int weight_per_row) {
     __shared__ float scratch[33];
+    pdl_launch_dependents();
+    pdl_wait();
     const int row = blockIdx.x;
     const int t = row / n_heads, h = row % n_heads;
     const float* xr = x + (size_t)row * d;
@@ -188,13 +192,10 @@ extern "C" int b200_gated_rmsnorm(const float* x, const float* w, const void* ga
     if (rows > 0x7fffffffLL) return b200::kErrUnsupportedSize;
     B200_DISPATCH_DTYPE(dtype, T,
         if (d >= 512)      // (a warp would walk such a row in 16 or more rounds, twice)
-            b200::gated_rmsnorm_wide_kernel<T><<<(int)rows, b200::kWideThreads, 0, stream>>>(x, w, (const T*)gate, ld_gate, (T*)out, ld_out, mul,
-                                                                                           n_heads, d, eps, gate_act, gate_first,
-                                                                                           weight_per_row);
-        else
-            b200::gated_rmsnorm_kernel<T><<<(int)((rows + 3) / 4), 128, 0, stream>>>(x, w, (const T*)gate, ld_gate, (T*)out, ld_out, mul,
-                                                                                     n_heads, d, (int)rows, eps, gate_act, gate_first,
-                                                                                     weight_per_row));
+            return b200::launch_pdl(b200::gated_rmsnorm_wide_kernel<T>, dim3((unsigned)rows), dim3(b200::kWideThreads), 0, stream, x, w,
+                                    (const T*)gate, ld_gate, (T*)out, ld_out, mul, n_heads, d, eps, gate_act, gate_first, weight_per_row);
+        return b200::launch_pdl(b200::gated_rmsnorm_kernel<T>, dim3((unsigned)((rows + 3) / 4)), dim3(128), 0, stream, x, w, (const T*)gate,
+                                ld_gate, (T*)out, ld_out, mul, n_heads, d, (int)rows, eps, gate_act, gate_first, weight_per_row));
     return b200::launch_status();
 }
 

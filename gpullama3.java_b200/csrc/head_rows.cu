@@ -162,6 +162,8 @@ template <typename T>
 __global__ void __launch_bounds__(kRowThreads)
 head_rows_kernel(const T* __restrict__ src, int ld_src, T* __restrict__ dst, int ld_dst, const float* __restrict__ bias,
                  const float* __restrict__ weight, RowSegments segs, float eps, CacheTarget cache, MixSource mix) {
+    pdl_launch_dependents();
+    pdl_wait();
     const int t = blockIdx.x, lane = threadIdx.x & 31;
     int row = blockIdx.y * (kRowThreads / 32) + (threadIdx.x >> 5);
     if (row >= segs.total_rows) return;
@@ -273,7 +275,7 @@ extern "C" int b200_head_rows(const void* src, int ld_src, void* dst, int ld_dst
         return b200::launch_status();
     }
     B200_DISPATCH_DTYPE(dtype, T,
-        b200::head_rows_kernel<T><<<grid, b200::kRowThreads, 0, stream>>>((const T*)src, ld_src, (T*)dst, ld_dst, bias,
-                                                                          weight, segs, eps, cache, mix));
+        return b200::launch_pdl(b200::head_rows_kernel<T>, grid, dim3(b200::kRowThreads), 0, stream, (const T*)src, ld_src, (T*)dst, ld_dst,
+                                bias, weight, segs, eps, cache, mix));
     return b200::launch_status();
 }

@@ -107,6 +107,10 @@ _SIGNATURES = {
                                         c_void_p, c_void_p, ctypes.c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
                                         c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_int, c_int, c_int, c_int,
                                         c_int, c_void_p, c_void_p]),
+    "b200_fixed_decay": ("fixed_decay", [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, ctypes.c_longlong,
+                                         c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int,
+                                         c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_int, c_int, c_void_p,
+                                         c_int, c_float, c_float]),
     "b200_moe_table_route": ("moe", [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int]),
     "b200_layernorm": ("norm", [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_float]),
     "b200_causal_conv_silu": ("delta_rule", [c_void_p, c_int, c_void_p, c_void_p, ctypes.c_longlong, c_void_p, c_void_p,
@@ -1274,6 +1278,64 @@ def linear_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.
                                    float(power), int(decay_kind), 1 if decay_per_head else 0, 1 if step_scales_value else 0,
                                    1 if qk_silu else 0, 1 if v_silu else 0, inv_freq.numel() if inv_freq is not None else 0,
                                    ptr(inv_freq), ptr(rot_pos), _stream()), "linear_scan")
+
+
+def fixed_decay_takes(dtype: torch.dtype, all_single: bool, d_k: int, d_v: int) -> bool:
+    """Whether ``fixed_decay`` takes these sizes: any of one token per sequence, in either precision; longer ones in bfloat16
+    where a run's tiles fit an SM's shared memory."""
+    if all_single:
+        return d_k <= 512
+    return dtype == torch.bfloat16 and int(library("fixed_decay").b200_fixed_decay_columns(c_int(d_k), c_int(d_v))) > 0
+
+
+def fixed_decay_finishes(all_single: bool, d_k: int, d_v: int) -> bool:
+    """Whether a CTA of ``fixed_decay`` has all of a head's values, so that it can also norm and gate them."""
+    lib = library("fixed_decay")
+    if all_single:
+        return bool(lib.b200_fixed_decay_step_finishes(c_int(d_v)))
+    return d_v <= int(lib.b200_fixed_decay_columns(c_int(d_k), c_int(d_v)))
+
+
+def fixed_decay(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, state: torch.Tensor, slots: torch.Tensor,
+                cu_seqlens: torch.Tensor, positions: torch.Tensor, heads: int, d_k: int, d_v: int, max_q_len: int, *,
+                q_scale: float = 1.0, qk_silu: bool = False, v_silu: bool = False, inv_freq: torch.Tensor | None = None,
+                angles: torch.Tensor | None = None, out: torch.Tensor | None = None, finish=None, alloc=None) -> None:
+    """S <- g S + k v^T, o = S^T (q_scale q) per head over a packed step, g = decay[h] (float32 [heads]), S the float32 [slots,
+    >= heads d_k d_v] ``state`` at the sequence's slot, updated in place.  q, k [T, >= heads d_k], v [T, >= heads d_v] of one type;
+    ``qk_silu`` / ``v_silu``: they pass through SiLU; ``inv_freq`` float32 [n] (and for steps of more than one token per sequence
+    ``angles`` float32 [n, T, 2], ``rope_angles`` of the pass): the pairs (i, i + n) of q and k are turned by the positions.
+    ``out`` float32 [T, heads d_v], or ``finish`` = (rows [T, heads d_v], gate [T, >= heads d_v], activation, eps, mul): rows = o /
+    sqrt(mean(o^2) + eps) per head * act(gate) * mul, rows being columns of a wider buffer."""
+    _dev(q, k, v, decay, state, slots, cu_seqlens, positions, inv_freq, angles, out)
+    T = q.shape[0]
+    assert q.dtype == k.dtype == v.dtype and q.stride(1) == k.stride(1) == v.stride(1) == 1
+    assert q.shape[1] >= heads * d_k and k.shape[1] >= heads * d_k and v.shape[1] >= heads * d_v
+    assert decay.dtype == state.dtype == torch.float32 and decay.numel() == heads and decay.is_contiguous() and state.stride(1) == 1
+    assert state.shape[1] >= heads * d_k * d_v and positions.dtype == torch.int32 and positions.numel() == T
+    pairs = inv_freq.numel() if inv_freq is not None else 0
+    single = T == slots.numel()
+    assert pairs == 0 or (inv_freq.dtype == torch.float32 and inv_freq.is_contiguous() and 2 * pairs <= d_k)
+    assert pairs == 0 or single or (angles.dtype == torch.float32 and angles.is_contiguous() and tuple(angles.shape) == (pairs, T, 2))
+    scratch = None
+    if not single:
+        shape = (int(library("fixed_decay").b200_fixed_decay_runs(c_int(T), c_int(slots.numel()))), heads, d_k, d_v)
+        scratch = alloc(shape, torch.float32) if alloc is not None else torch.empty(shape, dtype=torch.float32, device=q.device)
+    rows = gate = None
+    act, eps, mul = "silu", 0.0, 1.0
+    if finish is not None:
+        rows, gate, act, eps, mul = finish
+        _dev(rows, gate)
+        assert out is None and rows.dtype == gate.dtype == q.dtype and rows.stride(1) == gate.stride(1) == 1
+        assert tuple(rows.shape) == (T, heads * d_v) and gate.shape[0] == T and gate.shape[1] >= heads * d_v
+    else:
+        assert out.dtype == torch.float32 and out.is_contiguous() and tuple(out.shape) == (T, heads * d_v)
+    ptr = lambda t: t.data_ptr() if t is not None else None
+    _check(_fn("b200_fixed_decay")(
+        q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0), decay.data_ptr(), state.data_ptr(),
+        state.stride(0), slots.data_ptr(), cu_seqlens.data_ptr(), positions.data_ptr(), ptr(inv_freq), ptr(angles), pairs, ptr(out),
+        ptr(scratch), dtype_code(q.dtype), T, slots.numel(), int(max_q_len), heads, d_k, d_v, float(q_scale), 1 if qk_silu else 0,
+        1 if v_silu else 0, ptr(gate), gate.stride(0) if gate is not None else 0, GATE_ACTIVATIONS[act], ptr(rows),
+        rows.stride(0) if rows is not None else 0, float(eps), float(mul), _stream()), "fixed_decay" if not single else "fixed_decay:step")
 
 
 def delta_rule_supported(d_k: int) -> bool:

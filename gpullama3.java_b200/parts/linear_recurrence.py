@@ -23,7 +23,7 @@ delta rule's correction:  S_t = diag(g_t) S_(t-1) + k_t (b_t v_t)^T,  o_t = S_t^
 All keep, per sequence, S of every head in 32 bits (and the convolution's last inputs) in one row of their cache slot,
 starting from zero.  Decays, step sizes, the recurrence and the output norms are 32-bit in both precisions; projections
 and the convolution are computed in the run's precision.  The scan is the kernel of the delta rule, told to leave out
-the correction."""
+the correction; a decay fixed per head has kernels of its own, which take runs of tokens at once (``ops.fixed_decay``)."""
 from __future__ import annotations
 
 import torch
@@ -185,7 +185,7 @@ class FixedDecayAttention(Mixer, OpenEnded):
         if activation not in (None, "silu") or norm_over not in ("head", "all") or gate not in ops.GATE_ACTIVATIONS:
             raise ConfigError(f"fixed-decay attention: activation {activation!r}, norm over {norm_over!r}, gate {gate!r}")
         if position is not None and position.rotary_dim:
-            if position.rotary_dim > head_dim or position.pairing != PAIRING_CODES["half"]:
+            if position.rotary_dim > head_dim or position.pairing != PAIRING_CODES["half"] or not hasattr(position, "angles"):
                 raise ConfigError(f"fixed-decay attention turns pairs over halves of at most {head_dim} numbers")
         self.hidden_size, self.n_heads, self.key_dim, self.value_dim = int(hidden_size), int(n_heads), int(head_dim), int(value_dim)
         self.decay, self.norm_eps, self.scale = [float(g) for g in decay], float(norm_eps), float(scale)
@@ -240,13 +240,27 @@ class FixedDecayAttention(Mixer, OpenEnded):
 
     def rows_from(self, raw, ctx: StepContext, cache: StateView, rows, writes_cache=True, mul=1.0):
         H, dk, dv, T = self.n_heads, self.key_dim, self.value_dim, raw.shape[0]
-        o = ctx.empty((T, H * dv), torch.float32)
-        ops.linear_scan(raw[:, self.q_off:], raw[:, self.k_off:], raw[:, self.v_off:], None, cache.data, ctx.slots_dev,
-                        ctx.cu_seqlens, o, H, H, dk, dv, decay_kind=ops.DECAY_FIXED, decay_per_head=True, a_log=self.decays,
-                        q_scale=self.scale, qk_silu=self.silu, v_silu=self.silu,
-                        rotary=(ctx.positions, self.inv_freq) if self.inv_freq is not None else None, alloc=ctx.empty)
+        q, k, v, g = (raw[:, at:] for at in (self.q_off, self.k_off, self.v_off, self.g_off))
+        if ops.fixed_decay_takes(ctx.dtype, ctx.all_decode, dk, dv):
+            # (a head that is normed alone and without a weight is finished where its values are)
+            finish = None
+            if self.norm_over == "head" and self.weight is None and ops.fixed_decay_finishes(ctx.all_decode, dk, dv):
+                finish = (rows, g, self.gate, self.norm_eps, mul)
+            o = None if finish is not None else ctx.empty((T, H * dv), torch.float32)
+            angles = self.position.angles(ctx) if self.inv_freq is not None and not ctx.all_decode else None
+            ops.fixed_decay(q, k, v, self.decays, cache.data, ctx.slots_dev, ctx.cu_seqlens, ctx.positions, H, dk, dv, ctx.max_q_len,
+                            q_scale=self.scale, qk_silu=self.silu, v_silu=self.silu, inv_freq=self.inv_freq, angles=angles, out=o,
+                            finish=finish, alloc=ctx.empty)
+            if finish is not None:
+                return
+        else:
+            # (the true 32-bit run's prompts, and keys too long for a run's tiles: token by token)
+            o = ctx.empty((T, H * dv), torch.float32)
+            ops.linear_scan(q, k, v, None, cache.data, ctx.slots_dev, ctx.cu_seqlens, o, H, H, dk, dv, decay_kind=ops.DECAY_FIXED,
+                            decay_per_head=True, a_log=self.decays, q_scale=self.scale, qk_silu=self.silu, v_silu=self.silu,
+                            rotary=(ctx.positions, self.inv_freq) if self.inv_freq is not None else None, alloc=ctx.empty)
         parts, d = (H, dv) if self.norm_over == "head" else (1, H * dv)
-        ops.gated_rmsnorm(o, self.weight, raw[:, self.g_off:], rows, parts, d, self.norm_eps, self.gate, mul=mul)
+        ops.gated_rmsnorm(o, self.weight, g, rows, parts, d, self.norm_eps, self.gate, mul=mul)
 
     def forward(self, x, ctx: StepContext, cache: StateView, residual, writes_cache=True, then_norm=None):
         rows = ctx.empty((x.shape[0], self.open_columns()), ctx.dtype)
