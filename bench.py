@@ -2,7 +2,7 @@
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--model 1b|3b|8b] [--dtype bfloat16|float32]
                     [--batch 8] [--context 4096] [--layers L] [--sizes all|none]
-    python bench.py --design guduzen|pekerax|gatuzen|bisudra [--design-sizes s,m]     (another workload, see the end of this text)
+    python bench.py --design guduzen|pekerax|gatuzen|bisudra|fazezen [--design-sizes s,m]     (another workload, see the end of this text)
 
 Default run: the Llama-3.2-1B shape with random bfloat16 weights, a
 batch of 8 sequences at context length 4096.  A "step" is one decode step.  ``value`` is decoded
@@ -43,6 +43,12 @@ gated and layer-normed on their way back into it; a 4-tap input convolution; 64 
 the stream; every layer's result mixed with all earlier ones; feed-forwards dense and routed in turn, 8 experts of half
 the dense width, 2 per token) beside the Pekerax decoder, the closest existing model (window attention with an output
 gate, layer norms, dense and routed feed-forwards), and the Llama 3 decoder, all of equal width, depth and projections.
+
+``--design fazezen`` does the same for the Fazezen decoder (mixer and feed-forward side by side; layers in the order
+attention within runs of positions beside retention, lightning attention, lightning attention; dense GELU-gated
+feed-forwards with biases) beside the Guduzen decoder, the closest existing model (attention, a recurrence, dense
+GELU-gated feed-forwards), the Gatuzen decoder (linear attention on the scan) and the Llama 3 decoder, all of equal
+width, depth and projections.
 
 The library runs on one GPU: for --gpus N > 1 it says so and exits with 2.
 """
@@ -480,6 +486,21 @@ def bisudra_config(z):
             "token_side": {"dim": 64}, "layers": layers}
 
 
+def fazezen_config(z):
+    """Layers in the order parallel, lightning, lightning, repeated: in a parallel layer attention within runs of positions
+    and retention share the heads (half of them each: the projections have the sizes of the other decoders'), a
+    lightning layer has them all; every feed-forward dense, beside the mixer."""
+    H, G, d = z["heads"] // 2, max(1, z["kv_heads"] // 2), z["dim"]
+    left = {"heads": H, "kv_heads": G, "dim": d, "vdim": d, "scale": d ** -0.5, "mask": {"size": z["window"]},
+            "rot": {"base": 500000.0, "dims": d, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}
+    right = {"heads": H, "dim": d, "vdim": d, "decay": [1.0 - 2.0 ** -(5 + i % 8) for i in range(H)], "rot": {"base": 10000.0, "dims": d}}
+    par = {"left": left, "right": right, "left_scale": 1.0, "right_scale": 1.0}
+    lig = {"heads": 2 * H, "dim": d, "vdim": d, "decay": [1.0 - 2.0 ** -(1 + i % 10) for i in range(2 * H)]}
+    layers = [{"type": "parallel" if i % 3 == 0 else "lightning", "mixer": dict(par if i % 3 == 0 else lig),
+               "mlp": {"kind": "dense", "ff": z["ff"]}} for i in range(z["layers"])]
+    return {"architecture": "Fazezen", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-6}, "layers": layers}
+
+
 def llama_like(z):
     return {"architectures": ["LlamaForCausalLM"], "num_hidden_layers": z["layers"], "hidden_size": z["width"],
             "num_attention_heads": z["heads"], "num_key_value_heads": z["kv_heads"], "head_dim": z["dim"],
@@ -565,6 +586,8 @@ DESIGNS = {
                                 "layer-normed into the stream, input convolution, token input, every layer's result "
                                 "mixed with the earlier ones, feed-forwards dense and routed in turn (8 experts, 2 per "
                                 "token)", ("pekerax", "llama")),
+    "fazezen": (fazezen_config, "Fazezen, layers attention within runs of positions beside retention / lightning attention / "
+                                "lightning attention, dense feed-forwards beside the mixers", ("guduzen", "gatuzen", "llama")),
 }
 
 
@@ -576,7 +599,7 @@ def run_design(args, peaks, peak_source, clocks) -> int:
     sizes = {}
     name = args.design
     make, what, beside = DESIGNS[name]
-    others = {"guduzen": guduzen_config, "pekerax": pekerax_config, "llama": llama_like}
+    others = {"guduzen": guduzen_config, "pekerax": pekerax_config, "gatuzen": gatuzen_config, "llama": llama_like}
     for key in (args.design_sizes.split(",") if args.design_sizes else sorted(DESIGN_SIZES, reverse=True)):
         z = DESIGN_SIZES[key]
         sizes[key] = {"sizes": z, name: run_design_arm(make(z), f"{name} {key}", args, peaks)}

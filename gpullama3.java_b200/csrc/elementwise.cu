@@ -57,14 +57,41 @@ gated_rmsnorm_kernel(const float* __restrict__ x, const float* __restrict__ w, c
 }
 
 // a CTA per row, for rows too long for one warp (a norm over a large part of the mixer's output); the gated values stay
-// in registers between the two passes when the row has at most kWideKeep numbers per thread
+// in registers between the two passes when the row has at most kWideKeep * VEC numbers per thread.  VEC 4: 16-byte accesses of
+// the row and the weight, where sizes and pointers allow.
 constexpr int kWideThreads = 256, kWideKeep = 8;
-template <typename T>
+template <typename T, int VEC> __device__ __forceinline__ void load_row(const T* p, float (&f)[VEC]) {
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) f[e] = to_f32<T>(p[e]);
+}
+template <> __device__ __forceinline__ void load_row<float, 4>(const float* p, float (&f)[4]) {
+    const float4 v = *reinterpret_cast<const float4*>(p);
+    f[0] = v.x; f[1] = v.y; f[2] = v.z; f[3] = v.w;
+}
+template <> __device__ __forceinline__ void load_row<__nv_bfloat16, 4>(const __nv_bfloat16* p, float (&f)[4]) {
+    const uint2 v = *reinterpret_cast<const uint2*>(p);
+    f[0] = __uint_as_float(v.x << 16); f[1] = __uint_as_float(v.x & 0xffff0000u);
+    f[2] = __uint_as_float(v.y << 16); f[3] = __uint_as_float(v.y & 0xffff0000u);
+}
+template <typename T, int VEC> __device__ __forceinline__ void store_row(T* p, const float (&f)[VEC]) {
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) p[e] = from_f32<T>(f[e]);
+}
+template <> __device__ __forceinline__ void store_row<float, 4>(float* p, const float (&f)[4]) {
+    *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
+}
+template <> __device__ __forceinline__ void store_row<__nv_bfloat16, 4>(__nv_bfloat16* p, const float (&f)[4]) {
+    const __nv_bfloat162 a = __floats2bfloat162_rn(f[0], f[1]), b = __floats2bfloat162_rn(f[2], f[3]);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+}
+
+template <typename T, int VEC>
 __global__ void __launch_bounds__(kWideThreads)
 gated_rmsnorm_wide_kernel(const float* __restrict__ x, const float* __restrict__ w, const T* __restrict__ gate, int ld_gate,
                           T* __restrict__ out, int ld_out, float mul, int n_heads, int d, float eps, int gate_act, int gate_first,
                           int weight_per_row) {
     __shared__ float scratch[33];
+    constexpr int kKeep = VEC == 4 ? 2 : kWideKeep, kStep = kWideThreads * VEC;
     pdl_launch_dependents();
     pdl_wait();
     const int row = blockIdx.x;
@@ -72,33 +99,55 @@ gated_rmsnorm_wide_kernel(const float* __restrict__ x, const float* __restrict__
     const float* xr = x + (size_t)row * d;
     const T* g = gate + (size_t)t * ld_gate + (size_t)h * d;
     const float* wr = w ? w + (weight_per_row ? (size_t)h * d : 0) : nullptr;
-    auto weight = [&](int e) { return wr ? wr[e] : 1.f; };
-    auto act = [&](int e) {
-        const float z = to_f32<T>(g[e]);
-        const float sig = 1.0f / (1.0f + expf(-z));
-        return gate_act == 1 ? z * sig : sig;
-    };
-    float keep[kWideKeep], ss = 0.f;
+    // a piece of VEC numbers from column e on, multiplied by its gate where the gate comes first; `a` holds the gate otherwise
+    auto piece = [&](int e, float (&v)[VEC], float (&a)[VEC]) {
+        load_row<float, VEC>(xr + e, v);
+        load_row<T, VEC>(g + e, a);
 #pragma unroll
-    for (int i = 0; i < kWideKeep; ++i) {
-        const int e = threadIdx.x + i * kWideThreads;
-        keep[i] = e < d ? (gate_first ? xr[e] * act(e) : xr[e]) : 0.f;
-        ss += keep[i] * keep[i];
+        for (int i = 0; i < VEC; ++i) {
+            const float sig = 1.0f / (1.0f + expf(-a[i]));
+            a[i] = gate_act == 1 ? a[i] * sig : sig;
+            if (gate_first) { v[i] *= a[i]; a[i] = 1.f; }
+        }
+    };
+    float keep[kKeep][VEC], act[kKeep][VEC], ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < kKeep; ++i) {
+        const int e = threadIdx.x * VEC + i * kStep;
+        if (e < d) {
+            piece(e, keep[i], act[i]);
+#pragma unroll
+            for (int c = 0; c < VEC; ++c) ss += keep[i][c] * keep[i][c];
+        }
     }
-    for (int e = threadIdx.x + kWideKeep * kWideThreads; e < d; e += kWideThreads) {
-        const float v = gate_first ? xr[e] * act(e) : xr[e];
-        ss += v * v;
+    for (int e = threadIdx.x * VEC + kKeep * kStep; e < d; e += kStep) {
+        float v[VEC], a[VEC];
+        piece(e, v, a);
+#pragma unroll
+        for (int c = 0; c < VEC; ++c) ss += v[c] * v[c];
     }
     ss = block_sum(ss, scratch);
     const float scale = mul / sqrtf(ss / (float)d + eps);
     T* o = out + (size_t)t * ld_out + (size_t)h * d;
+    auto finish = [&](int e, float (&v)[VEC], const float (&a)[VEC]) {
+        float wv[VEC];
 #pragma unroll
-    for (int i = 0; i < kWideKeep; ++i) {
-        const int e = threadIdx.x + i * kWideThreads;
-        if (e < d) o[e] = from_f32<T>(gate_first ? keep[i] * scale * weight(e) : keep[i] * scale * weight(e) * act(e));
+        for (int c = 0; c < VEC; ++c) wv[c] = 1.f;
+        if (wr) load_row<float, VEC>(wr + e, wv);
+#pragma unroll
+        for (int c = 0; c < VEC; ++c) v[c] = v[c] * scale * wv[c] * a[c];
+        store_row<T, VEC>(o + e, v);
+    };
+#pragma unroll
+    for (int i = 0; i < kKeep; ++i) {
+        const int e = threadIdx.x * VEC + i * kStep;
+        if (e < d) finish(e, keep[i], act[i]);
     }
-    for (int e = threadIdx.x + kWideKeep * kWideThreads; e < d; e += kWideThreads)
-        o[e] = from_f32<T>(gate_first ? (xr[e] * act(e)) * scale * weight(e) : xr[e] * scale * weight(e) * act(e));
+    for (int e = threadIdx.x * VEC + kKeep * kStep; e < d; e += kStep) {
+        float v[VEC], a[VEC];
+        piece(e, v, a);
+        finish(e, v, a);
+    }
 }
 
 template <typename T>
@@ -139,8 +188,30 @@ differential_heads_kernel(const T* __restrict__ maps, const T* __restrict__ gate
     }
 }
 
+// VEC neighbouring pairs per thread (4: 8-byte accesses of 16-bit numbers, where sizes and pointers allow)
 constexpr int kTurnThreads = 128, kTurnPairs = 256;
-template <typename T>
+template <typename T, int VEC> struct TurnVec {
+    __device__ static void load(const T* p, float (&f)[VEC]) {
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) f[e] = to_f32<T>(p[e]);
+    }
+    __device__ static void store(T* p, const float (&f)[VEC]) {
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) p[e] = from_f32<T>(f[e]);
+    }
+};
+template <> struct TurnVec<__nv_bfloat16, 4> {
+    __device__ static void load(const __nv_bfloat16* p, float (&f)[4]) {
+        const uint2 v = *reinterpret_cast<const uint2*>(p);
+        f[0] = __uint_as_float(v.x << 16); f[1] = __uint_as_float(v.x & 0xffff0000u);
+        f[2] = __uint_as_float(v.y << 16); f[3] = __uint_as_float(v.y & 0xffff0000u);
+    }
+    __device__ static void store(__nv_bfloat16* p, const float (&f)[4]) {
+        const __nv_bfloat162 a = __floats2bfloat162_rn(f[0], f[1]), b = __floats2bfloat162_rn(f[2], f[3]);
+        *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+    }
+};
+template <typename T, int VEC>
 __global__ void __launch_bounds__(kTurnThreads)
 turn_back_rows_kernel(const T* __restrict__ x, const int* __restrict__ positions, const float* __restrict__ inv_freq,
                       T* __restrict__ out, int ld_out, int n_heads, int d, int d_pad, float mul) {
@@ -159,12 +230,20 @@ turn_back_rows_kernel(const T* __restrict__ x, const int* __restrict__ positions
             o[u] = from_f32<T>(to_f32<T>(xr[(size_t)(u / d) * d_pad + u % d]) * mul);
         return;
     }
-    for (int u = blockIdx.y * kTurnThreads + threadIdx.x; u < n_heads * n; u += gridDim.y * kTurnThreads) {
-        const int h = u / n, i = u % n;
-        const float a = to_f32<T>(xr[(size_t)h * d_pad + i]), b = to_f32<T>(xr[(size_t)h * d_pad + i + n]);
-        const float c = cos_s[i], s = sin_s[i];
-        o[(size_t)h * d + i] = from_f32<T>((a * c + b * s) * mul);
-        o[(size_t)h * d + i + n] = from_f32<T>((b * c - a * s) * mul);
+    const int per_head = n / VEC;
+    for (int u = blockIdx.y * kTurnThreads + threadIdx.x; u < n_heads * per_head; u += gridDim.y * kTurnThreads) {
+        const int h = u / per_head, i = (u % per_head) * VEC;
+        float a[VEC], b[VEC];
+        TurnVec<T, VEC>::load(xr + (size_t)h * d_pad + i, a);
+        TurnVec<T, VEC>::load(xr + (size_t)h * d_pad + i + n, b);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) {
+            const float c = cos_s[i + e], s = sin_s[i + e], p = a[e], q = b[e];
+            a[e] = (p * c + q * s) * mul;
+            b[e] = (q * c - p * s) * mul;
+        }
+        TurnVec<T, VEC>::store(o + (size_t)h * d + i, a);
+        TurnVec<T, VEC>::store(o + (size_t)h * d + i + n, b);
     }
 }
 
@@ -190,10 +269,17 @@ extern "C" int b200_gated_rmsnorm(const float* x, const float* w, const void* ga
     if (d < 1 || ld_out < n_heads * d) return b200::kErrBadArgument;
     const long long rows = (long long)n_tokens * n_heads;
     if (rows > 0x7fffffffLL) return b200::kErrUnsupportedSize;
+    const size_t el = dtype == b200::kF32 ? 4 : 2;
+    const bool wide4 = d % 4 == 0 && ld_gate % 4 == 0 && ld_out % 4 == 0 && (((uintptr_t)x | (uintptr_t)w) & 15) == 0 &&
+                       ((uintptr_t)gate % (4 * el)) == 0 && ((uintptr_t)out % (4 * el)) == 0;
     B200_DISPATCH_DTYPE(dtype, T,
-        if (d >= 512)      // (a warp would walk such a row in 16 or more rounds, twice)
-            return b200::launch_pdl(b200::gated_rmsnorm_wide_kernel<T>, dim3((unsigned)rows), dim3(b200::kWideThreads), 0, stream, x, w,
+        if (d >= 512) {    // (a warp would walk such a row in 16 or more rounds, twice)
+            if (wide4)
+                return b200::launch_pdl(b200::gated_rmsnorm_wide_kernel<T, 4>, dim3((unsigned)rows), dim3(b200::kWideThreads), 0, stream, x, w,
+                                        (const T*)gate, ld_gate, (T*)out, ld_out, mul, n_heads, d, eps, gate_act, gate_first, weight_per_row);
+            return b200::launch_pdl(b200::gated_rmsnorm_wide_kernel<T, 1>, dim3((unsigned)rows), dim3(b200::kWideThreads), 0, stream, x, w,
                                     (const T*)gate, ld_gate, (T*)out, ld_out, mul, n_heads, d, eps, gate_act, gate_first, weight_per_row);
+        }
         return b200::launch_pdl(b200::gated_rmsnorm_kernel<T>, dim3((unsigned)((rows + 3) / 4)), dim3(128), 0, stream, x, w, (const T*)gate,
                                 ld_gate, (T*)out, ld_out, mul, n_heads, d, (int)rows, eps, gate_act, gate_first, weight_per_row));
     return b200::launch_status();
@@ -238,11 +324,15 @@ extern "C" int b200_turn_back_rows(const void* x, const int* positions, const fl
     if (n_tokens <= 0 || n_heads <= 0) return 0;
     if (d < 1 || d_pad < d || ld_out < n_heads * d || (inv_freq && (d % 2 || !positions))) return b200::kErrBadArgument;
     if (inv_freq && d / 2 > b200::kTurnPairs) return b200::kErrUnsupportedSize;
-    const int units = n_heads * (inv_freq ? d / 2 : d);
+    const bool vec = inv_freq && d % 8 == 0 && d_pad % 4 == 0 && ld_out % 4 == 0 && (((uintptr_t)x | (uintptr_t)out) & 7) == 0 && dtype == b200::kBF16;
+    const int units = n_heads * (inv_freq ? d / 2 : d) / (vec ? 4 : 1);
     int ny = n_tokens >= 512 ? 1 : (units + b200::kTurnThreads - 1) / b200::kTurnThreads;   // few tokens: a token's heads over several CTAs
     if (ny > 64) ny = 64;
     B200_DISPATCH_DTYPE(dtype, T,
-        return b200::launch_pdl(b200::turn_back_rows_kernel<T>, dim3(n_tokens, ny), dim3(b200::kTurnThreads), 0, stream, (const T*)x,
+        if (vec)
+            return b200::launch_pdl(b200::turn_back_rows_kernel<T, 4>, dim3(n_tokens, ny), dim3(b200::kTurnThreads), 0, stream, (const T*)x,
+                                    positions, inv_freq, (T*)out, ld_out, n_heads, d, d_pad, mul);
+        return b200::launch_pdl(b200::turn_back_rows_kernel<T, 1>, dim3(n_tokens, ny), dim3(b200::kTurnThreads), 0, stream, (const T*)x,
                                 positions, inv_freq, (T*)out, ld_out, n_heads, d, d_pad, mul));
     return 0;
 }

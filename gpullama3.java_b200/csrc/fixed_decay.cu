@@ -13,10 +13,12 @@
 // so the work is (1) every run's own sum of outer products, all runs of all heads at once, (2) the states before every
 // run, a short sequential pass over the runs' sums, element by element, (3) the outputs, all runs of all heads at once.
 // (1) and (3) are products of 64-token tiles on the tensor cores.  What enters the recurrence is kept in 32 bits, and a
-// tensor-core operand has 16: q, k, the decayed keys, the decayed scores and the state therefore enter as the sum of two
-// bfloat16 numbers (x = hi + lo, 16 bits of mantissa), products of two such sums without the lo lo term; sums are 32-bit.
-// The powers of g are exact to 32-bit rounding (powf).  v enters as one bfloat16 number (it is a projection with its activation).
-// A sequence's runs start at the step's first token of the sequence; the last one may be short.
+// tensor-core operand has 16: turned queries and keys, the decayed keys, the decayed scores and the state therefore enter as
+// the sum of two bfloat16 numbers (x = hi + lo, 16 bits of mantissa), products of two such sums without the lo lo term; sums
+// are 32-bit.  The powers of g are exact to 32-bit rounding (powf).  Projections, with SiLU or without, enter as the one
+// bfloat16 number they are stored as.  A sequence's runs start at the step's first token of the sequence; the last one may be
+// short.  The tiles are read as they lie in memory, 16 bytes at a time: where queries and keys have to be turned or
+// activated, or a head's size is off that grid, a kernel in front of the three leaves them so (fixed_decay_prepare).
 #include "common.cuh"
 
 namespace b200 {
@@ -36,9 +38,14 @@ struct FixedDecayArgs {
     const int* cu_seqlens;
     const float* inv_freq;  // [pairs] or null
     const int* positions;   // [T]
-    const float2* angles;   // [pairs][T] (cos, sin) or null: the prompt kernels read these
     float* out;             // [T, heads d_v] 32-bit, or null when the head is finished here
-    float* runs;            // scratch of the prompt kernels: [run][head][d_k][d_v]
+    float* runs;            // scratch of the prompt kernels: [run][head][d_k][d_v]; behind the second one the state before the
+                            // run as (hi, lo) pairs of bfloat16 in the place of each number
+    // how the prompt kernels read the operands: rows of bfloat16 on 16-byte boundaries, head h at column h * head_qk (head_v)
+    const __nv_bfloat16* qt[2];   // hi and lo (the second where the operand has two parts)
+    const __nv_bfloat16* kt[2];
+    const __nv_bfloat16* vt;
+    int ld_qt, ld_kt, ld_vt, head_qk, head_v;
     int n_tokens, heads, d_k, d_v, pairs, qk_silu, v_silu;
     float q_scale;
     // the finished head: o / sqrt(mean(o^2) + eps) * act(gate) * mul into columns of a buffer of the operands' type
@@ -181,22 +188,10 @@ __device__ __forceinline__ uint32_t pack_pair(float lo, float hi) {
     const __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
     return *reinterpret_cast<const uint32_t*>(&v);
 }
-// x = hi + lo in two bfloat16 numbers
-__device__ __forceinline__ void split_store(__nv_bfloat16* hi, __nv_bfloat16* lo, float x) {
-    const __nv_bfloat16 h = __float2bfloat16_rn(x);
-    *hi = h;
-    *lo = __float2bfloat16_rn(x - __bfloat162float(h));
-}
-__device__ __forceinline__ void split_store8(__nv_bfloat16* hi, __nv_bfloat16* lo, const float (&x)[8]) {
-    uint32_t h[4], l[4];
-#pragma unroll
-    for (int i = 0; i < 4; ++i) {
-        const float a = x[2 * i], b = x[2 * i + 1];
-        h[i] = pack_pair(a, b);
-        l[i] = pack_pair(a - __uint_as_float(h[i] << 16), b - __uint_as_float(h[i] & 0xffff0000u));
-    }
-    *reinterpret_cast<uint4*>(hi) = make_uint4(h[0], h[1], h[2], h[3]);
-    *reinterpret_cast<uint4*>(lo) = make_uint4(l[0], l[1], l[2], l[3]);
+// a pair of numbers as bfloat16 pairs hi and lo, x = hi + lo
+__device__ __forceinline__ void split_pair(float a, float b, uint32_t& hi, uint32_t& lo) {
+    hi = pack_pair(a, b);
+    lo = pack_pair(a - __uint_as_float(hi << 16), b - __uint_as_float(hi & 0xffff0000u));
 }
 __device__ __forceinline__ void load8(const __nv_bfloat16* p, float (&f)[8]) {
     const uint4 v = *reinterpret_cast<const uint4*>(p);
@@ -208,96 +203,100 @@ __device__ __forceinline__ void load8(const __nv_bfloat16* p, float (&f)[8]) {
     }
 }
 
-// A run's rows of q or k as hi and lo tiles [kRun][ld] in shared memory (columns d_k .. d_pad and rows beyond the run
-// zero), each row times factor[row] (null: 1) and `scale`.  Two threads share a token's row; 8 numbers per access where the
-// rows lie on 16-byte boundaries.
-__device__ __forceinline__ void load_rows_split(const FixedDecayArgs& a, const __nv_bfloat16* src, int ld_src, int first, int n, int h,
-                                                __nv_bfloat16* hi, __nv_bfloat16* lo, int ld, int d_pad, float scale,
-                                                const float* factor) {
-    const int r = threadIdx.x & (kRun - 1), part = threadIdx.x >> 6;
-    __nv_bfloat16* hr = hi + (size_t)r * ld;
-    __nv_bfloat16* lr = lo + (size_t)r * ld;
-    if (r >= n) {
-        for (int c = part * 8; c < d_pad; c += 16) {
-            *reinterpret_cast<uint4*>(hr + c) = make_uint4(0, 0, 0, 0);
-            *reinterpret_cast<uint4*>(lr + c) = make_uint4(0, 0, 0, 0);
-        }
-        return;
+__device__ __forceinline__ void load4(const __nv_bfloat16* p, float (&f)[4]) {
+    const uint2 v = *reinterpret_cast<const uint2*>(p);
+    f[0] = __uint_as_float(v.x << 16); f[1] = __uint_as_float(v.x & 0xffff0000u);
+    f[2] = __uint_as_float(v.y << 16); f[3] = __uint_as_float(v.y & 0xffff0000u);
+}
+
+// Queries, keys and values as the run kernels read them, a CTA per token: heads d_pad (v_pad) wide with zeros behind them,
+// activated and turned, q and k in `parts` bfloat16 numbers each.  Angles once per token.
+struct PrepareRows {
+    __nv_bfloat16* qk[2][2];    // [q or k][hi or lo], rows of heads * d_pad; null: left as they are
+    __nv_bfloat16* v;           // rows of heads * v_pad, or null
+    int d_pad, v_pad;
+};
+
+__global__ void __launch_bounds__(128)
+fixed_decay_prepare_kernel(FixedDecayArgs a, PrepareRows p) {
+    extern __shared__ float turn[];      // [pairs] cos, [pairs] sin
+    const int t = blockIdx.x;
+    pdl_launch_dependents();
+    if (a.pairs > 0) {
+        const float pos = (float)a.positions[t];
+        for (int i = threadIdx.x; i < a.pairs; i += 128) sincosf(pos * a.inv_freq[i], &turn[a.pairs + i], &turn[i]);
+        __syncthreads();
     }
-    const size_t t = (size_t)first + r;
-    const __nv_bfloat16* x = src + t * ld_src + (size_t)h * a.d_k;
-    const float f = scale * (factor ? factor[r] : 1.f);
-    const float2* ang = a.angles + t;
-    const size_t T = (size_t)a.n_tokens;
-    const bool vec = a.d_k % 8 == 0 && a.pairs % 8 == 0 && ld_src % 8 == 0 && ((uintptr_t)src & 15) == 0;
-    if (vec) {
-        for (int c = part * 8; c < a.pairs; c += 16) {
-            float u[8], v[8];
-            load8(x + c, u);
-            load8(x + a.pairs + c, v);
+    pdl_wait();
+    if (p.qk[0][0] != nullptr) {
+        const bool vec = a.d_k % 4 == 0 && a.pairs % 4 == 0 && a.ld_q % 4 == 0 && a.ld_k % 4 == 0 && (((uintptr_t)a.q | (uintptr_t)a.k) & 7) == 0;
+        const int chunks = p.d_pad / 4, units = 2 * a.heads * chunks;      // four neighbouring numbers of a head
+        for (int u = threadIdx.x; u < units; u += 128) {
+            const int which = u / (a.heads * chunks), h = (u / chunks) % a.heads, c = (u % chunks) * 4;
+            const __nv_bfloat16* x = (which ? (const __nv_bfloat16*)a.k + (size_t)t * a.ld_k : (const __nv_bfloat16*)a.q + (size_t)t * a.ld_q) +
+                                     (size_t)h * a.d_k;
+            float y[4];
+            if (vec) {      // (the four numbers, and their partners, lie side by side)
+                const bool first = c < a.pairs, turned = c < 2 * a.pairs;
+                const int o = !turned ? c : first ? c + a.pairs : c - a.pairs, f = first ? c : o;
+                float z[4] = {0.f, 0.f, 0.f, 0.f}, zo[4] = {0.f, 0.f, 0.f, 0.f};
+                if (c < a.d_k) {
+                    load4(x + c, z);
+                    if (turned) load4(x + o, zo);
+                }
 #pragma unroll
-            for (int e = 0; e < 8; ++e) {
-                if (a.qk_silu) { u[e] = silu_32(u[e]); v[e] = silu_32(v[e]); }
-                const float2 cs = ang[(size_t)(c + e) * T];
-                const float p = u[e] * cs.x - v[e] * cs.y, q = v[e] * cs.x + u[e] * cs.y;
-                u[e] = p * f;
-                v[e] = q * f;
+                for (int e = 0; e < 4; ++e) {
+                    if (a.qk_silu) { z[e] = silu_32(z[e]); zo[e] = silu_32(zo[e]); }
+                    y[e] = !turned ? z[e] : z[e] * turn[f + e] + (first ? -zo[e] : zo[e]) * turn[a.pairs + f + e];
+                }
+            } else
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const int i = c + e;
+                float z = i < a.d_k ? __bfloat162float(x[i]) : 0.f;
+                if (a.qk_silu) z = silu_32(z);
+                if (i < 2 * a.pairs) {
+                    const bool first = i < a.pairs;
+                    const int o = first ? i + a.pairs : i - a.pairs, f = first ? i : o;
+                    float zo = __bfloat162float(x[o]);
+                    if (a.qk_silu) zo = silu_32(zo);
+                    z = first ? z * turn[f] - zo * turn[a.pairs + f] : z * turn[f] + zo * turn[a.pairs + f];
+                }
+                y[e] = z;
             }
-            split_store8(hr + c, lr + c, u);
-            split_store8(hr + a.pairs + c, lr + a.pairs + c, v);
-        }
-        for (int c = 2 * a.pairs + part * 8; c < a.d_k; c += 16) {
-            float u[8];
-            load8(x + c, u);
-#pragma unroll
-            for (int e = 0; e < 8; ++e) u[e] = (a.qk_silu ? silu_32(u[e]) : u[e]) * f;
-            split_store8(hr + c, lr + c, u);
-        }
-    } else {
-        for (int c = part; c < a.pairs; c += 2) {
-            float u = __bfloat162float(x[c]), v = __bfloat162float(x[c + a.pairs]);
-            if (a.qk_silu) { u = silu_32(u); v = silu_32(v); }
-            const float2 cs = ang[(size_t)c * T];
-            split_store(hr + c, lr + c, (u * cs.x - v * cs.y) * f);
-            split_store(hr + c + a.pairs, lr + c + a.pairs, (v * cs.x + u * cs.y) * f);
-        }
-        for (int c = 2 * a.pairs + part; c < a.d_k; c += 2) {
-            const float u = __bfloat162float(x[c]);
-            split_store(hr + c, lr + c, (a.qk_silu ? silu_32(u) : u) * f);
+            const size_t at = ((size_t)t * a.heads + h) * p.d_pad + c;
+            uint32_t hi[2], lo[2];
+            split_pair(y[0], y[1], hi[0], lo[0]);
+            split_pair(y[2], y[3], hi[1], lo[1]);
+            *reinterpret_cast<uint2*>(p.qk[which][0] + at) = make_uint2(hi[0], hi[1]);
+            if (p.qk[which][1] != nullptr) *reinterpret_cast<uint2*>(p.qk[which][1] + at) = make_uint2(lo[0], lo[1]);
         }
     }
-    for (int c = a.d_k + part; c < d_pad; c += 2) {
-        hr[c] = __float2bfloat16_rn(0.f);
-        lr[c] = __float2bfloat16_rn(0.f);
+    if (p.v != nullptr) {
+        const __nv_bfloat16* x = (const __nv_bfloat16*)a.v + (size_t)t * a.ld_v;
+        for (int u = threadIdx.x; u < a.heads * p.v_pad; u += 128) {
+            const int h = u / p.v_pad, c = u % p.v_pad;
+            const float z = c < a.d_v ? __bfloat162float(x[(size_t)h * a.d_v + c]) : 0.f;
+            p.v[(size_t)t * a.heads * p.v_pad + u] = __float2bfloat16_rn(a.v_silu ? silu_32(z) : z);
+        }
     }
 }
 
-// columns col0 .. col0 + NS of the run's values as one tile [kRun][ld]
-template <int NS>
-__device__ __forceinline__ void load_values(const FixedDecayArgs& a, int first, int n, int h, int col0, __nv_bfloat16* dst, int ld) {
-    const __nv_bfloat16* src = (const __nv_bfloat16*)a.v;
-    const bool vec = a.d_v % 8 == 0 && a.ld_v % 8 == 0 && ((uintptr_t)src & 15) == 0;
-    for (int i = threadIdx.x; i < kRun * (NS / 8); i += kRunThreads) {
-        const int r = i / (NS / 8), c = (i % (NS / 8)) * 8;
-        __nv_bfloat16* o = dst + (size_t)r * ld + c;
-        const __nv_bfloat16* x = src + ((size_t)first + r) * a.ld_v + (size_t)h * a.d_v + col0 + c;
-        if (r >= n || col0 + c >= a.d_v) {
-            *reinterpret_cast<uint4*>(o) = make_uint4(0, 0, 0, 0);
-        } else if (vec) {
-            if (a.v_silu) {
-                float f[8];
-                load8(x, f);
-                *reinterpret_cast<uint4*>(o) = make_uint4(pack_pair(silu_32(f[0]), silu_32(f[1])), pack_pair(silu_32(f[2]), silu_32(f[3])),
-                                                         pack_pair(silu_32(f[4]), silu_32(f[5])), pack_pair(silu_32(f[6]), silu_32(f[7])));
-            } else {
-                *reinterpret_cast<uint4*>(o) = *reinterpret_cast<const uint4*>(x);
-            }
-        } else {
-            for (int e = 0; e < 8; ++e) {
-                const float f = col0 + c + e < a.d_v ? __bfloat162float(x[e]) : 0.f;
-                o[e] = __float2bfloat16_rn(a.v_silu ? silu_32(f) : f);
-            }
-        }
+__device__ __forceinline__ void copy_16(__nv_bfloat16* dst, const __nv_bfloat16* src, bool take) {
+    const int n = take ? 16 : 0;      // (0: zeros are written)
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src), "r"(n) : "memory");
+}
+__device__ __forceinline__ void copies_done() {
+    asm volatile("cp.async.commit_group;\ncp.async.wait_group 0;" ::: "memory");
+}
+
+// columns 0 .. width of a run's rows as a tile [kRun][ld] (rows beyond the run and columns beyond `limit` zero)
+__device__ __forceinline__ void load_tile(__nv_bfloat16* dst, int ld, const __nv_bfloat16* src, int ld_src, int n, int width, int limit) {
+    const int per_row = width / 8;
+    for (int i = threadIdx.x; i < kRun * per_row; i += kRunThreads) {
+        const int r = i / per_row, c = (i % per_row) * 8;
+        const bool take = r < n && c < limit;
+        copy_16(dst + (size_t)r * ld + c, take ? src + (size_t)r * ld_src + c : src, take);
     }
 }
 
@@ -310,7 +309,7 @@ __device__ __forceinline__ void powers(float* pw, float g) {
 }
 
 // (1) U[d_k, columns] = sum_j g^(n - 1 - j) k_j v_j^T of one run
-template <int NS>
+template <int NS, int PARTS>
 __global__ void __launch_bounds__(kRunThreads)
 fixed_decay_run_sums_kernel(FixedDecayArgs a) {
     extern __shared__ __align__(16) uint8_t run_smem[];
@@ -322,16 +321,36 @@ fixed_decay_run_sums_kernel(FixedDecayArgs a) {
     __nv_bfloat16* khi = reinterpret_cast<__nv_bfloat16*>(run_smem);
     __nv_bfloat16* klo = khi + kRun * ld;
     __nv_bfloat16* vs = klo + kRun * ld;
-    __shared__ float pw[kRun + 1], factor[kRun];
+    __shared__ float pw[kRun + 1];
     powers(pw, a.decay[h]);
-    __syncthreads();
     const int first = seq0 + run * kRun, n = min(kRun, q_len - run * kRun);
-    if (threadIdx.x < kRun) factor[threadIdx.x] = (int)threadIdx.x < n ? pw[n - 1 - threadIdx.x] : 0.f;
     __syncthreads();
     pdl_wait();
     if (n <= 0) return;
-    load_rows_split(a, (const __nv_bfloat16*)a.k, a.ld_k, first, n, h, khi, klo, ld, d_pad, 1.f, factor);
-    load_values<NS>(a, first, n, h, col0, vs, ldv);
+    load_tile(vs, ldv, a.vt + (size_t)first * a.ld_vt + (size_t)h * a.head_v + col0, a.ld_vt, n, NS, (a.d_v - col0 + 7) / 8 * 8);
+    // the keys times the decay until the run's end, in two parts again
+    const int per_row = d_pad / 8;
+    for (int i = threadIdx.x; i < kRun * per_row; i += kRunThreads) {
+        const int r = i / per_row, c = (i % per_row) * 8;
+        uint32_t hi[4] = {0, 0, 0, 0}, lo[4] = {0, 0, 0, 0};
+        if (r < n) {
+            const float f = pw[n - 1 - r];
+            const size_t at = (size_t)(first + r) * a.ld_kt + (size_t)h * a.head_qk + c;
+            float x[8];
+            load8(a.kt[0] + at, x);
+            if constexpr (PARTS == 2) {
+                float y[8];
+                load8(a.kt[1] + at, y);
+#pragma unroll
+                for (int e = 0; e < 8; ++e) x[e] += y[e];
+            }
+#pragma unroll
+            for (int e = 0; e < 4; ++e) split_pair(x[2 * e] * f, x[2 * e + 1] * f, hi[e], lo[e]);
+        }
+        *reinterpret_cast<uint4*>(khi + (size_t)r * ld + c) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+        *reinterpret_cast<uint4*>(klo + (size_t)r * ld + c) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+    }
+    copies_done();
     __syncthreads();
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, mi = lane >> 3, mr = lane & 7, gq = lane >> 2, tq = lane & 3;
     float* U = a.runs + ((size_t)(first_run(a.cu_seqlens, seq) + run) * a.heads + h) * a.d_k * a.d_v;
@@ -377,8 +396,8 @@ fixed_decay_run_sums_kernel(FixedDecayArgs a) {
     }
 }
 
-// (2) per element, run after run: the scratch's run sum is replaced by the state before the run; the state after the last
-// run goes back to the slot.  Eight runs' sums are asked for at once.
+// (2) per element, run after run: the scratch's run sum is replaced by the state before the run, as its hi and lo part; the
+// state after the last run goes back to the slot.  Sixteen runs' sums are asked for at once.
 __global__ void __launch_bounds__(256)
 fixed_decay_carry_kernel(FixedDecayArgs a) {
     const int h = blockIdx.y, seq = blockIdx.z;
@@ -393,14 +412,16 @@ fixed_decay_carry_kernel(FixedDecayArgs a) {
     float carry = *S;
     const size_t step = (size_t)a.heads * per_head;
     float* u = a.runs + ((size_t)first_run(a.cu_seqlens, seq) * a.heads + h) * per_head + e;
-    for (int r0 = 0; r0 < n_runs; r0 += 8) {
-        float x[8];
+    for (int r0 = 0; r0 < n_runs; r0 += 16) {
+        float x[16];
 #pragma unroll
-        for (int i = 0; i < 8; ++i) x[i] = r0 + i < n_runs ? u[(size_t)(r0 + i) * step] : 0.f;
+        for (int i = 0; i < 16; ++i) x[i] = r0 + i < n_runs ? u[(size_t)(r0 + i) * step] : 0.f;
 #pragma unroll
-        for (int i = 0; i < 8; ++i) {
+        for (int i = 0; i < 16; ++i) {
             if (r0 + i < n_runs) {
-                u[(size_t)(r0 + i) * step] = carry;
+                const __nv_bfloat16 hi = __float2bfloat16_rn(carry);
+                const __nv_bfloat162 both = __halves2bfloat162(hi, __float2bfloat16_rn(carry - __bfloat162float(hi)));
+                u[(size_t)(r0 + i) * step] = __uint_as_float(*reinterpret_cast<const uint32_t*>(&both));
                 carry = (r0 + i == n_runs - 1 ? g_last : g_run) * carry + x[i];
             }
         }
@@ -409,7 +430,7 @@ fixed_decay_carry_kernel(FixedDecayArgs a) {
 }
 
 // (3) outputs of one run
-template <int NS>
+template <int NS, int PARTS>
 __global__ void __launch_bounds__(kRunThreads)
 fixed_decay_outputs_kernel(FixedDecayArgs a) {
     extern __shared__ __align__(16) uint8_t run_smem[];
@@ -418,11 +439,9 @@ fixed_decay_outputs_kernel(FixedDecayArgs a) {
     const int seq0 = a.cu_seqlens[seq], q_len = a.cu_seqlens[seq + 1] - seq0;
     pdl_launch_dependents();
     const int d_pad = (a.d_k + 15) / 16 * 16, ld = d_pad + 8, ldv = NS + 8;
-    __nv_bfloat16* qhi = reinterpret_cast<__nv_bfloat16*>(run_smem);
-    __nv_bfloat16* qlo = qhi + kRun * ld;
-    __nv_bfloat16* khi = qlo + kRun * ld;
-    __nv_bfloat16* klo = khi + kRun * ld;
-    __nv_bfloat16* vs = klo + kRun * ld;
+    __nv_bfloat16* qs = reinterpret_cast<__nv_bfloat16*>(run_smem);      // PARTS tiles
+    __nv_bfloat16* ks = qs + PARTS * kRun * ld;
+    __nv_bfloat16* vs = ks + PARTS * kRun * ld;
     __nv_bfloat16* shi = vs + kRun * ldv;
     __nv_bfloat16* slo = shi + d_pad * ldv;
     __shared__ float pw[kRun + 1];
@@ -430,26 +449,32 @@ fixed_decay_outputs_kernel(FixedDecayArgs a) {
     const int first = seq0 + run * kRun, n = min(kRun, q_len - run * kRun);
     pdl_wait();
     if (n <= 0) return;
-    load_rows_split(a, (const __nv_bfloat16*)a.q, a.ld_q, first, n, h, qhi, qlo, ld, d_pad, a.q_scale, nullptr);
-    load_rows_split(a, (const __nv_bfloat16*)a.k, a.ld_k, first, n, h, khi, klo, ld, d_pad, 1.f, nullptr);
-    load_values<NS>(a, first, n, h, col0, vs, ldv);
-    {   // the state before the run: 8 numbers per thread and access where the rows allow it
-        const float* S = a.runs + ((size_t)(first_run(a.cu_seqlens, seq) + run) * a.heads + h) * a.d_k * a.d_v;
-        const bool vec = a.d_v % 8 == 0 && ((uintptr_t)a.runs & 15) == 0;
-        for (int i = threadIdx.x; i < d_pad * (NS / 8); i += kRunThreads) {
-            const int r = i / (NS / 8), c = (i % (NS / 8)) * 8;
-            float x[8];
-            if (r < a.d_k && col0 + c + 8 <= a.d_v && vec) {
-                const float4* p = reinterpret_cast<const float4*>(S + (size_t)r * a.d_v + col0 + c);
-                const float4 u = p[0], v = p[1];
-                x[0] = u.x; x[1] = u.y; x[2] = u.z; x[3] = u.w; x[4] = v.x; x[5] = v.y; x[6] = v.z; x[7] = v.w;
-            } else {
 #pragma unroll
-                for (int e = 0; e < 8; ++e) x[e] = (r < a.d_k && col0 + c + e < a.d_v) ? S[(size_t)r * a.d_v + col0 + c + e] : 0.f;
+    for (int p = 0; p < PARTS; ++p) {
+        load_tile(qs + p * kRun * ld, ld, a.qt[p] + (size_t)first * a.ld_qt + (size_t)h * a.head_qk, a.ld_qt, n, d_pad, d_pad);
+        load_tile(ks + p * kRun * ld, ld, a.kt[p] + (size_t)first * a.ld_kt + (size_t)h * a.head_qk, a.ld_kt, n, d_pad, d_pad);
+    }
+    load_tile(vs, ldv, a.vt + (size_t)first * a.ld_vt + (size_t)h * a.head_v + col0, a.ld_vt, n, NS, (a.d_v - col0 + 7) / 8 * 8);
+    {   // the state before the run, (hi, lo) pairs: four numbers per thread and access where the rows allow it
+        const uint32_t* S = reinterpret_cast<const uint32_t*>(a.runs) + ((size_t)(first_run(a.cu_seqlens, seq) + run) * a.heads + h) * a.d_k * a.d_v;
+        const bool vec = a.d_v % 4 == 0;
+        for (int i = threadIdx.x; i < d_pad * (NS / 4); i += kRunThreads) {
+            const int r = i / (NS / 4), c = (i % (NS / 4)) * 4;
+            uint32_t w[4] = {0, 0, 0, 0};
+            if (r < a.d_k && col0 + c < a.d_v) {
+                if (vec) {
+                    const uint4 x = *reinterpret_cast<const uint4*>(S + (size_t)r * a.d_v + col0 + c);
+                    w[0] = x.x; w[1] = x.y; w[2] = x.z; w[3] = x.w;
+                } else {
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) w[e] = col0 + c + e < a.d_v ? S[(size_t)r * a.d_v + col0 + c + e] : 0u;
+                }
             }
-            split_store8(shi + (size_t)r * ldv + c, slo + (size_t)r * ldv + c, x);
+            *reinterpret_cast<uint2*>(shi + (size_t)r * ldv + c) = make_uint2(__byte_perm(w[0], w[1], 0x5410), __byte_perm(w[2], w[3], 0x5410));
+            *reinterpret_cast<uint2*>(slo + (size_t)r * ldv + c) = make_uint2(__byte_perm(w[0], w[1], 0x7632), __byte_perm(w[2], w[3], 0x7632));
         }
     }
+    copies_done();
     __syncthreads();
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, mi = lane >> 3, mr = lane & 7, gq = lane >> 2, tq = lane & 3;
     const int row0 = warp * 16;
@@ -467,21 +492,23 @@ fixed_decay_outputs_kernel(FixedDecayArgs a) {
     for (int kk = 0; kk < d_pad / 16; ++kk) {
         uint32_t ah[4], al[4];
         const int at = (row0 + (mi & 1) * 8 + mr) * ld + kk * 16 + (mi >> 1) * 8;
-        ldsm4(ah, qhi + at);
-        ldsm4(al, qlo + at);
+        ldsm4(ah, qs + at);
+        if constexpr (PARTS == 2) ldsm4(al, qs + kRun * ld + at);
 #pragma unroll
         for (int j = 0; j < kRun / 16; ++j) {
             if (j <= warp) {
                 uint32_t bh[4], bl[4];
                 const int bt = (j * 16 + (mi >> 1) * 8 + mr) * ld + kk * 16 + (mi & 1) * 8;
-                ldsm4(bh, khi + bt);
-                ldsm4(bl, klo + bt);
+                ldsm4(bh, ks + bt);
                 mma_run(sc[2 * j], ah, bh[0], bh[1]);
-                mma_run(sc[2 * j], ah, bl[0], bl[1]);
-                mma_run(sc[2 * j], al, bh[0], bh[1]);
                 mma_run(sc[2 * j + 1], ah, bh[2], bh[3]);
-                mma_run(sc[2 * j + 1], ah, bl[2], bl[3]);
-                mma_run(sc[2 * j + 1], al, bh[2], bh[3]);
+                if constexpr (PARTS == 2) {
+                    ldsm4(bl, ks + kRun * ld + bt);
+                    mma_run(sc[2 * j], ah, bl[0], bl[1]);
+                    mma_run(sc[2 * j + 1], ah, bl[2], bl[3]);
+                    mma_run(sc[2 * j], al, bh[0], bh[1]);
+                    mma_run(sc[2 * j + 1], al, bh[2], bh[3]);
+                }
             }
         }
 #pragma unroll
@@ -491,11 +518,13 @@ fixed_decay_outputs_kernel(FixedDecayArgs a) {
             ldsm4t(bh, shi + bt);
             ldsm4t(bl, slo + bt);
             mma_run(o[2 * j], ah, bh[0], bh[1]);
-            mma_run(o[2 * j], ah, bl[0], bl[1]);
-            mma_run(o[2 * j], al, bh[0], bh[1]);
             mma_run(o[2 * j + 1], ah, bh[2], bh[3]);
+            mma_run(o[2 * j], ah, bl[0], bl[1]);
             mma_run(o[2 * j + 1], ah, bl[2], bl[3]);
-            mma_run(o[2 * j + 1], al, bh[2], bh[3]);
+            if constexpr (PARTS == 2) {
+                mma_run(o[2 * j], al, bh[0], bh[1]);
+                mma_run(o[2 * j + 1], al, bh[2], bh[3]);
+            }
         }
     }
     const int i0 = row0 + gq, i1 = i0 + 8;
@@ -535,6 +564,10 @@ fixed_decay_outputs_kernel(FixedDecayArgs a) {
             mma_run(o[2 * jj + 1], al, b[2], b[3]);
         }
     }
+#pragma unroll
+    for (int j = 0; j < NS / 8; ++j)
+#pragma unroll
+        for (int i = 0; i < 4; ++i) o[j][i] *= a.q_scale;
 #pragma unroll
     for (int hh = 0; hh < 2; ++hh) {
         const int i = hh ? i1 : i0;
@@ -581,9 +614,9 @@ fixed_decay_outputs_kernel(FixedDecayArgs a) {
     }
 }
 
-static size_t outputs_smem(int d_k, int ns) {
+static size_t outputs_smem(int d_k, int ns, int parts) {
     const int d_pad = (d_k + 15) / 16 * 16;
-    return sizeof(__nv_bfloat16) * ((size_t)4 * kRun * (d_pad + 8) + (size_t)kRun * (ns + 8) + (size_t)2 * d_pad * (ns + 8));
+    return sizeof(__nv_bfloat16) * ((size_t)2 * parts * kRun * (d_pad + 8) + (size_t)kRun * (ns + 8) + (size_t)2 * d_pad * (ns + 8));
 }
 static size_t sums_smem(int d_k, int ns) {
     const int d_pad = (d_k + 15) / 16 * 16;
@@ -593,31 +626,42 @@ constexpr size_t kMostSmem = 227 * 1024 - 1024;    // (a kilobyte for the static
 
 // columns of the values a CTA takes: all of a head's up to 128 where shared memory allows, else slices of 64; 0: no fit
 static int run_columns(int d_k, int d_v) {
-    if (d_v > 64 && outputs_smem(d_k, 128) <= kMostSmem) return 128;
-    return outputs_smem(d_k, 64) <= kMostSmem ? 64 : 0;
+    if (d_v > 64 && outputs_smem(d_k, 128, 2) <= kMostSmem) return 128;
+    return outputs_smem(d_k, 64, 2) <= kMostSmem ? 64 : 0;
 }
 
-template <int NS>
+template <int NS, int PARTS>
 static int launch_runs(const FixedDecayArgs& a, int n_seqs, int max_q_len, cudaStream_t stream) {
-    const size_t s1 = sums_smem(a.d_k, NS), s3 = outputs_smem(a.d_k, NS);
+    const size_t s1 = sums_smem(a.d_k, NS), s3 = outputs_smem(a.d_k, NS, PARTS);
     static size_t have1 = 48 * 1024, have3 = 48 * 1024;
     if (s1 > have1) {
-        const int e = (int)cudaFuncSetAttribute(fixed_decay_run_sums_kernel<NS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s1);
+        const int e = (int)cudaFuncSetAttribute(fixed_decay_run_sums_kernel<NS, PARTS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s1);
         if (e != 0) return e;
         have1 = s1;
     }
     if (s3 > have3) {
-        const int e = (int)cudaFuncSetAttribute(fixed_decay_outputs_kernel<NS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s3);
+        const int e = (int)cudaFuncSetAttribute(fixed_decay_outputs_kernel<NS, PARTS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s3);
         if (e != 0) return e;
         have3 = s3;
     }
     const int n_runs = (max_q_len + kRun - 1) / kRun, slices = (a.d_v + NS - 1) / NS;
     const dim3 grid(n_runs * slices, a.heads, n_seqs);
-    int st = launch_pdl(fixed_decay_run_sums_kernel<NS>, grid, dim3(kRunThreads), s1, stream, a);
+    int st = launch_pdl(fixed_decay_run_sums_kernel<NS, PARTS>, grid, dim3(kRunThreads), s1, stream, a);
     if (st != 0) return st;
     st = launch_pdl(fixed_decay_carry_kernel, dim3((a.d_k * a.d_v + 255) / 256, a.heads, n_seqs), dim3(256), 0, stream, a);
     if (st != 0) return st;
-    return launch_pdl(fixed_decay_outputs_kernel<NS>, grid, dim3(kRunThreads), s3, stream, a);
+    return launch_pdl(fixed_decay_outputs_kernel<NS, PARTS>, grid, dim3(kRunThreads), s3, stream, a);
+}
+
+// Whether queries and keys, and values, can be read as they lie, or a kernel has to leave them on the run kernels' grid first.
+static bool qk_ready(const FixedDecayArgs& a) {
+    return !a.qk_silu && a.pairs == 0 && a.d_k % 16 == 0 && a.ld_q % 8 == 0 && a.ld_k % 8 == 0 && (((uintptr_t)a.q | (uintptr_t)a.k) & 15) == 0;
+}
+static bool v_ready(const FixedDecayArgs& a) {
+    return !a.v_silu && a.d_v % 8 == 0 && a.ld_v % 8 == 0 && ((uintptr_t)a.v & 15) == 0;
+}
+static size_t run_floats(int n_tokens, int n_seqs, int heads, int d_k, int d_v) {   // of the runs' sums, to a multiple of 4
+    return (((size_t)(n_tokens / kRun + n_seqs + 1) * heads * d_k * d_v) + 3) / 4 * 4;
 }
 
 template <typename T, int VEC, int TPR>
@@ -634,15 +678,18 @@ static int launch_step(const FixedDecayArgs& a, cudaStream_t stream) {
 // they, or the one-token kernel, can finish a head (all its values in one CTA).
 extern "C" int b200_fixed_decay_columns(int d_k, int d_v) { return b200::run_columns(d_k, d_v); }
 extern "C" int b200_fixed_decay_step_finishes(int d_v) { return d_v % 4 == 0 ? d_v <= 128 : d_v <= 32; }
-// Runs the scratch of the prompt kernels has room for: n_runs * heads * d_k * d_v floats.
-extern "C" int b200_fixed_decay_runs(int n_tokens, int n_seqs) { return n_tokens / b200::kRun + n_seqs + 1; }
+// Floats of scratch the prompt kernels need: the runs' sums, then queries, keys and values in the run kernels' layout.
+extern "C" long long b200_fixed_decay_scratch(int n_tokens, int n_seqs, int heads, int d_k, int d_v) {
+    const long long d_pad = (d_k + 15) / 16 * 16, v_pad = (d_v + 7) / 8 * 8;
+    return (long long)b200::run_floats(n_tokens, n_seqs, heads, d_k, d_v) + ((4 * d_pad + v_pad) * n_tokens * heads + 1) / 2;
+}
 
 // The recurrence over a packed step (see the head of this file).  n_tokens == n_seqs: one token per sequence, operands of
-// either type; otherwise bfloat16 operands, `scratch` as b200_fixed_decay_runs says and `angles` [pairs][T] (cos, sin).
+// either type; otherwise bfloat16 operands and `scratch` as b200_fixed_decay_scratch says.
 // out: float32 [T, heads d_v], or rows (not null): the finished heads, o / rms(o) * act(gate) * mul, into [T, ld_rows].
 extern "C" int b200_fixed_decay(const void* q, int ld_q, const void* k, int ld_k, const void* v, int ld_v, const float* decay,
                                 float* state, long long slot_stride, const int* slots, const int* cu_seqlens, const int* positions,
-                                const float* inv_freq, const float* angles, int pairs, float* out, float* scratch, int dtype,
+                                const float* inv_freq, int pairs, float* out, float* scratch, int dtype,
                                 int n_tokens, int n_seqs, int max_q_len, int heads, int d_k, int d_v, float q_scale, int qk_silu,
                                 int v_silu, const void* gate, int ld_gate, int gate_act, void* rows, int ld_rows, float eps, float mul,
                                 cudaStream_t stream) {
@@ -652,11 +699,14 @@ extern "C" int b200_fixed_decay(const void* q, int ld_q, const void* k, int ld_k
         return kErrBadArgument;
     if ((rows == nullptr) == (out == nullptr) || (rows != nullptr && (!gate || ld_rows < heads * d_v || ld_gate < heads * d_v)))
         return kErrBadArgument;
-    FixedDecayArgs a = {q, k, v, ld_q, ld_k, ld_v, decay, state, (size_t)slot_stride, slots, cu_seqlens, inv_freq, positions,
-                        (const float2*)angles, out, scratch, n_tokens, heads, d_k, d_v, pairs, qk_silu, v_silu, q_scale, gate, ld_gate,
-                        gate_act, rows, ld_rows, eps, mul};
+    if (pairs > 0 && (!inv_freq || !positions)) return kErrBadArgument;
+    FixedDecayArgs a = {};
+    a.q = q; a.k = k; a.v = v; a.ld_q = ld_q; a.ld_k = ld_k; a.ld_v = ld_v;
+    a.decay = decay; a.state = state; a.slot_stride = (size_t)slot_stride; a.slots = slots; a.cu_seqlens = cu_seqlens;
+    a.inv_freq = inv_freq; a.positions = positions; a.out = out; a.runs = scratch;
+    a.n_tokens = n_tokens; a.heads = heads; a.d_k = d_k; a.d_v = d_v; a.pairs = pairs; a.qk_silu = qk_silu; a.v_silu = v_silu;
+    a.q_scale = q_scale; a.gate = gate; a.ld_gate = ld_gate; a.gate_act = gate_act; a.rows = rows; a.ld_rows = ld_rows; a.eps = eps; a.mul = mul;
     if (n_tokens == n_seqs) {
-        if (pairs > 0 && (!inv_freq || !positions)) return kErrBadArgument;
         if (rows != nullptr && !b200_fixed_decay_step_finishes(d_v)) return kErrUnsupportedSize;
         const bool vec = d_v % 4 == 0 && slot_stride % 4 == 0 && ((uintptr_t)state & 15) == 0;
         if (rows != nullptr && !vec && d_v > 32) return kErrUnsupportedSize;
@@ -670,6 +720,33 @@ extern "C" int b200_fixed_decay(const void* q, int ld_q, const void* k, int ld_k
     const int ns = run_columns(d_k, d_v);
     if (ns == 0) return kErrUnsupportedSize;
     if (rows != nullptr && d_v > ns) return kErrUnsupportedSize;
-    if (!scratch || ((uintptr_t)scratch & 15) || (pairs > 0 && !angles)) return kErrBadArgument;
-    return ns == 128 ? launch_runs<128>(a, n_seqs, max_q_len, stream) : launch_runs<64>(a, n_seqs, max_q_len, stream);
+    if (!scratch || ((uintptr_t)scratch & 15)) return kErrBadArgument;
+    // queries and keys have two parts where they are turned (32-bit numbers), one where they are projections
+    const int parts = pairs > 0 ? 2 : 1;
+    PrepareRows prep = {};
+    prep.d_pad = (d_k + 15) / 16 * 16;
+    prep.v_pad = (d_v + 7) / 8 * 8;
+    __nv_bfloat16* room = reinterpret_cast<__nv_bfloat16*>(scratch + run_floats(n_tokens, n_seqs, heads, d_k, d_v));
+    const size_t qk_size = (size_t)n_tokens * heads * prep.d_pad;
+    a.qt[0] = (const __nv_bfloat16*)q; a.kt[0] = (const __nv_bfloat16*)k; a.vt = (const __nv_bfloat16*)v;
+    a.ld_qt = ld_q; a.ld_kt = ld_k; a.ld_vt = ld_v; a.head_qk = d_k; a.head_v = d_v;
+    if (!qk_ready(a)) {
+        for (int w = 0; w < 2; ++w)
+            for (int p = 0; p < parts; ++p) prep.qk[w][p] = room + (size_t)(2 * w + p) * qk_size;
+        for (int p = 0; p < parts; ++p) { a.qt[p] = prep.qk[0][p]; a.kt[p] = prep.qk[1][p]; }
+        a.ld_qt = a.ld_kt = heads * prep.d_pad;
+        a.head_qk = prep.d_pad;
+    }
+    if (!v_ready(a)) {
+        prep.v = room + 4 * qk_size;
+        a.vt = prep.v;
+        a.ld_vt = heads * prep.v_pad;
+        a.head_v = prep.v_pad;
+    }
+    if (prep.qk[0][0] != nullptr || prep.v != nullptr) {
+        const int st = launch_pdl(fixed_decay_prepare_kernel, dim3(n_tokens), dim3(128), sizeof(float) * 2 * pairs, stream, a, prep);
+        if (st != 0) return st;
+    }
+    if (ns == 128) return parts == 2 ? launch_runs<128, 2>(a, n_seqs, max_q_len, stream) : launch_runs<128, 1>(a, n_seqs, max_q_len, stream);
+    return parts == 2 ? launch_runs<64, 2>(a, n_seqs, max_q_len, stream) : launch_runs<64, 1>(a, n_seqs, max_q_len, stream);
 }

@@ -26,7 +26,8 @@
 // of squares: the completing product then writes two copies, bfloat16(x * w) and bfloat16(x * w2).
 //
 // A bias (float32 [N], one number per output) joins every sum before the epilogue: before the activation of the gated
-// ones, once per element of the residual add.  It is a weight: it is fetched before the dependency wait.
+// ones, once per element of the residual add.  It is a weight: it is fetched before the dependency wait.  The store epilogue
+// may pass its first `silu_cols` columns through SiLU (projections that are used activated).
 #include "common.cuh"
 
 namespace b200 {
@@ -67,6 +68,7 @@ struct NormLink {
     const void* out_weight2;    // [N] weights of a second norm of the same rows (of out_weight's type), or null
     __nv_bfloat16* out_act2;    // [M][ld_out_act]
     const float* bias;          // [N] or null
+    int silu_cols;              // epilogue 0: columns below this one are stored as silu(sum)
     // the gated epilogue's activation of the gate value: 0 SiLU, 1 GELU in its tanh form, 2 the clamped form
     // min(g, limit) sigmoid(slope min(g, limit)) (clamp(u, -limit, limit) + 1)
     int gate_act;
@@ -224,7 +226,7 @@ gemm_decode_kernel(const __nv_bfloat16* __restrict__ A, int lda, const __nv_bflo
                     square = x * x;
                 }
             } else {
-                *c = from_f32<TC>(s);
+                *c = from_f32<TC>(row0 + row < link.silu_cols ? s / (1.0f + expf(-s)) : s);
             }
         }
         if (LINK && EPI == 1 && NT <= 2 && link.out_weight != nullptr) {
@@ -347,9 +349,10 @@ static int gemm_decode_launch(const void* A, int lda, const void* W, int ldw, vo
 // 3 gated GELU (tanh form), 4 gated and clamped (gate_limit, gate_slope).  bias: float32 [N] or null.
 extern "C" int b200_gemm_decode(const void* A, int lda, const void* W, int ldw, void* C, int c_dtype, int ldc, int M,
                                 int N, int K, int epilogue, float gate_limit, float gate_slope, const float* bias,
-                                cudaStream_t stream) {
+                                int silu_cols, cudaStream_t stream) {
     b200::NormLink link{};
     link.bias = bias;
+    link.silu_cols = silu_cols;
     link.gate_limit = gate_limit;
     link.gate_slope = gate_slope;
     return b200::gemm_decode_launch(A, lda, W, ldw, C, c_dtype, ldc, M, N, K, epilogue, link, stream);
@@ -373,7 +376,7 @@ extern "C" int b200_gemm_decode_linked(const void* A, int lda, const void* W, in
                                        int N, int K, int epilogue, const float* in_partials, int n_in, float eps,
                                        int norm_dim, const void* out_weight, int out_weight_dtype, void* out_act,
                                        int ld_out_act, float* out_partials, const void* out_weight2, void* out_act2,
-                                       const float* bias, cudaStream_t stream) {
+                                       const float* bias, int silu_cols, cudaStream_t stream) {
     using namespace b200;
     if (M > 16) return kErrUnsupportedSize;
     if (in_partials != nullptr && (n_in <= 0 || norm_dim <= 0)) return kErrBadArgument;
@@ -383,6 +386,7 @@ extern "C" int b200_gemm_decode_linked(const void* A, int lda, const void* W, in
     if (out_weight2 != nullptr && (out_weight == nullptr || out_act2 == nullptr)) return kErrBadArgument;
     NormLink link{};
     link.bias = bias;
+    link.silu_cols = silu_cols;
     link.out_weight2 = out_weight2;
     link.out_act2 = (__nv_bfloat16*)out_act2;
     link.in_partials = in_partials;

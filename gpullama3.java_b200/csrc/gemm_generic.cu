@@ -13,7 +13,8 @@
 //   3  gated GELU    the same with gelu(g) = 0.5 g (1 + tanh(sqrt(2/pi) (g + 0.044715 g^3))), the tanh form
 //   4  gated, clamped  with g = min(acc[2j], limit), u = clamp(acc[2j+1], -limit, limit):
 //                    C[M, N/2] = g sigmoid(slope g) (u + 1); limit and slope are arguments
-// A bias (float32 [N]) joins every sum before the epilogue.
+// A bias (float32 [N]) joins every sum before the epilogue.  The store epilogue may pass its first `silu_cols` columns through
+// SiLU (projections that are used activated).
 #include "common.cuh"
 
 namespace b200 {
@@ -34,7 +35,9 @@ struct ProductExtras {
     long long a, w, c;
     float gate_limit, gate_slope;   // epilogue 4 alone reads these
     const float* bias;              // [N] or null
+    int silu_cols;                  // epilogue 0: columns below this one are stored as silu(sum)
 };
+__device__ __forceinline__ float stored(const ProductExtras& x, int n, float sum) { return n < x.silu_cols ? sum / (1.0f + expf(-sum)) : sum; }
 __device__ __forceinline__ float bias_of(const ProductExtras& x, int n) { return x.bias ? x.bias[n] : 0.f; }
 
 constexpr int kTileM = 64, kTileN = 64, kTileK = 16, kGemmThreads = 256;
@@ -98,7 +101,7 @@ gemm_generic_kernel(const TA* __restrict__ A, int lda, const TW* __restrict__ W,
                 TC* c = C + (size_t)m * ldc + n;
                 const float sum = acc[i][j] + bias_of(batch, n);
                 if (epilogue == 1) *c = from_f32<TC>(to_f32<TC>(*c) + sum);
-                else *c = from_f32<TC>(sum);
+                else *c = from_f32<TC>(stored(batch, n, sum));
             }
         }
     }
@@ -176,7 +179,7 @@ gemm_generic_big_kernel(const TA* __restrict__ A, int lda, const TW* __restrict_
                 TC* c = C + (size_t)m * ldc + n;
                 const float sum = acc[i][j] + bias_of(batch, n);
                 if (epilogue == 1) *c = from_f32<TC>(to_f32<TC>(*c) + sum);
-                else *c = from_f32<TC>(sum);
+                else *c = from_f32<TC>(stored(batch, n, sum));
             }
         }
     }
@@ -275,7 +278,7 @@ gemm_fewrows_kernel(const TA* __restrict__ A, int lda, const TW* __restrict__ W,
     } else if (m < M && n < N) {
         TC* c = C + (size_t)m * ldc + n;
         if (epilogue == 1) *c = from_f32<TC>(to_f32<TC>(*c) + sum);
-        else *c = from_f32<TC>(sum);
+        else *c = from_f32<TC>(stored(batch, n, sum));
     }
 }
 
@@ -323,9 +326,9 @@ static int gemm_generic_launch(const void* A, int a_dtype, int lda, const void* 
 
 extern "C" int b200_gemm_generic(const void* A, int a_dtype, int lda, const void* W, int w_dtype, int ldw, void* C,
                                  int c_dtype, int ldc, int M, int N, int K, int epilogue, float gate_limit,
-                                 float gate_slope, const float* bias, cudaStream_t stream) {
+                                 float gate_slope, const float* bias, int silu_cols, cudaStream_t stream) {
     return gemm_generic_launch(A, a_dtype, lda, W, w_dtype, ldw, C, c_dtype, ldc, M, N, K, epilogue, 1,
-                               b200::ProductExtras{0, 0, 0, gate_limit, gate_slope, bias}, stream);
+                               b200::ProductExtras{0, 0, 0, gate_limit, gate_slope, bias, silu_cols}, stream);
 }
 
 // n_batch products of the same shape: product z uses A + z a_step, W + z w_step, C + z c_step (steps in elements).
@@ -333,5 +336,5 @@ extern "C" int b200_gemm_generic_batched(const void* A, int a_dtype, int lda, lo
                                          int ldw, long long w_step, void* C, int c_dtype, int ldc, long long c_step, int M,
                                          int N, int K, int n_batch, cudaStream_t stream) {
     return gemm_generic_launch(A, a_dtype, lda, W, w_dtype, ldw, C, c_dtype, ldc, M, N, K, 0, n_batch,
-                               b200::ProductExtras{a_step, w_step, c_step, 0.f, 0.f, nullptr}, stream);
+                               b200::ProductExtras{a_step, w_step, c_step, 0.f, 0.f, nullptr, 0}, stream);
 }

@@ -89,6 +89,7 @@ struct RopeEpilogue {
                                // 2 the clamped form g' sigmoid(slope g') (u' + 1), g' = min(g, limit), u' = clamp(u, -limit, limit)
     float gate_limit, gate_slope;
     const float* bias;         // [N] float32 or null: joins every sum before the store, residual and gated epilogues (not EPI 3)
+    int silu_cols;             // EPI 0: columns below this one are stored as silu(sum) (projections that are used activated)
 };
 
 __device__ __forceinline__ float gated_clamped(float gate, float up, float limit, float slope) {
@@ -96,8 +97,13 @@ __device__ __forceinline__ float gated_clamped(float gate, float up, float limit
     return g / (1.0f + expf(-slope * g)) * (u + 1.0f);
 }
 
+// z sigmoid(y) for results that are rounded to bfloat16: the quotient by the fast exponential and division (a few 32-bit
+// roundings; an infinite denominator gives 0)
+__device__ __forceinline__ float times_sigmoid(float z, float y) { return __fdividef(z, 1.0f + __expf(-y)); }
+
 __device__ __forceinline__ float gated_pair(float gate, float up, int act) {
-    if (act == 1) return 0.5f * gate * (1.0f + tanhf(0.7978845608028654f * (gate + 0.044715f * gate * gate * gate))) * up;
+    // (0.5 (1 + tanh(y)) = sigmoid(2 y))
+    if (act == 1) return times_sigmoid(gate, 1.5957691216057308f * (gate + 0.044715f * gate * gate * gate)) * up;
     return (gate / (1.0f + expf(-gate))) * up;
 }
 
@@ -220,6 +226,15 @@ __device__ __forceinline__ void epilogue_tile(uint32_t acc, int quarter, int lan
             } else {
 #pragma unroll
                 for (int j = 0; j < 32; ++j) if (n0 + c0 + j < N) v[j] += rope.bias[n0 + c0 + j];
+            }
+        }
+        if (EPI == 0 && n0 + c0 < rope.silu_cols) {
+            if (n0 + c0 + 32 <= rope.silu_cols) {
+#pragma unroll
+                for (int j = 0; j < 32; ++j) v[j] = sizeof(TC) == 2 ? times_sigmoid(v[j], v[j]) : v[j] / (1.0f + expf(-v[j]));
+            } else {
+#pragma unroll
+                for (int j = 0; j < 32; ++j) if (n0 + c0 + j < rope.silu_cols) v[j] = v[j] / (1.0f + expf(-v[j]));
             }
         }
         if (EPI == 1 && reduce_c) {
@@ -778,7 +793,8 @@ __device__ __forceinline__ float4 cluster_load_f32x4(uint32_t addr) {
 template <int EPI, typename TC>
 __global__ void __launch_bounds__(kGemmTcThreads, 1)
 gemm_tcgen05_spans_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_w,
-                          TC* __restrict__ C, int ldc, int M, int N, int K, int blocks_per_span, const float* __restrict__ bias) {
+                          TC* __restrict__ C, int ldc, int M, int N, int K, int blocks_per_span, const float* __restrict__ bias,
+                          int silu_cols) {
     constexpr int BN = kSplitBN, STAGES = kSplitStages;
     using Smem = GemmSmem<BN, STAGES>;
     static_assert(sizeof(float) * BM * kSplitPitch <= sizeof(Smem::a), "the partial tile fits in the stages of A");
@@ -891,6 +907,12 @@ gemm_tcgen05_spans_kernel(const __grid_constant__ CUtensorMap map_a, const __gri
                 if (col + 2 < N) acc.z += bias[col + 2];
                 if (col + 3 < N) acc.w += bias[col + 3];
             }
+            if (EPI == 0 && col < silu_cols) {
+                acc.x = acc.x / (1.0f + expf(-acc.x));
+                if (col + 1 < silu_cols) acc.y = acc.y / (1.0f + expf(-acc.y));
+                if (col + 2 < silu_cols) acc.z = acc.z / (1.0f + expf(-acc.z));
+                if (col + 3 < silu_cols) acc.w = acc.w / (1.0f + expf(-acc.w));
+            }
             const float v[4] = {acc.x, acc.y, acc.z, acc.w};
             if (EPI == 2) {  // columns are gate, up, gate, up
                 TC* dst = C + (size_t)row * ldc + (col >> 1);
@@ -1000,8 +1022,9 @@ static int launch_tc(const void* A, int lda, const void* W, int ldw, void* C, in
 
 template <int BN, int STAGES>
 static int launch_width(const void* A, int lda, const void* W, int ldw, void* C, int c_dtype, int ldc, int M, int N, int K,
-                        int epilogue, cudaStream_t stream, int gate_act, float gate_limit, float gate_slope, const float* bias) {
+                        int epilogue, cudaStream_t stream, int gate_act, float gate_limit, float gate_slope, const float* bias, int silu_cols) {
     RopeEpilogue more = {};
+    more.silu_cols = silu_cols;
     more.gate_act = gate_act;
     more.gate_limit = gate_limit;
     more.gate_slope = gate_slope;
@@ -1052,8 +1075,9 @@ static int launch_pair(const void* A, int lda, const void* W, int ldw, void* C, 
 
 template <int BN, int STAGES>
 static int launch_pair_width(const void* A, int lda, const void* W, int ldw, void* C, int c_dtype, int ldc, int M, int N, int K,
-                             int epilogue, cudaStream_t stream, int gate_act, float gate_limit, float gate_slope, const float* bias) {
+                             int epilogue, cudaStream_t stream, int gate_act, float gate_limit, float gate_slope, const float* bias, int silu_cols) {
     RopeEpilogue more = {};
+    more.silu_cols = silu_cols;
     more.gate_act = gate_act;
     more.gate_limit = gate_limit;
     more.gate_slope = gate_slope;
@@ -1086,7 +1110,7 @@ static int k_spans_for(int M, int N, int K) {
 
 template <int EPI, typename TC>
 static int launch_spans(const void* A, int lda, const void* W, int ldw, void* C, int ldc, int M, int N, int K, int spans,
-                        cudaStream_t stream, const float* bias) {
+                        cudaStream_t stream, const float* bias, int silu_cols) {
     CUtensorMap ma, mw;
     if (!make_map(&ma, A, M, K, lda, BM) || !make_map(&mw, W, N, K, ldw, kSplitBN)) return kErrUnsupportedSize;
     const size_t smem = sizeof(GemmSmem<kSplitBN, kSplitStages>) + 1024;
@@ -1100,7 +1124,7 @@ static int launch_spans(const void* A, int lda, const void* W, int ldw, void* C,
     const int kb = (K + BK - 1) / BK;
     const int tiles = ((N + kSplitBN - 1) / kSplitBN) * ((M + BM - 1) / BM);
     return launch_pdl_cluster(kernel, dim3(tiles, spans), dim3(kGemmTcThreads), smem, stream, dim3(1, spans, 1), true,
-                              ma, mw, (TC*)C, ldc, M, N, K, (kb + spans - 1) / spans, bias);
+                              ma, mw, (TC*)C, ldc, M, N, K, (kb + spans - 1) / spans, bias, silu_cols);
 }
 
 template <int BN, int STAGES, int EPI, typename TC>
@@ -1168,11 +1192,12 @@ extern "C" int b200_gemm_tcgen05_k_spans(int M, int N, int K) {
 // tile_width: 256, 128 or 64 output columns per tile; 0 lets the product's shape decide.
 // k_spans: 2 or 4 cuts K among the CTAs of a cluster (128-column tiles; tile_width is then ignored), 1 never does,
 // 0 lets the shape decide.
-// bias: float32 [N] or null, joins every sum before the epilogue.
+// bias: float32 [N] or null, joins every sum before the epilogue.  silu_cols: epilogue 0 stores its first so many columns as
+// silu(sum).
 // cta_pair: 1 computes 256-row tiles by pairs of CTAs (tile_width 256 or 128), -1 never does, 0 lets the shape decide.
 extern "C" int b200_gemm_tcgen05(const void* A, int lda, const void* W, int ldw, void* C, int c_dtype, int ldc, int M,
                                  int N, int K, int epilogue, int tile_width, int k_spans, int cta_pair, float gate_limit,
-                                 float gate_slope, const float* bias, cudaStream_t stream) {
+                                 float gate_slope, const float* bias, int silu_cols, cudaStream_t stream) {
     using namespace b200;
     if (M <= 0 || N <= 0) return 0;
     if (K < 8 || K % 8 != 0 || lda % 8 != 0 || ldw % 8 != 0 || (((uintptr_t)A | (uintptr_t)W) & 15)) return kErrUnsupportedSize;
@@ -1188,8 +1213,8 @@ extern "C" int b200_gemm_tcgen05(const void* A, int lda, const void* W, int ldw,
     if (c_dtype != kF32 && c_dtype != kBF16) return kErrBadArgument;
     if (k_spans != 0 && k_spans != 1 && k_spans != 2 && k_spans != 4) return kErrBadArgument;
     if (cta_pair > 0) {
-        if (tile_width == 128) return launch_pair_width<128, 8>(A, lda, W, ldw, C, c_dtype, ldc, M, N, K, epilogue, stream, gate_act, gate_limit, gate_slope, bias);
-        if (tile_width == 256 || tile_width == 0) return launch_pair_width<256, 6>(A, lda, W, ldw, C, c_dtype, ldc, M, N, K, epilogue, stream, gate_act, gate_limit, gate_slope, bias);
+        if (tile_width == 128) return launch_pair_width<128, 8>(A, lda, W, ldw, C, c_dtype, ldc, M, N, K, epilogue, stream, gate_act, gate_limit, gate_slope, bias, silu_cols);
+        if (tile_width == 256 || tile_width == 0) return launch_pair_width<256, 6>(A, lda, W, ldw, C, c_dtype, ldc, M, N, K, epilogue, stream, gate_act, gate_limit, gate_slope, bias, silu_cols);
         return kErrBadArgument;
     }
     // left the choice: pairs of CTAs as soon as their 256 x 256 tiles occupy two thirds of the SMs (measured: from there on
@@ -1197,23 +1222,23 @@ extern "C" int b200_gemm_tcgen05(const void* A, int lda, const void* W, int ldw,
     if (cta_pair == 0 && tile_width == 0 && (k_spans == 0 || gate_act != 0)) {
         const long long pair_tiles = (long long)((M + 2 * BM - 1) / (2 * BM)) * ((N + 255) / 256);
         if (pair_tiles * 3 >= (long long)(sm_count() / 2) * 2) {
-            const int st = launch_pair_width<256, 6>(A, lda, W, ldw, C, c_dtype, ldc, M, N, K, epilogue, stream, gate_act, gate_limit, gate_slope, bias);
+            const int st = launch_pair_width<256, 6>(A, lda, W, ldw, C, c_dtype, ldc, M, N, K, epilogue, stream, gate_act, gate_limit, gate_slope, bias, silu_cols);
             if (st != kErrUnsupportedSize) return st;   // (no two SMs that can form a pair: the single-CTA kernels below)
         }
     }
     const int spans = k_spans > 0 ? k_spans : (tile_width > 0 ? 1 : k_spans_for(M, N, K));
     if (spans > 1) {
         if ((K + BK - 1) / BK < spans) return kErrBadArgument;
-        if (epilogue == 2) return launch_spans<2, __nv_bfloat16>(A, lda, W, ldw, C, ldc, M, N, K, spans, stream, bias);
-        if (epilogue == 1) return launch_spans<1, float>(A, lda, W, ldw, C, ldc, M, N, K, spans, stream, bias);
-        if (c_dtype == kF32) return launch_spans<0, float>(A, lda, W, ldw, C, ldc, M, N, K, spans, stream, bias);
-        return launch_spans<0, __nv_bfloat16>(A, lda, W, ldw, C, ldc, M, N, K, spans, stream, bias);
+        if (epilogue == 2) return launch_spans<2, __nv_bfloat16>(A, lda, W, ldw, C, ldc, M, N, K, spans, stream, bias, silu_cols);
+        if (epilogue == 1) return launch_spans<1, float>(A, lda, W, ldw, C, ldc, M, N, K, spans, stream, bias, silu_cols);
+        if (c_dtype == kF32) return launch_spans<0, float>(A, lda, W, ldw, C, ldc, M, N, K, spans, stream, bias, silu_cols);
+        return launch_spans<0, __nv_bfloat16>(A, lda, W, ldw, C, ldc, M, N, K, spans, stream, bias, silu_cols);
     }
     // a stage holds 16 KB of A and BN / 8 KB of W: the narrower the tile, the deeper the ring
     const int width = tile_width > 0 ? tile_width : tile_width_for(M, N);
-    if (width == 256) return launch_width<256, 4>(A, lda, W, ldw, C, c_dtype, ldc, M, N, K, epilogue, stream, gate_act, gate_limit, gate_slope, bias);
-    if (width == 128) return launch_width<128, 6>(A, lda, W, ldw, C, c_dtype, ldc, M, N, K, epilogue, stream, gate_act, gate_limit, gate_slope, bias);
-    if (width == 64) return launch_width<64, 8>(A, lda, W, ldw, C, c_dtype, ldc, M, N, K, epilogue, stream, gate_act, gate_limit, gate_slope, bias);
+    if (width == 256) return launch_width<256, 4>(A, lda, W, ldw, C, c_dtype, ldc, M, N, K, epilogue, stream, gate_act, gate_limit, gate_slope, bias, silu_cols);
+    if (width == 128) return launch_width<128, 6>(A, lda, W, ldw, C, c_dtype, ldc, M, N, K, epilogue, stream, gate_act, gate_limit, gate_slope, bias, silu_cols);
+    if (width == 64) return launch_width<64, 8>(A, lda, W, ldw, C, c_dtype, ldc, M, N, K, epilogue, stream, gate_act, gate_limit, gate_slope, bias, silu_cols);
     return kErrBadArgument;
 }
 

@@ -175,6 +175,124 @@ head_rows_kernel(const T* __restrict__ src, int ld_src, T* __restrict__ dst, int
     head_row<T>(src, ld_src, dst, ld_dst, bias, weight, segs.seg[s], t, row, lane, eps, 0.f, cache, mix);
 }
 
+// For launches of many tokens whose rows lie on a grid of eights (turned over halves or not at all; no norm over a whole
+// segment, no mixing): a CTA takes kTile tokens, makes their angles once, and its warps take (row, tokens) in turn.  G
+// lanes share a row, each with one piece of it in registers: four pairs (u[0..3], v[0..3]) of a turned part, or eight
+// numbers behind it; a warp's 32 / G rows are the same row of neighbouring tokens, so that values, which lie transposed in
+// their pages, leave as runs of positions.
+constexpr int kTile = 8, kTileThreads = 256, kTileFreqs = 512;
+
+template <typename T> struct Piece;      // four neighbouring numbers
+template <> struct Piece<__nv_bfloat16> {
+    __device__ static void load(const __nv_bfloat16* p, float* f) {
+        const uint2 v = *reinterpret_cast<const uint2*>(p);
+        f[0] = __uint_as_float(v.x << 16); f[1] = __uint_as_float(v.x & 0xffff0000u);
+        f[2] = __uint_as_float(v.y << 16); f[3] = __uint_as_float(v.y & 0xffff0000u);
+    }
+    __device__ static void store(__nv_bfloat16* p, const float* f) {
+        const __nv_bfloat162 a = __floats2bfloat162_rn(f[0], f[1]), b = __floats2bfloat162_rn(f[2], f[3]);
+        *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+    }
+};
+template <> struct Piece<float> {
+    __device__ static void load(const float* p, float* f) {
+        const float4 v = *reinterpret_cast<const float4*>(p);
+        f[0] = v.x; f[1] = v.y; f[2] = v.z; f[3] = v.w;
+    }
+    __device__ static void store(float* p, const float* f) { *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]); }
+};
+
+template <typename T, int G>
+__global__ void __launch_bounds__(kTileThreads)
+head_rows_tile_kernel(const T* __restrict__ src, int ld_src, T* __restrict__ dst, int ld_dst, const float* __restrict__ bias,
+                      const float* __restrict__ weight, RowSegments segs, float eps, CacheTarget cache, int n_freqs, int n_tokens) {
+    extern __shared__ float2 turn[];      // [kTile][n_freqs]
+    constexpr int RPW = 32 / G;           // tokens a warp takes at once
+    pdl_launch_dependents();
+    const int t0 = blockIdx.x * kTile, lane = threadIdx.x & 31, sub = lane % G;
+    // (positions were copied in before the step's first kernel)
+    for (int i = threadIdx.x; i < kTile * n_freqs; i += kTileThreads) {
+        const int t = min(t0 + i / n_freqs, n_tokens - 1);
+        sincosf((float)cache.positions[t] * cache.inv_freq[i % n_freqs], &turn[i].y, &turn[i].x);
+    }
+    __syncthreads();
+    pdl_wait();
+    const int tasks = segs.total_rows * (kTile / RPW);
+    for (int task = threadIdx.x >> 5; task < tasks; task += kTileThreads / 32) {
+        int s = 0, row = task / (kTile / RPW);
+        const int tt = (task % (kTile / RPW)) * RPW + lane / G, t = t0 + tt;
+        while (s + 1 < segs.n && row >= segs.seg[s].n_rows) {
+            row -= segs.seg[s].n_rows;
+            ++s;
+        }
+        const RowSegment& g = segs.seg[s];
+        const int n = g.rotate == 2 ? g.pairs : 0;
+        const bool pair = sub < n / 4;                             // this lane's piece: pairs, or numbers behind them
+        const int c0 = pair ? sub * 4 : 2 * n + (sub - n / 4) * 8, c1 = pair ? c0 + n : c0 + 4;
+        const bool live = t < n_tokens && c0 < g.d;
+        float z[8] = {};
+        if (live) {
+            const T* x = src + (size_t)t * ld_src + g.src_off + (size_t)row * (g.src_stride >= 0 ? g.src_stride : g.d);
+            Piece<T>::load(x + c0, z);
+            Piece<T>::load(x + c1, z + 4);
+            if (g.bias_off >= 0) {
+                const float* b = bias + g.bias_off + (size_t)row * g.d;
+#pragma unroll
+                for (int e = 0; e < 4; ++e) { z[e] += b[c0 + e]; z[4 + e] += b[c1 + e]; }
+            }
+        }
+        float factor = g.mul;
+        if (g.norm) {
+            float ss = 0.f;
+#pragma unroll
+            for (int e = 0; e < 8; ++e) ss += z[e] * z[e];
+#pragma unroll
+            for (int o = G / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+            factor *= 1.0f / sqrtf(ss / (float)g.d + eps);
+        }
+        if (t >= n_tokens) continue;      // (behind the exchanges)
+        if (live) {
+            const float* w = g.weight_off >= 0 ? weight + g.weight_off + (g.weight_per_row ? (size_t)row * g.d : 0) : nullptr;
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                z[e] *= factor * (w ? w[c0 + e] : 1.f);
+                z[4 + e] *= factor * (w ? w[c1 + e] : 1.f);
+            }
+            if (pair) {
+                const float2* a = turn + tt * n_freqs + g.freq_off + c0;
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    const float u = z[e], v = z[4 + e];
+                    z[e] = u * a[e].x - v * a[e].y;
+                    z[4 + e] = v * a[e].x + u * a[e].y;
+                }
+            }
+        }
+        T* o = dst + (size_t)t * ld_dst + g.dst_off + (size_t)row * (g.dst_stride >= 0 ? g.dst_stride : g.d_pad);
+        if (g.target != 0) {
+            const int pos = cache.positions[t];
+            const size_t page = cache.page_table[(size_t)cache.seq_ids[t] * cache.table_stride + pos / kPageTokens];
+            const size_t head = (page * g.n_rows + row) * kPageTokens * g.d_pad;
+            if (g.target == 2) {          // a row per dimension, positions side by side
+                T* vp = (T*)cache.v_pool + head + (pos % kPageTokens);
+                if (c0 < g.d_pad) {
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) {
+                        vp[(size_t)(c0 + e) * kPageTokens] = from_f32<T>(z[e]);
+                        vp[(size_t)(c1 + e) * kPageTokens] = from_f32<T>(z[4 + e]);
+                    }
+                }
+                continue;
+            }
+            o = (T*)cache.k_pool + head + (size_t)(pos % kPageTokens) * g.d_pad;
+        }
+        if (c0 < g.d_pad) {
+            Piece<T>::store(o + c0, z);
+            Piece<T>::store(o + c1, z + 4);
+        }
+    }
+}
+
 // For launches in which some segment's norm runs over all its rows: a CTA sums such a segment once (its threads in a
 // fixed order), then its warps take the token's rows in turn.
 constexpr int kTokenThreads = 256;
@@ -273,6 +391,32 @@ extern "C" int b200_head_rows(const void* src, int ld_src, void* dst, int ld_dst
             b200::head_rows_token_kernel<T><<<token_grid, b200::kTokenThreads, 0, stream>>>((const T*)src, ld_src, (T*)dst, ld_dst,
                                                                                           bias, weight, segs, eps, cache, mix));
         return b200::launch_status();
+    }
+    // many tokens on a grid of eights: tiles of tokens
+    int n_freqs = 0, lanes = 8;
+    bool tiles = n_tokens >= 256 && ld_src % 4 == 0 && (dst == nullptr || ld_dst % 4 == 0) && positions != nullptr;
+    const size_t el = dtype == b200::kF32 ? 4 : 2;
+    tiles = tiles && (uintptr_t)src % (4 * el) == 0 && (uintptr_t)dst % (4 * el) == 0 && (uintptr_t)k_pool % (4 * el) == 0;
+    for (int i = 0; i < n_segments && tiles; ++i) {
+        const b200::RowSegment& g = segs.seg[i];
+        const int n = g.rotate == 2 ? g.pairs : 0;
+        tiles = g.rotate != 1 && g.mix_off < 0 && g.lead == 0 && g.cache_dim < 0 && g.d % 8 == 0 && g.d_pad % 8 == 0 && n % 4 == 0 &&
+                g.d_pad <= 256 && g.src_off % 4 == 0 && g.dst_off % 4 == 0 && (g.src_stride < 0 || g.src_stride % 4 == 0) &&
+                (g.dst_stride < 0 || g.dst_stride % 4 == 0);
+        if (n > 0 && g.freq_off + n > n_freqs) n_freqs = g.freq_off + n;
+        while (tiles && lanes * 8 < g.d_pad) lanes *= 2;
+    }
+    if (tiles && n_freqs > 0 && n_freqs <= b200::kTileFreqs) {
+        const dim3 tile_grid((n_tokens + b200::kTile - 1) / b200::kTile);
+        const size_t smem = sizeof(float2) * b200::kTile * n_freqs;
+#define B200_TILE(G)                                                                                                               \
+        B200_DISPATCH_DTYPE(dtype, T,                                                                                              \
+            return b200::launch_pdl(b200::head_rows_tile_kernel<T, G>, tile_grid, dim3(b200::kTileThreads), smem, stream,          \
+                                    (const T*)src, ld_src, (T*)dst, ld_dst, bias, weight, segs, eps, cache, n_freqs, n_tokens))
+        if (lanes == 8) B200_TILE(8);
+        if (lanes == 16) B200_TILE(16);
+        B200_TILE(32);
+#undef B200_TILE
     }
     B200_DISPATCH_DTYPE(dtype, T,
         return b200::launch_pdl(b200::head_rows_kernel<T>, grid, dim3(b200::kRowThreads), 0, stream, (const T*)src, ld_src, (T*)dst, ld_dst,

@@ -11,20 +11,21 @@ import torch
 from . import ops
 
 
-def try_gemm(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, epilogue: int, gate_args=(0.0, 0.0), bias=None) -> bool:
+def try_gemm(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, epilogue: int, gate_args=(0.0, 0.0), bias=None,
+             silu_columns: int = 0) -> bool:
     if a.dtype != torch.bfloat16 or w.dtype != torch.bfloat16:
         return False
     M = a.shape[0]
     if M <= 16:
-        return ops.gemm_decode(a, w, c, epilogue, gate_args, bias)
-    if bias is not None:
-        # (the few-token tensor-core kernel has no bias: what it adds to the residual stream gets the bias behind it)
-        if M <= 128 and epilogue == ops.EPILOGUE_RESIDUAL_ADD and c.is_contiguous() and ops.gemm_skinny(a, w, c, epilogue):
+        return ops.gemm_decode(a, w, c, epilogue, gate_args, bias, silu_columns)
+    if bias is not None or silu_columns:
+        # (the few-token tensor-core kernel has neither: what it adds to the residual stream gets the bias behind it)
+        if bias is not None and M <= 128 and epilogue == ops.EPILOGUE_RESIDUAL_ADD and c.is_contiguous() and ops.gemm_skinny(a, w, c, epilogue):
             ops.add_row(c, bias)
             return True
-        if M <= 64 and ops.gemm_decode(a, w, c, epilogue, gate_args, bias):
+        if M <= 64 and ops.gemm_decode(a, w, c, epilogue, gate_args, bias, silu_columns):
             return True
-        return ops.gemm_tcgen05(a, w, c, epilogue, gate_args=gate_args, bias=bias)
+        return ops.gemm_tcgen05(a, w, c, epilogue, gate_args=gate_args, bias=bias, silu_columns=silu_columns)
     # (the few-token tensor-core kernel has the gated epilogue with SiLU only; the other activations' sizes go to the other two)
     if M <= 128 and epilogue in (ops.EPILOGUE_STORE, ops.EPILOGUE_RESIDUAL_ADD, ops.EPILOGUE_GATED_SILU) and ops.gemm_skinny(a, w, c, epilogue):
         return True

@@ -42,17 +42,17 @@ _SIGNATURES = {
                                                    c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
                                                    c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int]),
     "b200_gemm_generic": ("gemm_generic", [c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_void_p, c_int, c_int,
-                                           c_int, c_int, c_int, c_int, c_float, c_float, c_void_p]),
+                                           c_int, c_int, c_int, c_int, c_float, c_float, c_void_p, c_int]),
     "b200_gemm_generic_batched": ("gemm_generic", [c_void_p, c_int, c_int, ctypes.c_longlong, c_void_p, c_int, c_int,
                                                    ctypes.c_longlong, c_void_p, c_int, c_int, ctypes.c_longlong, c_int, c_int,
                                                    c_int, c_int]),
     "b200_gemm_decode": ("gemm_decode", [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int,
-                                         c_int, c_float, c_float, c_void_p]),
+                                         c_int, c_float, c_float, c_void_p, c_int]),
     "b200_gemm_decode_linked": ("gemm_decode", [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int,
                                                 c_int, c_int, c_void_p, c_int, c_float, c_int, c_void_p, c_int, c_void_p,
-                                                c_int, c_void_p, c_void_p, c_void_p, c_void_p]),
+                                                c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int]),
     "b200_gemm_tcgen05": ("gemm_tcgen05", [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int,
-                                           c_int, c_int, c_int, c_int, c_float, c_float, c_void_p]),
+                                           c_int, c_int, c_int, c_int, c_float, c_float, c_void_p, c_int]),
     "b200_gemm_tcgen05_grouped": ("gemm_tcgen05", [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
                                                    c_void_p, c_int, c_float, c_float]),
     "b200_gemm_tcgen05_qkv_rope": ("gemm_tcgen05", [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p,
@@ -108,7 +108,7 @@ _SIGNATURES = {
                                         c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_int, c_int, c_int, c_int,
                                         c_int, c_void_p, c_void_p]),
     "b200_fixed_decay": ("fixed_decay", [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, ctypes.c_longlong,
-                                         c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int,
+                                         c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int,
                                          c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_int, c_int, c_void_p,
                                          c_int, c_float, c_float]),
     "b200_moe_table_route": ("moe", [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int]),
@@ -367,10 +367,12 @@ def _bias_ptr(bias: torch.Tensor | None, n: int):
 
 
 def gemm_generic(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, epilogue: int = EPILOGUE_STORE,
-                 gate_args: tuple[float, float] = (0.0, 0.0), bias: torch.Tensor | None = None) -> None:
+                 gate_args: tuple[float, float] = (0.0, 0.0), bias: torch.Tensor | None = None,
+                 silu_columns: int = 0) -> None:
     """c = a @ w.T (store), c += a @ w.T (residual add, c float32) or c = act(gate) * up with
     gate/up rows interleaved in w (act: SiLU, or GELU in its tanh form).  32-bit FMA accumulation, no tensor cores.
-    ``bias`` float32 [w.shape[0]] joins every sum before the epilogue."""
+    ``bias`` float32 [w.shape[0]] joins every sum before the epilogue; the store epilogue passes the first ``silu_columns``
+    results through SiLU."""
     _dev(a, w, c)
     M, K = a.shape
     N = w.shape[0]
@@ -379,7 +381,7 @@ def gemm_generic(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, epilogue: in
     _check(_fn("b200_gemm_generic")(
         a.data_ptr(), dtype_code(a.dtype), a.stride(0), w.data_ptr(), dtype_code(w.dtype), w.stride(0), c.data_ptr(),
         dtype_code(c.dtype), c.stride(0), M, N, K, epilogue, float(gate_args[0]), float(gate_args[1]),
-        _bias_ptr(bias, N), _stream()), "gemm_generic")
+        _bias_ptr(bias, N), int(silu_columns), _stream()), "gemm_generic")
 
 
 def gemm_per_head(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor) -> None:
@@ -396,7 +398,7 @@ def gemm_per_head(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor) -> None:
 
 
 def gemm_decode(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, epilogue: int = EPILOGUE_STORE,
-                gate_args: tuple[float, float] = (0.0, 0.0), bias: torch.Tensor | None = None) -> bool:
+                gate_args: tuple[float, float] = (0.0, 0.0), bias: torch.Tensor | None = None, silu_columns: int = 0) -> bool:
     """The decode-step matrix product (bfloat16 operands, at most 64 tokens, K a multiple of 32).
     Returns False, having done nothing, for operands it does not take."""
     M, K = a.shape
@@ -409,7 +411,7 @@ def gemm_decode(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, epilogue: int
     assert c.shape[1] == (N // 2 if epilogue in GATED_EPILOGUES else N)
     _check(_fn("b200_gemm_decode")(a.data_ptr(), a.stride(0), w.data_ptr(), w.stride(0), c.data_ptr(),
                                    dtype_code(c.dtype), c.stride(0), M, N, K, epilogue, float(gate_args[0]),
-                                   float(gate_args[1]), _bias_ptr(bias, N), _stream()), "gemm_decode")
+                                   float(gate_args[1]), _bias_ptr(bias, N), int(silu_columns), _stream()), "gemm_decode")
     return True
 
 
@@ -426,7 +428,7 @@ def gemm_decode_partials(n_rows: int, n_out: int) -> int:
 
 
 def gemm_decode_linked(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, epilogue: int, *, row_factors=None,
-                       emit=None, emit_second=None, bias: torch.Tensor | None = None) -> None:
+                       emit=None, emit_second=None, bias: torch.Tensor | None = None, silu_columns: int = 0) -> None:
     """``gemm_decode`` as one half, or both, of an RMSNorm split between two products (at most 16 rows).
 
     ``row_factors = (partials [M, P] float32, eps, dim)``: the rows of ``a`` are x * w of a norm; every
@@ -463,12 +465,12 @@ def gemm_decode_linked(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, epilog
     _check(_fn("b200_gemm_decode_linked")(
         a.data_ptr(), a.stride(0), w.data_ptr(), w.stride(0), c.data_ptr(), dtype_code(c.dtype), c.stride(0), M, N, K,
         epilogue, in_p, n_in, float(eps), int(dim), out_w, out_w_dtype, out_act, ld_act, out_p, out_w2, out_act2,
-        _bias_ptr(bias, N), _stream()), "gemm_decode_linked")
+        _bias_ptr(bias, N), int(silu_columns), _stream()), "gemm_decode_linked")
 
 
 def gemm_tcgen05(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, epilogue: int = EPILOGUE_STORE,
                  tile_width: int = 0, k_spans: int = 0, cta_pair: int = 0,
-                 gate_args: tuple[float, float] = (0.0, 0.0), bias: torch.Tensor | None = None) -> bool:
+                 gate_args: tuple[float, float] = (0.0, 0.0), bias: torch.Tensor | None = None, silu_columns: int = 0) -> bool:
     """The prefill matrix product on tcgen05 tensor cores (bfloat16 operands, rows 16-byte aligned).
     ``tile_width``: 256, 128 or 64 output columns per tile; 0 lets the shape decide (narrower tiles when the
     widest would leave SMs without one).  ``k_spans``: 2 or 4 cuts K among the CTAs of a cluster, which add their
@@ -491,7 +493,7 @@ def gemm_tcgen05(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, epilogue: in
     assert Kw == K and c_inner == 1 and c.shape == (M, N // 2 if epilogue in GATED_EPILOGUES else N)
     _check(_fn("b200_gemm_tcgen05")(pa, lda, pw, ldw, c.data_ptr(), dtype_code(c.dtype), ldc, M, N, K, epilogue,
                                     tile_width, k_spans, cta_pair, float(gate_args[0]), float(gate_args[1]),
-                                    _bias_ptr(bias, N), _stream()), "gemm_tcgen05")
+                                    _bias_ptr(bias, N), int(silu_columns), _stream()), "gemm_tcgen05")
     return True
 
 
@@ -1299,14 +1301,14 @@ def fixed_decay_finishes(all_single: bool, d_k: int, d_v: int) -> bool:
 def fixed_decay(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, state: torch.Tensor, slots: torch.Tensor,
                 cu_seqlens: torch.Tensor, positions: torch.Tensor, heads: int, d_k: int, d_v: int, max_q_len: int, *,
                 q_scale: float = 1.0, qk_silu: bool = False, v_silu: bool = False, inv_freq: torch.Tensor | None = None,
-                angles: torch.Tensor | None = None, out: torch.Tensor | None = None, finish=None, alloc=None) -> None:
+                out: torch.Tensor | None = None, finish=None, alloc=None) -> None:
     """S <- g S + k v^T, o = S^T (q_scale q) per head over a packed step, g = decay[h] (float32 [heads]), S the float32 [slots,
     >= heads d_k d_v] ``state`` at the sequence's slot, updated in place.  q, k [T, >= heads d_k], v [T, >= heads d_v] of one type;
-    ``qk_silu`` / ``v_silu``: they pass through SiLU; ``inv_freq`` float32 [n] (and for steps of more than one token per sequence
-    ``angles`` float32 [n, T, 2], ``rope_angles`` of the pass): the pairs (i, i + n) of q and k are turned by the positions.
+    ``qk_silu`` / ``v_silu``: they pass through SiLU; ``inv_freq`` float32 [n]: the pairs (i, i + n) of q and k are turned by the
+    positions.  Steps of more than one token per sequence take bfloat16 operands.
     ``out`` float32 [T, heads d_v], or ``finish`` = (rows [T, heads d_v], gate [T, >= heads d_v], activation, eps, mul): rows = o /
     sqrt(mean(o^2) + eps) per head * act(gate) * mul, rows being columns of a wider buffer."""
-    _dev(q, k, v, decay, state, slots, cu_seqlens, positions, inv_freq, angles, out)
+    _dev(q, k, v, decay, state, slots, cu_seqlens, positions, inv_freq, out)
     T = q.shape[0]
     assert q.dtype == k.dtype == v.dtype and q.stride(1) == k.stride(1) == v.stride(1) == 1
     assert q.shape[1] >= heads * d_k and k.shape[1] >= heads * d_k and v.shape[1] >= heads * d_v
@@ -1315,10 +1317,11 @@ def fixed_decay(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.
     pairs = inv_freq.numel() if inv_freq is not None else 0
     single = T == slots.numel()
     assert pairs == 0 or (inv_freq.dtype == torch.float32 and inv_freq.is_contiguous() and 2 * pairs <= d_k)
-    assert pairs == 0 or single or (angles.dtype == torch.float32 and angles.is_contiguous() and tuple(angles.shape) == (pairs, T, 2))
     scratch = None
     if not single:
-        shape = (int(library("fixed_decay").b200_fixed_decay_runs(c_int(T), c_int(slots.numel()))), heads, d_k, d_v)
+        floats = library("fixed_decay").b200_fixed_decay_scratch
+        floats.restype = ctypes.c_longlong
+        shape = (int(floats(c_int(T), c_int(slots.numel()), c_int(heads), c_int(d_k), c_int(d_v))),)
         scratch = alloc(shape, torch.float32) if alloc is not None else torch.empty(shape, dtype=torch.float32, device=q.device)
     rows = gate = None
     act, eps, mul = "silu", 0.0, 1.0
@@ -1332,7 +1335,7 @@ def fixed_decay(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.
     ptr = lambda t: t.data_ptr() if t is not None else None
     _check(_fn("b200_fixed_decay")(
         q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0), decay.data_ptr(), state.data_ptr(),
-        state.stride(0), slots.data_ptr(), cu_seqlens.data_ptr(), positions.data_ptr(), ptr(inv_freq), ptr(angles), pairs, ptr(out),
+        state.stride(0), slots.data_ptr(), cu_seqlens.data_ptr(), positions.data_ptr(), ptr(inv_freq), pairs, ptr(out),
         ptr(scratch), dtype_code(q.dtype), T, slots.numel(), int(max_q_len), heads, d_k, d_v, float(q_scale), 1 if qk_silu else 0,
         1 if v_silu else 0, ptr(gate), gate.stride(0) if gate is not None else 0, GATE_ACTIVATIONS[act], ptr(rows),
         rows.stride(0) if rows is not None else 0, float(eps), float(mul), _stream()), "fixed_decay" if not single else "fixed_decay:step")

@@ -12,22 +12,24 @@ from .base import ScaledRows
 
 
 class Linear:
-    def __init__(self, weight: torch.Tensor, bias: torch.Tensor | None = None):
+    def __init__(self, weight: torch.Tensor, bias: torch.Tensor | None = None, silu_columns: int = 0):
         """``bias``: one number per row of the weight, kept in 32 bits; it joins the sums before whatever the product's
-        epilogue does with them."""
+        epilogue does with them.  ``silu_columns``: how many of the first results pass through SiLU as they are stored
+        (``store`` and ``into``)."""
         assert weight.dim() == 2 and weight.is_contiguous()
         self.weight = weight
+        self.silu_columns = int(silu_columns)
         self.bias = bias.to(device=weight.device, dtype=torch.float32).contiguous() if bias is not None else None
         self.out_features, self.in_features = weight.shape
 
     def _run(self, a, c: torch.Tensor, epilogue: int, gate_args=(0.0, 0.0)) -> None:
         if isinstance(a, ScaledRows):  # only handed to a product that said it links (links_with)
             ops.gemm_decode_linked(a.data, self.weight, c, epilogue, row_factors=(a.partials, a.eps, a.dim),
-                                   bias=self.bias)
+                                   bias=self.bias, silu_columns=self.silu_columns)
             return
-        if fast.try_gemm(a, self.weight, c, epilogue, gate_args, self.bias):
+        if fast.try_gemm(a, self.weight, c, epilogue, gate_args, self.bias, self.silu_columns):
             return
-        ops.gemm_generic(a, self.weight, c, epilogue, gate_args, self.bias)
+        ops.gemm_generic(a, self.weight, c, epilogue, gate_args, self.bias, self.silu_columns)
 
     def links_with(self, n_rows: int, dtype: torch.dtype) -> bool:
         """Whether this product can be one half of a split norm for ``n_rows`` rows of ``dtype``."""

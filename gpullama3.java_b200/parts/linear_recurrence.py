@@ -41,8 +41,9 @@ def _pad8(n: int) -> int:
     return -(-n // 8) * 8
 
 
-def _stacked(groups: list[torch.Tensor], device) -> tuple[Linear, list[int]]:
-    """One product for several weights: their rows one after the other, each group padded to a multiple of 8 rows."""
+def _stacked(groups: list[torch.Tensor], device, silu_groups: int = 0) -> tuple[Linear, list[int]]:
+    """One product for several weights: their rows one after the other, each group padded to a multiple of 8 rows.
+    ``silu_groups``: so many of the first groups' results are stored activated."""
     common = torch.float32 if any(g.dtype == torch.float32 for g in groups) else groups[0].dtype
     rows, offsets, at = [], [], 0
     for g in groups:
@@ -52,7 +53,8 @@ def _stacked(groups: list[torch.Tensor], device) -> tuple[Linear, list[int]]:
         if pad:
             rows.append(torch.zeros((pad, g.shape[1]), dtype=common, device=device))
         at += _pad8(g.shape[0])
-    return Linear(torch.cat(rows, dim=0).contiguous()), offsets
+    offsets.append(at)
+    return Linear(torch.cat(rows, dim=0).contiguous(), silu_columns=offsets[silu_groups]), offsets[:-1]
 
 
 class GatedLinearAttention(Mixer):
@@ -185,7 +187,7 @@ class FixedDecayAttention(Mixer, OpenEnded):
         if activation not in (None, "silu") or norm_over not in ("head", "all") or gate not in ops.GATE_ACTIVATIONS:
             raise ConfigError(f"fixed-decay attention: activation {activation!r}, norm over {norm_over!r}, gate {gate!r}")
         if position is not None and position.rotary_dim:
-            if position.rotary_dim > head_dim or position.pairing != PAIRING_CODES["half"] or not hasattr(position, "angles"):
+            if position.rotary_dim > head_dim or position.pairing != PAIRING_CODES["half"]:
                 raise ConfigError(f"fixed-decay attention turns pairs over halves of at most {head_dim} numbers")
         self.hidden_size, self.n_heads, self.key_dim, self.value_dim = int(hidden_size), int(n_heads), int(head_dim), int(value_dim)
         self.decay, self.norm_eps, self.scale = [float(g) for g in decay], float(norm_eps), float(scale)
@@ -211,7 +213,8 @@ class FixedDecayAttention(Mixer, OpenEnded):
 
     def load(self, tensors, dtype, device):
         run = lambda t: t.to(device).to(torch.float32 if dtype == torch.float32 else t.dtype)
-        self.inputs, (self.q_off, self.k_off, self.v_off, self.g_off) = _stacked([run(tensors[n]) for n in ("q", "k", "v", "g")], device)
+        self.inputs, (self.q_off, self.k_off, self.v_off, self.g_off) = _stacked([run(tensors[n]) for n in ("q", "k", "v", "g")], device,
+                                                                                      silu_groups=3 if self.silu else 0)
         self.o = Linear(run(tensors["o"]).contiguous())
         self.weight = tensors["norm"].to(device=device, dtype=torch.float32).contiguous() if self.norm_weight else None
         self.decays = torch.tensor(self.decay, dtype=torch.float64).to(torch.float32).to(device)
@@ -230,15 +233,19 @@ class FixedDecayAttention(Mixer, OpenEnded):
 
     def take_input(self):
         weight, self.inputs = self.inputs.weight, None
-        return weight
+        return weight     # (whoever multiplies with it stores the results as they are: ``rows_from`` activates them)
 
     def takes_scaled_rows(self, ctx: StepContext) -> bool:
         return ctx.all_decode and self.inputs is not None and self.inputs.links_with(ctx.n_tokens, ctx.dtype)
 
     def rows_into(self, x, ctx: StepContext, cache: StateView, rows, writes_cache=True, mul=1.0):
-        self.rows_from(self.inputs.store(x, ctx.dtype, ctx.empty), ctx, cache, rows, writes_cache, mul)
+        self._recur(self.inputs.store(x, ctx.dtype, ctx.empty), ctx, cache, rows, mul, silu=False)   # (activated by the product)
 
     def rows_from(self, raw, ctx: StepContext, cache: StateView, rows, writes_cache=True, mul=1.0):
+        self._recur(raw, ctx, cache, rows, mul, silu=self.silu)
+
+    def _recur(self, raw, ctx: StepContext, cache: StateView, rows, mul: float, silu: bool):
+        """``silu``: whether the projections still have to be activated."""
         H, dk, dv, T = self.n_heads, self.key_dim, self.value_dim, raw.shape[0]
         q, k, v, g = (raw[:, at:] for at in (self.q_off, self.k_off, self.v_off, self.g_off))
         if ops.fixed_decay_takes(ctx.dtype, ctx.all_decode, dk, dv):
@@ -247,9 +254,8 @@ class FixedDecayAttention(Mixer, OpenEnded):
             if self.norm_over == "head" and self.weight is None and ops.fixed_decay_finishes(ctx.all_decode, dk, dv):
                 finish = (rows, g, self.gate, self.norm_eps, mul)
             o = None if finish is not None else ctx.empty((T, H * dv), torch.float32)
-            angles = self.position.angles(ctx) if self.inv_freq is not None and not ctx.all_decode else None
             ops.fixed_decay(q, k, v, self.decays, cache.data, ctx.slots_dev, ctx.cu_seqlens, ctx.positions, H, dk, dv, ctx.max_q_len,
-                            q_scale=self.scale, qk_silu=self.silu, v_silu=self.silu, inv_freq=self.inv_freq, angles=angles, out=o,
+                            q_scale=self.scale, qk_silu=silu, v_silu=silu, inv_freq=self.inv_freq, out=o,
                             finish=finish, alloc=ctx.empty)
             if finish is not None:
                 return
@@ -257,7 +263,7 @@ class FixedDecayAttention(Mixer, OpenEnded):
             # (the true 32-bit run's prompts, and keys too long for a run's tiles: token by token)
             o = ctx.empty((T, H * dv), torch.float32)
             ops.linear_scan(q, k, v, None, cache.data, ctx.slots_dev, ctx.cu_seqlens, o, H, H, dk, dv, decay_kind=ops.DECAY_FIXED,
-                            decay_per_head=True, a_log=self.decays, q_scale=self.scale, qk_silu=self.silu, v_silu=self.silu,
+                            decay_per_head=True, a_log=self.decays, q_scale=self.scale, qk_silu=silu, v_silu=silu,
                             rotary=(ctx.positions, self.inv_freq) if self.inv_freq is not None else None, alloc=ctx.empty)
         parts, d = (H, dv) if self.norm_over == "head" else (1, H * dv)
         ops.gated_rmsnorm(o, self.weight, g, rows, parts, d, self.norm_eps, self.gate, mul=mul)

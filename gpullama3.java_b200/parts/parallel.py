@@ -12,7 +12,9 @@ feed-forward write their rows into neighbouring columns of one buffer and ONE pr
 layer's whole result into the stream; two mixers likewise start with one product over their joined input weights.  The
 factors of ``ParallelMixers`` are applied to the rows in 32 bits.  The two norms differ in their weights alone, so a prompt
 makes both in one read of the stream, and in a decode step the product that completes the stream leaves both copies for
-the next block's products (``ScaledRows``), whose shared row factor they apply themselves."""
+the next block's products (``ScaledRows``), whose shared row factor they apply themselves.  In a decode step the
+feed-forward's first product, which streams most of a layer's weights, runs on a stream of its own beside the mixer's short
+kernels (a recorded step has two branches there, which meet in the layer's last product)."""
 from __future__ import annotations
 
 import torch
@@ -57,6 +59,24 @@ def _joined(outputs, device=None) -> Linear:
         for b in biases[1:]:
             bias += b
     return Linear(torch.cat([w.to(common) for w in weights], dim=1).contiguous(), bias)
+
+
+_side_streams: dict = {}
+
+
+def _beside(device):
+    """Launches inside run on a stream of their own behind everything the current stream holds so far, beside what it is
+    given next, until ``_join``."""
+    side = _side_streams.get(device)
+    if side is None:
+        side = _side_streams[device] = torch.cuda.Stream(device)
+    side.wait_stream(torch.cuda.current_stream(device))
+    return torch.cuda.stream(side)
+
+
+def _join(device) -> None:
+    """The current stream waits for what runs beside it."""
+    torch.cuda.current_stream(device).wait_stream(_side_streams[device])
 
 
 class ParallelBlock(Block):
@@ -118,8 +138,15 @@ class ParallelBlock(Block):
             return None
         rows = ctx.empty((residual.shape[0], self.out.in_features), ctx.dtype)
         n = self.columns[0]
-        self.mixer.rows_into(h, ctx, cache, rows[:, :n], writes_cache)
-        if self.feed_forward is not None:
+        if self.feed_forward is None:
+            self.mixer.rows_into(h, ctx, cache, rows, writes_cache)
+        elif ctx.all_decode:
+            with _beside(ctx.device):
+                self.feed_forward.rows_into(g, ctx, None, rows[:, n:])
+            self.mixer.rows_into(h, ctx, cache, rows[:, :n], writes_cache)
+            _join(ctx.device)
+        else:
+            self.mixer.rows_into(h, ctx, cache, rows[:, :n], writes_cache)
             self.feed_forward.rows_into(g, ctx, None, rows[:, n:])
         return self.out.add_to(rows, residual, then_norm)
 

@@ -27,10 +27,10 @@ def _gelu_gated(s):
     return P.gelu_tanh(s[:, 0::2]) * s[:, 1::2]
 
 
-def _epilogue(kind, a, w, bias, c0):
+def _epilogue(kind, a, w, bias, c0, silu):
     s = a.cpu().to(F) @ w.cpu().to(F).T + bias.cpu().to(F)
     if kind == "store":
-        return s
+        return torch.cat([P.silu(s[:, :silu]), s[:, silu:]], dim=1)
     return c0.cpu().to(F) + s if kind == "add" else _gelu_gated(s)
 
 
@@ -40,8 +40,9 @@ EPILOGUES = {"store": ops.EPILOGUE_STORE, "add": ops.EPILOGUE_RESIDUAL_ADD, "gel
 @pytest.mark.parametrize("kind", sorted(EPILOGUES))
 @pytest.mark.parametrize("M, N, K", [(1, 48, 64), (5, 130, 96), (16, 40, 32), (30, 96, 64), (64, 4128, 64), (100, 64, 72), (130, 200, 64),
                                      (300, 264, 136), (520, 1032, 512), (200, 72, 4096)])
-def test_biases_of_every_product(kind, M, N, K):
+def test_biases_and_activated_columns_of_every_product(kind, M, N, K):
     torch.manual_seed(M + N)
+    silu = N // 2 + 5 if kind == "store" else 0     # (a border inside every kernel's run of columns)
     g = dict(device="cuda")
     a, w = torch.randn(M, K, **g), torch.randn(N, K, **g) / K ** 0.5
     bias = torch.randn(N, **g)
@@ -52,13 +53,13 @@ def test_biases_of_every_product(kind, M, N, K):
         A, W = a.to(dtype), w.to(dtype)
         out_type = torch.float32 if kind == "add" else dtype
         c0 = torch.randn(M, n_out, **g).to(out_type)
-        want = _epilogue(kind, A, W, bias, c0)
+        want = _epilogue(kind, A, W, bias, c0, silu)
         rel = 3e-6 if dtype == torch.float32 else 1e-2
         c = c0.clone()
-        Linear(W.contiguous(), bias)._run(A, c, EPILOGUES[kind])
+        Linear(W.contiguous(), bias, silu)._run(A, c, EPILOGUES[kind])
         _close(c, want, rel, f"chosen kernel {dtype} {kind}")
         c = c0.clone()
-        ops.gemm_generic(A, W, c, EPILOGUES[kind], bias=bias)
+        ops.gemm_generic(A, W, c, EPILOGUES[kind], bias=bias, silu_columns=silu)
         _close(c, want, rel, f"plain kernel {dtype} {kind}")
         if dtype == torch.bfloat16:
             variants = [dict(tile_width=t, cta_pair=-1, k_spans=1) for t in (64, 128, 256)] + [dict(cta_pair=1, tile_width=t) for t in (128, 256)]
@@ -66,7 +67,7 @@ def test_biases_of_every_product(kind, M, N, K):
                 variants += [dict(k_spans=s) for s in (2, 4)]
             for v in variants:
                 c = c0.clone()
-                if ops.gemm_tcgen05(A, W, c, EPILOGUES[kind], bias=bias, **v):
+                if ops.gemm_tcgen05(A, W, c, EPILOGUES[kind], bias=bias, silu_columns=silu, **v):
                     _close(c, want, rel, f"tcgen05 {v} {kind}")
             assert ops.gemm_tcgen05_status() == 0
 
@@ -91,8 +92,9 @@ def test_one_product_leaves_two_norms(M, N, K):
     if N % 32 == 0:
         w2, b2 = (torch.randn(40, N, **g) / N ** 0.5).bfloat16(), torch.randn(40, **g)
         out = torch.empty(M, 40, dtype=torch.float32, **g)
-        ops.gemm_decode_linked(acts[1], w2, out, ops.EPILOGUE_STORE, row_factors=(parts, 1e-5, N), bias=b2)
+        ops.gemm_decode_linked(acts[1], w2, out, ops.EPILOGUE_STORE, row_factors=(parts, 1e-5, N), bias=b2, silu_columns=13)
         want = P.over_root_mean_square(x, 1e-5) * n2.cpu().to(F) @ w2.cpu().to(F).T + b2.cpu().to(F)
+        want[:, :13] = P.silu(want[:, :13])
         _close(out, want, 1e-2, "the product behind it")
 
 
@@ -116,10 +118,11 @@ def _pages(n_tokens, n_kv, D, dtype, order_seed=0):
 
 
 @DTYPES
+@pytest.mark.parametrize("T", [70, 300])      # (few tokens: a warp per row; many: a CTA per token)
 @pytest.mark.parametrize("d, dv, D, pairs, vpairs", [(16, 24, 32, 8, 12), (12, 20, 32, 2, 10), (64, 64, 64, 32, 32), (40, 96, 96, 5, 48), (8, 8, 16, 0, 0)])
-def test_rows_turned_over_halves_on_their_way_into_the_cache(dtype, d, dv, D, pairs, vpairs):
+def test_rows_turned_over_halves_on_their_way_into_the_cache(dtype, T, d, dv, D, pairs, vpairs):
     torch.manual_seed(d)
-    T, H, G, start = 70, 4, 2, 31
+    H, G, start = 4, 2, 31
     raw = torch.randn(T, (H + G) * d + G * dv + 3, device="cuda").to(dtype)
     weight = torch.cat([1 + 0.3 * torch.randn(d), 1 + 0.3 * torch.randn(d)]).cuda()
     fk = torch.tensor(P.pair_frequencies(100.0, 2 * pairs), dtype=torch.float32) if pairs else torch.zeros(0)
@@ -262,8 +265,8 @@ CASES = [  # heads, d_k, d_v, pairs, silu, decays
 def test_fixed_decays(dtype, H, dk, dv, pairs, silu, decays, cut):
     """Two sequences through steps of the given numbers of tokens each, against the recurrence in float64: the outputs and the
     state that is left, in slots that others have used.  The bfloat16 run's operands are rounded once (the projections); what
-    the recurrence does with them must be 32-bit: the bound is a hundredth of one bfloat16 rounding, unless the values pass
-    through SiLU (an activation of the projection, which may be rounded)."""
+    the recurrence does with them must be 32-bit: the bound is a hundredth of one bfloat16 rounding, unless the operands pass
+    through SiLU (an activation of the projections, which is rounded: q, k and v once each)."""
     torch.manual_seed(dk + dv)
     lens = [sum(c[i] for c in cut) for i in range(2)]
     data = [[torch.randn(n, H, d).to(dtype) for d in (dk, dk, dv, dv)] for n in lens]
@@ -288,8 +291,7 @@ def test_fixed_decays(dtype, H, dk, dv, pairs, silu, decays, cut):
         single = all(n == 1 for n in ns)
         finished = None
         if ops.fixed_decay_takes(dtype, single, dk, dv):
-            angles = ops.rope_angles(pos, freqs, pairs) if pairs and not single else None
-            kw = dict(q_scale=scale, qk_silu=silu, v_silu=silu, inv_freq=freqs, angles=angles)
+            kw = dict(q_scale=scale, qk_silu=silu, v_silu=silu, inv_freq=freqs)
             before = state.clone()
             if ops.fixed_decay_finishes(single, dk, dv):
                 wide = torch.zeros(T, H * dv + 3, dtype=dtype, device="cuda")
@@ -320,7 +322,7 @@ def test_fixed_decays(dtype, H, dk, dv, pairs, silu, decays, cut):
             f = freqs.cpu().to(F).tolist()
             q, k = P.turn_halves(q, f), P.turn_halves(k, f)
         want = P.decayed_outer_sum(q * scale, k, v, [float(x) for x in decay.cpu()])
-        tol = 1e-5 if dtype == torch.float32 else (4e-3 if silu else 4e-5)
+        tol = 1e-5 if dtype == torch.float32 else (8e-3 if silu else 4e-5)
         _close(torch.cat(got[i]).view(-1, H, dv), want, tol, f"outputs of sequence {i}")
         S = torch.zeros(H, dk, dv, dtype=F)
         for t in range(lens[i]):
@@ -332,6 +334,23 @@ def test_fixed_decays(dtype, H, dk, dv, pairs, silu, decays, cut):
             if r is not None:
                 _close(r.view(n, H, dv), done[a:a + n], 2e-4 if dtype == torch.float32 else 2e-2, "finished heads")
             a += n
+
+
+@DTYPES
+@pytest.mark.parametrize("gate_first", [False, True])
+@pytest.mark.parametrize("T, parts, d, weighted", [(5, 1, 120, True), (3, 2, 512, False), (70, 1, 2048, True), (9, 1, 4100, True), (4, 3, 515, True)])
+def test_gated_norms_with_and_without_a_weight(dtype, gate_first, T, parts, d, weighted):
+    torch.manual_seed(d)
+    x, w = torch.randn(T, parts * d, device="cuda"), torch.randn(parts * d, device="cuda")
+    gate = torch.randn(T, parts * d + 4, device="cuda").to(dtype)[:, :parts * d]
+    for off in (0, 3):
+        wide = torch.zeros(T, parts * d + 8, dtype=dtype, device="cuda")
+        ops.gated_rmsnorm(x, w if weighted else None, gate, wide[:, off:off + parts * d], parts, d, 1e-5, "silu", gate_first=gate_first, mul=0.6)
+        z, g = (a.cpu().to(F).view(T, parts, d) for a in (x, gate))
+        g = P.silu(g)
+        n = P.over_root_mean_square(z * g if gate_first else z, 1e-5) * (w.cpu().to(F).view(parts, d) if weighted else 1.0) * 0.6
+        _close(wide[:, off:off + parts * d].reshape(T, parts, d), n if gate_first else n * g, 3e-6 if dtype == torch.float32 else 6e-3)
+        assert float(wide[:, :off].abs().sum()) == 0.0 and float(wide[:, off + parts * d:].abs().sum()) == 0.0
 
 
 def test_parts_that_keep_their_products_run_one_after_the_other(session_tmp):
