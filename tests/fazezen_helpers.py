@@ -75,7 +75,7 @@ FAZEZEN_C = {
 FAZEZEN_D = {
     "architecture": "Fazezen", "vocab": 120, "width": 640, "norm": {"eps": 1e-5}, "initializer_range": 0.04,
     "layers": [
-        _par(_left(8, 2, 64, 64, 0.15, 130, _rot(10000.0, 64, (8.0, 1.0, 4.0, 128))), _rec(128, 128, (0.99, 0.9), _rot(20000.0, 128)), 1.2, 0.9, 256),
+        _par(_left(8, 2, 64, 64, 0.15, 130, _rot(10000.0, 64, (8.0, 1.0, 4.0, 128))), _rec(128, 128, (0.99, 0.9), _rot(20000.0, 128)), 1.25, 0.85, 256),
         _lig(128, 192, (0.97, 0.999)),
         _par(_left(4, 4, 128, 96, 0.1, 33, _rot(700.0, 64)), _rec(32, 64, (0.8, 0.95, 0.99), _rot(100.0, 16)), 0.8, 1.1, 128),
     ],

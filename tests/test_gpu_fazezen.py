@@ -223,6 +223,32 @@ def test_logits_do_not_depend_on_the_batch(setup, dtype):
     cache.check_invariants()
 
 
+@DTYPES
+@pytest.mark.parametrize("name, n", [("B", 20), ("D", 40), ("B", 70), ("C", 130)])
+def test_large_batches(session_tmp, dtype, name, n):
+    """More sequences than the decode products take at once: prompts of unequal length in one step, then tokens decoded
+    together (17 to 64, up to 128 and more rows go to other product kernels), each sequence against the plain
+    implementation of it alone."""
+    from gpullama3.java_b200.engine.step import SequenceInput, StepFunction
+    from gpullama3.java_b200.engine.trace import load_model
+
+    d = make_fazezen_dir(session_tmp, CONFIGS[name], seed=11)
+    cfg, weights = plain_inputs(d)
+    lengths = [3 + (7 * i) % 11 for i in range(n)]
+    prompts = random_prompts(cfg["vocab"], lengths, seed=31)
+    model = load_model(d, dtype)
+    cache = model.new_cache(64 * n, max_slots=n)
+    step = StepFunction(model, cache)
+    slots = [cache.acquire() for _ in range(n)]
+    outs = [step([SequenceInput(s, p[:-2], [len(p) - 3]) for s, p in zip(slots, prompts)]).cpu().clone()]
+    for k in (2, 1):
+        outs.append(step([SequenceInput(s, [p[-k]], [0]) for s, p in zip(slots, prompts)]).cpu().clone())
+    got = torch.stack(outs, dim=1)
+    for i in range(0, n, max(1, n // 12)):
+        ref = reference(cfg, weights, prompts[i])
+        assert_logits(got[i], ref[-3:], dtype, f"sequence {i} of {n}")
+
+
 def test_trace_run_program(setup, tmp_path):
     """The program itself, as a user starts it: steps on standard input, 'done <step>' lines out, and a cache sized
     from the tokens alone (no allowance for partly filled pages)."""
