@@ -30,7 +30,8 @@
 // keep_first positions stay visible (their blocks of keys are walked ahead of the window's, and count in the span plan);
 // a distance penalty slopes[h] * (position - key) taken off every score; a sink per head, a key without a value whose
 // exponential joins the denominator (the first warp of a sequence's first span starts its running maximum and sum
-// at (sinks[h], 1)); a gate per (sequence, head): the output is multiplied by sigmoid(gate).
+// at (sinks[h], 1)); a gate per (sequence, head): the output is multiplied by sigmoid(gate); a soft cap: score <- softcap *
+// tanh(score / softcap), before the penalty.
 //
 // A further mask (DecodeTerms.chunk): positions are cut into runs of `chunk`, counted from position 0, and the token sees
 // the keys of its own run only.  It reaches the kernel as the window that ends at the token and starts with its run.
@@ -88,6 +89,7 @@ struct DecodeTerms {
     const float* sinks;            // [n_heads] or null
     const __nv_bfloat16* gate;     // [n_seqs][ld_gate], column h, or null
     int ld_gate;
+    float softcap;                 // 0: none
 };
 
 struct RopeArgs {            // what the fused variant needs beyond the plain one
@@ -171,7 +173,7 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_row_stride, _
                         float* __restrict__ part_o, float* __restrict__ part_ml, int n_heads, int n_kv_heads,
                         int window, int n_splits, RopeArgs rope, DecodeTerms given) {
     constexpr int D = KB * 32;
-    const DecodeTerms terms = TERMS ? given : DecodeTerms{0, 0, nullptr, nullptr, nullptr, 0};
+    const DecodeTerms terms = TERMS ? given : DecodeTerms{0, 0, nullptr, nullptr, nullptr, 0, 0.f};
     constexpr int NJ = D / 8;  // output tiles of 8 dims
     constexpr int SLOTS = kAttnDecodeWarps + (FUSED ? 1 : 0);  // partials merged per CTA: the warps, and the new key
     // Rows of the tiles that exist: 8 without the upper half.  (Shared memory is taken from the SM's L1, through which the
@@ -299,6 +301,7 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_row_stride, _
     // scores are scaled by a multiplication: a division by sqrt(d) that is no power of two (head sizes 32, 96, 128) is a
     // subroutine that, with this kernel's registers all taken, cost more than the block's tensor-core work
     const float inv_sqrt_d = 1.f / sqrtf((float)D);
+    const float cap_log2 = TERMS && terms.softcap > 0.f ? 2.885390081777927f / terms.softcap : 0.f;    // 2 log2(e) / softcap
 
     for (int vblk = blk_begin + warp; vblk < blk_end; vblk += kAttnDecodeWarps) {
         const int base = block_of(vblk) * 32;
@@ -337,6 +340,13 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_row_stride, _
                     mma16816_lo(s[i][0], s[i][1], ql[kb].z, ql[kb].w, kf[i][kb].z, kf[i][kb].w);
                 }
             }
+        }
+        if (TERMS && terms.softcap > 0.f) {   // (back in units of q.k, as the scores below are)
+            const float sqrt_d = sqrtf((float)D);
+#pragma unroll
+            for (int i = 0; i < 4; ++i)
+#pragma unroll
+                for (int c = 0; c < (HI ? 4 : 2); ++c) s[i][c] = soft_capped_fast(s[i][c] * inv_sqrt_d, terms.softcap, cap_log2) * sqrt_d;
         }
         // lane t's columns of tile i are keys base + 8t + 2i and + 2i + 1
         float bm_lo = -INFINITY, bm_hi = -INFINITY;
@@ -604,8 +614,9 @@ static int launch_attention_decode(const void* q, int q_row_stride, void* out, c
                                    int table_stride, void* k_pool, void* v_pool, float* scratch, long long scratch_floats,
                                    int n_seqs, int n_heads, int n_kv_heads, int head_dim, int window, int n_splits,
                                    bool fused, RopeArgs rope, bool early_start, cudaStream_t stream,
-                                   DecodeTerms terms = DecodeTerms{0, 0, nullptr, nullptr, nullptr, 0}) {
+                                   DecodeTerms terms = DecodeTerms{0, 0, nullptr, nullptr, nullptr, 0, 0.f}) {
     if (n_seqs <= 0) return 0;
+    if (!(terms.softcap >= 0.f)) return kErrBadArgument;
     if (terms.keep_first < 0 || (terms.keep_first > 0 && window <= 0)) return kErrBadArgument;
     if (terms.chunk < 0 || (terms.chunk > 0 && (window > 0 || terms.keep_first > 0))) return kErrBadArgument;
     if (n_kv_heads <= 0 || n_heads % n_kv_heads != 0 || n_splits < 1) return kErrBadArgument;
@@ -628,7 +639,7 @@ static int launch_attention_decode(const void* q, int q_row_stride, void* out, c
     auto vv = (__nv_bfloat16*)v_pool;
     auto oo = (__nv_bfloat16*)out;
     int st = 0;
-    const bool any_term = terms.keep_first > 0 || terms.chunk > 0 || terms.slopes || terms.sinks || terms.gate;
+    const bool any_term = terms.keep_first > 0 || terms.chunk > 0 || terms.slopes || terms.sinks || terms.gate || terms.softcap > 0.f;
     if (any_term && fused) return kErrBadArgument;   // (the fused variant is not built with the terms)
 #define B200_LAUNCH(KB, F) do { if (group > 8) B200_LAUNCH_T(KB, F, true); else B200_LAUNCH_T(KB, F, false); } while (0)
 #define B200_LAUNCH_T(KB, F, HI) do { if (!F && any_term) B200_LAUNCH_H(KB, F, HI, !F); else B200_LAUNCH_H(KB, F, HI, false); } while (0)
@@ -710,17 +721,17 @@ extern "C" int b200_attention_decode(const void* q, int q_row_stride, void* out,
                                          head_dim, window, n_splits, false, b200::RopeArgs{nullptr, 0, 0}, early_start != 0, stream);
 }
 
-// The same with the further terms of DecodeTerms (null pointers and keep_first 0 switch each off).
+// The same with the further terms of DecodeTerms (null pointers, keep_first 0 and softcap 0 switch each off).
 extern "C" int b200_attention_decode_terms(const void* q, int q_row_stride, void* out, const int* kv_lens,
                                            const int* page_table, int table_stride, const void* k_pool, const void* v_pool,
                                            float* scratch, long long scratch_floats, int n_seqs, int n_heads, int n_kv_heads,
                                            int head_dim, int window, int n_splits, int early_start, int keep_first, int chunk,
                                            const float* slopes, const float* sinks, const void* gate, int ld_gate,
-                                           cudaStream_t stream) {
+                                           float softcap, cudaStream_t stream) {
     return b200::launch_attention_decode(q, q_row_stride, out, kv_lens, page_table, table_stride, const_cast<void*>(k_pool),
                                          const_cast<void*>(v_pool), scratch, scratch_floats, n_seqs, n_heads, n_kv_heads,
                                          head_dim, window, n_splits, false, b200::RopeArgs{nullptr, 0, 0}, early_start != 0, stream,
-                                         b200::DecodeTerms{keep_first, chunk, slopes, sinks, (const __nv_bfloat16*)gate, ld_gate});
+                                         b200::DecodeTerms{keep_first, chunk, slopes, sinks, (const __nv_bfloat16*)gate, ld_gate, softcap});
 }
 
 // The fused variant: `qkv` holds the step's raw projections [n_seqs, (n_heads + 2 n_kv_heads) head_dim]; queries

@@ -20,6 +20,7 @@
 //   sinks       a learned number per query head whose exponential joins the softmax's denominator (a key without
 //               a value): the running maximum and sum start at (sinks[h], 1) instead of (-inf, 0)
 //   gate        a number per (token, head), before its sigmoid: the head's output is multiplied by sigmoid(gate)
+//   softcap     score <- softcap * tanh(score / softcap), before the penalty (the sink is not capped)
 #include "common.cuh"
 
 namespace b200 {
@@ -34,6 +35,7 @@ struct AttentionTerms {
     const float* sinks;    // [n_heads] or null
     const void* gate;      // [T][ld_gate] of the run's storage type, column h, or null
     int ld_gate;
+    float softcap;         // 0: none
 };
 
 template <typename T> struct Vec16;  // 16-byte vector of storage type T
@@ -138,7 +140,12 @@ attention_paged_kernel(const T* __restrict__ q, int q_row_stride, T* __restrict_
         __syncwarp();
         const int key = base + tid;          // from here on a thread is a key
         const int j = key < n_keep ? key : key + shift;   // the key's position
-        const float s = key <= last ? s_s[tid] / sqrt_d - slope * (float)(pos - j) : -INFINITY;
+        float s = -INFINITY;
+        if (key <= last) {
+            s = s_s[tid] / sqrt_d;
+            if (terms.softcap > 0.f) s = soft_capped(s, terms.softcap);
+            s -= slope * (float)(pos - j);
+        }
         const float m_tile = block_max(s, red);
         const float m_new = fmaxf(m_run, m_tile);
         const float p = key <= last ? expf(s - m_new) : 0.f;
@@ -226,11 +233,12 @@ extern "C" int b200_attention_paged(const void* q, int q_row_stride, void* out, 
                                     const int* seq_ids, const int* page_table, int table_stride, const void* k_pool,
                                     const void* v_pool, int n_tokens, int n_heads, int n_kv_heads, int head_dim,
                                     int window, int n_splits, float* scratch, int keep_first, int chunk, const float* slopes,
-                                    const float* sinks, const void* gate, int ld_gate, cudaStream_t stream) {
+                                    const float* sinks, const void* gate, int ld_gate, float softcap, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
+    if (!(softcap >= 0.f)) return b200::kErrBadArgument;
     if (keep_first < 0 || (keep_first > 0 && window <= 0)) return b200::kErrBadArgument;
     if (chunk < 0 || (chunk > 0 && (window > 0 || keep_first > 0))) return b200::kErrBadArgument;
-    const b200::AttentionTerms terms = {keep_first, chunk, slopes, sinks, gate, ld_gate};
+    const b200::AttentionTerms terms = {keep_first, chunk, slopes, sinks, gate, ld_gate, softcap};
     if (n_splits < 1 || n_splits > 64 || (n_splits > 1 && scratch == nullptr)) return b200::kErrBadArgument;
     if (head_dim % 16 != 0 || head_dim < 16 || head_dim > 32 * b200::kMaxDimBlocks) return b200::kErrUnsupportedSize;
     if (n_kv_heads <= 0 || n_heads % n_kv_heads != 0) return b200::kErrBadArgument;

@@ -15,7 +15,7 @@
 // keep_first positions stay visible (their blocks of keys are walked ahead of the window's); a distance penalty
 // slopes[h] * (position - key) taken off every score, in 32 bits; a sink per head whose exponential joins the
 // denominator (every row's running maximum and sum start at (sinks[h], 1)); a gate per (token, head): the output is
-// multiplied by sigmoid(gate).
+// multiplied by sigmoid(gate); a soft cap: score <- softcap * tanh(score / softcap), before the penalty.
 //
 // A further mask (PrefillTerms.chunk): positions are cut into runs of `chunk`, counted from position 0, and i sees j <= i
 // of its own run only.
@@ -32,6 +32,7 @@ struct PrefillTerms {
     const float* sinks;            // [n_heads] or null
     const __nv_bfloat16* gate;     // [T][ld_gate], column h, or null
     int ld_gate;
+    float softcap;                 // 0: none
 };
 
 constexpr int kPrefillWarps = 4;
@@ -115,6 +116,8 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_row_stride, 
     const float scale_log2 = 1.4426950408889634f / sqrtf((float)D);  // log2(e) / sqrt(d)
     // scores stay in units of q.k until the exponential: the penalty per position and the sink are carried into them
     const float slope_qk = terms.slopes ? terms.slopes[head] * sqrtf((float)D) : 0.f;
+    // the cap in units of q.k, and what takes such a score to 2 log2(e) s / cap
+    const float cap_qk = terms.softcap * sqrtf((float)D), cap_log2 = terms.softcap > 0.f ? 2.885390081777927f / cap_qk : 0.f;
     if (terms.sinks) {
         const float sink_qk = terms.sinks[head] * sqrtf((float)D);
 #pragma unroll
@@ -167,6 +170,12 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_row_stride, 
                     mma_pf(s[i], ql[mt][kb].x, qh[mt][kb].x, ql[mt][kb].y, qh[mt][kb].y, kf[i][kb].x, kf[i][kb].y);
                     mma_pf(s[i], ql[mt][kb].z, qh[mt][kb].z, ql[mt][kb].w, qh[mt][kb].w, kf[i][kb].z, kf[i][kb].w);
                 }
+            }
+            if (terms.softcap > 0.f) {
+#pragma unroll
+                for (int i = 0; i < 4; ++i)
+#pragma unroll
+                    for (int c = 0; c < 4; ++c) s[i][c] = soft_capped_fast(s[i][c], cap_qk, cap_log2);
             }
             // scores stay in units of q.k; exp((s - m) / sqrt(d)) is evaluated as exp2((s - m) * scale_log2)
             float bm[2] = {-INFINITY, -INFINITY};
@@ -265,12 +274,13 @@ extern "C" int b200_attention_prefill(const void* q, int q_row_stride, void* out
                                       const int* kv_lens, const int* page_table, int table_stride, const void* k_pool,
                                       const void* v_pool, int n_seqs, int max_q_len, int n_heads, int n_kv_heads,
                                       int head_dim, int window, int keep_first, int chunk, const float* slopes, const float* sinks,
-                                      const void* gate, int ld_gate, cudaStream_t stream) {
+                                      const void* gate, int ld_gate, float softcap, cudaStream_t stream) {
     using namespace b200;
     if (n_seqs <= 0 || max_q_len <= 0) return 0;
+    if (!(softcap >= 0.f)) return kErrBadArgument;
     if (keep_first < 0 || (keep_first > 0 && window <= 0)) return kErrBadArgument;
     if (chunk < 0 || (chunk > 0 && (window > 0 || keep_first > 0))) return kErrBadArgument;
-    const PrefillTerms terms = {keep_first, chunk, slopes, sinks, (const __nv_bfloat16*)gate, ld_gate};
+    const PrefillTerms terms = {keep_first, chunk, slopes, sinks, (const __nv_bfloat16*)gate, ld_gate, softcap};
     if (n_kv_heads <= 0 || n_heads % n_kv_heads != 0) return kErrBadArgument;
     if (head_dim % 32 != 0 || head_dim < 32 || head_dim > 128 || q_row_stride % 8 != 0) return kErrUnsupportedSize;
     if (n_seqs > 65535 || n_heads > 65535) return kErrUnsupportedSize;

@@ -16,7 +16,9 @@
 //
 // The single-tile kernel takes a window, or `chunk` (positions cut into runs counted from position 0, i sees j <= i of its
 // own run), and a sink per head: a key without a value whose exponential joins the row's sum when the row is finished (the
-// running reference maximum is only a reference, so the sink need not take part in it).
+// running reference maximum is only a reference, so the sink need not take part in it).  Both kernels take a sink and, compiled in
+// for the mixers that have them (FaTerms), a soft cap on the scores and a gate per (token, head): the output is multiplied by
+// sigmoid(gate).  The cap is monotone, so a block's maximum is found before it.
 //
 // Roles (320 threads): warp 0 lane 0 issues TMA; warp 1 lane 0 issues MMAs (warp 1 owns the 256 TMEM
 // columns: S 128, O head_dim); warps 2-9 are the softmax (two threads per query row) and the epilogue.  Every mbarrier wait is bounded;
@@ -31,6 +33,15 @@ constexpr int kFaThreads = 320;  // TMA warp, MMA warp, eight softmax warps
 constexpr int kFaRows = 128, kFaKeys = 128;
 
 __device__ int g_fa_status = 0;
+
+struct FaTerms {
+    float softcap;                 // score <- softcap * tanh(score / softcap); 0: none
+    const __nv_bfloat16* gate;     // [T][ld_gate], column h, before its sigmoid; or null
+    int ld_gate;
+};
+__device__ __forceinline__ float gate_factor(const FaTerms& terms, size_t token, int head) {
+    return terms.gate ? 1.0f / (1.0f + expf(-__bfloat162float(terms.gate[token * terms.ld_gate + head]))) : 1.0f;
+}
 
 // Operand tiles are stored as "atoms" of 64 elements (128 bytes, one swizzle span) along the contraction:
 // Q and K as D/64 atoms of 128 rows, V^T as one atom of D rows per page, P as two atoms of 128 rows.
@@ -95,13 +106,13 @@ __device__ __forceinline__ void zero_values_beyond_end(__nv_bfloat16* v0, __nv_b
     }
 }
 
-template <int D>
+template <int D, bool TERMS>
 __global__ void __launch_bounds__(kFaThreads, D == 64 ? 2 : 1)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                             const __grid_constant__ CUtensorMap map_v, __nv_bfloat16* __restrict__ out,
                             const int* __restrict__ cu_seqlens, const int* __restrict__ kv_lens,
                             const int* __restrict__ page_table, int table_stride, int n_heads, int n_kv_heads,
-                            int window, int chunk, const float* __restrict__ sinks, int k_rows_total, int v_rows_total) {
+                            int window, int chunk, const float* __restrict__ sinks, int k_rows_total, int v_rows_total, FaTerms terms) {
     // Two CTAs share an SM only if each stays within 113 KB, which leaves no room for an alignment pad: the
     // dynamic shared memory of a kernel without static shared memory starts at the CTA's window, 1024-aligned;
     // if it ever does not, the kernel records that and leaves.
@@ -218,6 +229,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         const uint32_t lane_base = (uint32_t)(quarter * 32) << 16;
         const int pos = start + q0 + min(r, rows_here - 1);  // rows past the end mirror the last one (never stored)
         const float scale_log2 = 1.4426950408889634f / sqrtf((float)D);
+        // the cap in units of q.k, and what takes such a score to 2 log2(e) score / cap
+        const float cap_qk = TERMS ? terms.softcap * sqrtf((float)D) : 0.f, cap_log2 = TERMS && cap_qk > 0.f ? 2.885390081777927f / cap_qk : 0.f;
         float m_ref = -INFINITY, l = 0.f;  // reference maximum (units of q.k); this thread's share of the running sum
         bool ok = true;
         int it = 0;
@@ -251,6 +264,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             sm.row_max[half][r] = __float2bfloat16_rn(m_blk);
             asm volatile("bar.sync 1, 256;" ::: "memory");
             m_blk = fmaxf(__bfloat162float(sm.row_max[0][r]), __bfloat162float(sm.row_max[1][r]));
+            if (TERMS && cap_qk > 0.f && m_blk > -INFINITY) m_blk = soft_capped_fast(m_blk, cap_qk, cap_log2);
             // the reference maximum moves only when the block exceeds it by more than 2^8 after scaling
             const bool move = m_blk > m_ref && (m_ref == -INFINITY || (m_blk - m_ref) * scale_log2 > 8.f);
             if (__any_sync(0xffffffffu, move)) {
@@ -276,6 +290,10 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             for (int c = 0; c < 2; ++c) {
                 float v[32];
                 tmem_ld32(tmem_s + lane_base + half * 64 + c * 32, v);
+                if (TERMS && cap_qk > 0.f) {
+#pragma unroll
+                    for (int j = 0; j < 32; ++j) v[j] = soft_capped_fast(v[j], cap_qk, cap_log2);
+                }
                 uint32_t pk[16];
                 float l0 = 0.f, l1 = 0.f;
 #pragma unroll
@@ -328,7 +346,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         asm volatile("bar.sync 1, 256;" ::: "memory");
         if (ok) {
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-            const float inv_l = 1.0f / sm.row_sum[r];
+            const float inv_l = (TERMS && r < rows_here ? gate_factor(terms, (size_t)tok0 + q0 + r, head) : 1.0f) / sm.row_sum[r];
             __nv_bfloat16* orow = out + ((size_t)(tok0 + q0 + r) * n_heads + head) * D;
 #pragma unroll 1
             for (int c0 = half * (D / 2); c0 < (half + 1) * (D / 2); c0 += 32) {
@@ -458,13 +476,13 @@ __device__ __forceinline__ void umma_bf16_a_tmem(uint32_t tmem_d, uint32_t tmem_
 // another in one stream.
 __device__ unsigned int g_pair_ctl[4];
 
-template <int D>
+template <int D, bool TERMS>
 __global__ void __launch_bounds__(kPairThreads, 1)
 attention_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                               const __grid_constant__ CUtensorMap map_v, __nv_bfloat16* __restrict__ out,
                               const int* __restrict__ cu_seqlens, const int* __restrict__ kv_lens,
                               const int* __restrict__ page_table, int table_stride, int n_heads, int n_kv_heads,
-                              int k_rows_total, int v_rows_total, int n_seqs, int n_pairs) {
+                              int k_rows_total, int v_rows_total, int n_seqs, int n_pairs, const float* __restrict__ sinks, FaTerms terms) {
     static_assert(D == 64 || D == 128, "the pair kernel is laid out for head_dim 64 and 128");
     // Tensor memory, 512 columns.  Tile t: S in columns 128 t, O in 256 + D t.  P (bfloat16 pairs, 64 columns): with
     // head_dim 64 in columns 384 + 64 t; with head_dim 128 nothing is left, so P overwrites the first half of S, which
@@ -646,6 +664,7 @@ attention_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const _
                 const int pos = p_first + min(r, max(rows_t, 1) - 1);  // rows past the end mirror the last one (never stored)
                 const float scale_log2 = 1.4426950408889634f / sqrtf((float)D);
                 const uint32_t tmem_s = tmem + 128 * t, tmem_o = tmem + 256 + D * t, tmem_p = D == 64 ? tmem + 384 + 64 * t : tmem_s;
+                const float cap_qk = TERMS ? terms.softcap * sqrtf((float)D) : 0.f, cap_log2 = TERMS && cap_qk > 0.f ? 2.885390081777927f / cap_qk : 0.f;
                 float m_ref = -INFINITY, l = 0.f;
                 bool ok = true;
                 for (int j = 0; j < nbt; ++j) {
@@ -682,6 +701,7 @@ attention_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const _
                                 m4[c] = max3(m4[c], __uint_as_float(sr[c][i]), __uint_as_float(sr[c][i + 1]));
                         m_blk = fmaxf(fmaxf(m4[0], m4[1]), fmaxf(m4[2], m4[3]));
                     }
+                    if (TERMS && cap_qk > 0.f && m_blk > -INFINITY) m_blk = soft_capped_fast(m_blk, cap_qk, cap_log2);
                     // the block before must have left P and O alone before either is touched (it has, long ago, as a rule)
                     if (j > 0) {
                         ok = mbar_wait(&sm.pv_done[t], (tile_blocks[t] + j - 1) & 1, abort_flag);
@@ -713,6 +733,12 @@ attention_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const _
                     if (!ok && lane == 0) { *abort_flag = 1; atomicCAS(&g_fa_status, 0, (19 << 8) | (t * 4 + quarter)); }
                     ok = __shfl_sync(0xffffffffu, ok ? 1 : 0, 0) != 0;
                     if (!ok) break;
+                    if (TERMS && cap_qk > 0.f) {
+#pragma unroll
+                        for (int c = 0; c < 4; ++c)
+#pragma unroll
+                            for (int i = 0; i < 32; ++i) sr[c][i] = __float_as_uint(soft_capped_fast(__uint_as_float(sr[c][i]), cap_qk, cap_log2));
+                    }
                     // probabilities as bfloat16 pairs into this row's lane of P: key k of the block in column k / 2
                     float l4[4] = {0.f, 0.f, 0.f, 0.f};
                     if (masked) {  // the few blocks on the diagonal: every key is compared with the row's position
@@ -799,7 +825,8 @@ attention_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const _
                     ok = __shfl_sync(0xffffffffu, ok ? 1 : 0, 0) != 0;
                     if (ok) {
                         asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-                        const float inv_l = 1.0f / l;
+                        if (TERMS && sinks != nullptr) l += ex2(sinks[head] * 1.4426950408889634f - (m_ref == -INFINITY ? 0.f : m_ref * scale_log2));
+                        const float inv_l = (TERMS && r < rows_t ? gate_factor(terms, (size_t)tok0 + q0 + kFaRows * t + r, head) : 1.0f) / l;
                         __nv_bfloat16* orow = out + ((size_t)(tok0 + q0 + kFaRows * t + r) * n_heads + head) * D;
 #pragma unroll 1
                         for (int c0 = 0; c0 < D; c0 += 32) {
@@ -875,33 +902,33 @@ extern "C" int b200_attention_prefill_tc_status() {
 }
 
 namespace b200 {
-template <int D>
+template <int D, bool TERMS>
 static int launch_fa(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, void* out, const int* cu_seqlens,
                      const int* kv_lens, const int* page_table, int table_stride, int n_seqs, int max_q_len, int n_heads,
-                     int n_kv_heads, int window, int chunk, const float* sinks, int k_rows, int v_rows, cudaStream_t stream) {
+                     int n_kv_heads, int window, int chunk, const float* sinks, int k_rows, int v_rows, FaTerms terms, cudaStream_t stream) {
     static_assert(D != 64 || sizeof(FaSmem<64>) <= 113 * 1024, "two CTAs per SM need at most 113 KB each");
     const size_t smem = sizeof(FaSmem<D>);
     static bool configured = false;
     if (!configured) {
-        if (cudaFuncSetAttribute(attention_prefill_tc_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
+        if (cudaFuncSetAttribute(attention_prefill_tc_kernel<D, TERMS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
             return (int)cudaGetLastError();
         configured = true;
     }
     dim3 grid((max_q_len + kFaRows - 1) / kFaRows, n_heads, n_seqs);
-    return launch_pdl(attention_prefill_tc_kernel<D>, grid, dim3(kFaThreads), smem, stream, mq, mk, mv, (__nv_bfloat16*)out,
-                      cu_seqlens, kv_lens, page_table, table_stride, n_heads, n_kv_heads, window, chunk, sinks, k_rows, v_rows);
+    return launch_pdl(attention_prefill_tc_kernel<D, TERMS>, grid, dim3(kFaThreads), smem, stream, mq, mk, mv, (__nv_bfloat16*)out,
+                      cu_seqlens, kv_lens, page_table, table_stride, n_heads, n_kv_heads, window, chunk, sinks, k_rows, v_rows, terms);
 }
 }  // namespace b200
 
 namespace b200 {
-template <int D>
+template <int D, bool TERMS>
 static int launch_pair(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, void* out, const int* cu_seqlens,
                        const int* kv_lens, const int* page_table, int table_stride, int n_seqs, int max_q_len, int n_heads,
-                       int n_kv_heads, int k_rows, int v_rows, cudaStream_t stream) {
+                       int n_kv_heads, int k_rows, int v_rows, const float* sinks, FaTerms terms, cudaStream_t stream) {
     const size_t smem = sizeof(PairSmem<D>) + 1024;
     static bool configured = false;
     if (!configured) {
-        if (cudaFuncSetAttribute(attention_prefill_pair_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
+        if (cudaFuncSetAttribute(attention_prefill_pair_kernel<D, TERMS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
             return (int)cudaGetLastError();
         configured = true;
     }
@@ -914,23 +941,24 @@ static int launch_pair(const CUtensorMap& mq, const CUtensorMap& mk, const CUten
     if (e != cudaSuccess) return (int)e;
     if (dev < 0 || dev >= 64) return kErrBadArgument;
     const int grid = (int)(units < n_sms ? units : n_sms);  // one CTA per SM; each takes units until none are left
-    return launch_pdl(attention_prefill_pair_kernel<D>, dim3(grid), dim3(kPairThreads), smem, stream, mq, mk, mv,
+    return launch_pdl(attention_prefill_pair_kernel<D, TERMS>, dim3(grid), dim3(kPairThreads), smem, stream, mq, mk, mv,
                       (__nv_bfloat16*)out, cu_seqlens, kv_lens, page_table, table_stride, n_heads, n_kv_heads, k_rows, v_rows,
-                      n_seqs, n_pairs);
+                      n_seqs, n_pairs, sinks, terms);
 }
 }  // namespace b200
 
 // q: packed rows of q_row_stride elements whose first n_heads * head_dim are the rotated queries (n_rows of them);
 // k_pool [n_pages][n_kv_heads][64][head_dim], v_pool [n_pages][n_kv_heads][head_dim][64] (values transposed).
-// head_dim 64 or 128.  window, or chunk (not both; 0: none); sinks: float32 [n_heads] or null.
+// head_dim 64 or 128.  window, or chunk (not both; 0: none); sinks: float32 [n_heads] or null; gate bfloat16 [T][ld_gate] or null;
+// softcap 0: none.
 extern "C" int b200_attention_prefill_tc(const void* q, int q_row_stride, int n_rows, void* out, const int* cu_seqlens,
                                          const int* kv_lens, const int* page_table, int table_stride,
                                          const void* k_pool, const void* v_pool, int n_pages, int n_seqs, int max_q_len,
                                          int n_heads, int n_kv_heads, int head_dim, int window, int chunk, const float* sinks,
-                                         cudaStream_t stream) {
+                                         const void* gate, int ld_gate, float softcap, cudaStream_t stream) {
     using namespace b200;
     if (n_seqs <= 0 || max_q_len <= 0) return 0;
-    if (n_kv_heads <= 0 || n_heads % n_kv_heads != 0 || chunk < 0 || (chunk > 0 && window > 0)) return kErrBadArgument;
+    if (n_kv_heads <= 0 || n_heads % n_kv_heads != 0 || chunk < 0 || (chunk > 0 && window > 0) || !(softcap >= 0.f)) return kErrBadArgument;
     if ((head_dim != 64 && head_dim != 128) || q_row_stride % 8 != 0 ||
         (((uintptr_t)q | (uintptr_t)k_pool | (uintptr_t)v_pool | (uintptr_t)out) & 15))
         return kErrUnsupportedSize;
@@ -941,17 +969,22 @@ extern "C" int b200_attention_prefill_tc(const void* q, int q_row_stride, int n_
     if (!make_map_2d(&mq, q, n_rows, n_heads * head_dim, q_row_stride, 64, kFaRows) ||
         !make_map_2d(&mk, k_pool, k_rows, head_dim, head_dim, 64, 64) || !make_map_2d(&mv, v_pool, v_rows, 64, 64, 64, head_dim))
         return kErrUnsupportedSize;
+    const FaTerms terms = {softcap, (const __nv_bfloat16*)gate, ld_gate};
+    const bool more = softcap > 0.f || gate != nullptr;
+#define B200_GO(F, D, T, ...)                                                                                                  \
+    F<D, T>(mq, mk, mv, out, cu_seqlens, kv_lens, page_table, table_stride, n_seqs, max_q_len, n_heads, n_kv_heads, __VA_ARGS__, stream)
     // tiles in pairs when there are enough pairs to give every SM one (fewer: the single-tile kernel fills more SMs)
-    if (window <= 0 && chunk <= 0 && sinks == nullptr && (long long)((max_q_len + 2 * kFaRows - 1) / (2 * kFaRows)) * n_heads * n_seqs >= device_sm_count()) {
+    if (window <= 0 && chunk <= 0 && (long long)((max_q_len + 2 * kFaRows - 1) / (2 * kFaRows)) * n_heads * n_seqs >= device_sm_count()) {
         if (head_dim == 64)
-            return launch_pair<64>(mq, mk, mv, out, cu_seqlens, kv_lens, page_table, table_stride, n_seqs, max_q_len, n_heads,
-                                   n_kv_heads, (int)k_rows, (int)v_rows, stream);
-        return launch_pair<128>(mq, mk, mv, out, cu_seqlens, kv_lens, page_table, table_stride, n_seqs, max_q_len, n_heads,
-                                n_kv_heads, (int)k_rows, (int)v_rows, stream);
+            return more || sinks != nullptr ? B200_GO(launch_pair, 64, true, (int)k_rows, (int)v_rows, sinks, terms)
+                                            : B200_GO(launch_pair, 64, false, (int)k_rows, (int)v_rows, sinks, terms);
+        return more || sinks != nullptr ? B200_GO(launch_pair, 128, true, (int)k_rows, (int)v_rows, sinks, terms)
+                                        : B200_GO(launch_pair, 128, false, (int)k_rows, (int)v_rows, sinks, terms);
     }
     if (head_dim == 64)
-        return launch_fa<64>(mq, mk, mv, out, cu_seqlens, kv_lens, page_table, table_stride, n_seqs, max_q_len, n_heads,
-                             n_kv_heads, window, chunk, sinks, (int)k_rows, (int)v_rows, stream);
-    return launch_fa<128>(mq, mk, mv, out, cu_seqlens, kv_lens, page_table, table_stride, n_seqs, max_q_len, n_heads,
-                          n_kv_heads, window, chunk, sinks, (int)k_rows, (int)v_rows, stream);
+        return more ? B200_GO(launch_fa, 64, true, window, chunk, sinks, (int)k_rows, (int)v_rows, terms)
+                    : B200_GO(launch_fa, 64, false, window, chunk, sinks, (int)k_rows, (int)v_rows, terms);
+    return more ? B200_GO(launch_fa, 128, true, window, chunk, sinks, (int)k_rows, (int)v_rows, terms)
+                : B200_GO(launch_fa, 128, false, window, chunk, sinks, (int)k_rows, (int)v_rows, terms);
+#undef B200_GO
 }

@@ -70,6 +70,17 @@ __device__ __forceinline__ float block_max(float v, float* scratch) {
     return scratch[32];
 }
 
+// Attention scores under a soft cap, cap * tanh(s / cap), in 32 bits.  The first form calls the library's tanh; the second,
+// for kernels whose inner loops are their exponentials, takes tanh(x) = 1 - 2 / (e^(2x) + 1) with the hardware's power of two
+// (absolute error about 2^-22 of the cap).  `to_log2` is 2 log2(e) / cap.
+__device__ __forceinline__ float soft_capped(float s, float cap) { return cap * tanhf(s / cap); }
+__device__ __forceinline__ float soft_capped_fast(float s, float cap, float to_log2) {
+    float e, r;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(s * to_log2));
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(e + 1.f));
+    return cap - 2.f * cap * r;
+}
+
 inline int launch_status() { return (int)cudaPeekAtLastError(); }
 
 // SMs of the current device (asked once per device; 148, a B200's, only if the driver does not answer).

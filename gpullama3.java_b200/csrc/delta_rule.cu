@@ -27,6 +27,10 @@
 // skip = D), or a fixed decay per head (retention, lightning attention: g given, beta = 1, the keys and queries optionally
 // turned by their positions or passed through SiLU in 32 bits); linear_scan_prepare makes their rows.  causal_conv is the convolution in its general form: input and output
 // types of their own, an optional bias, SiLU or no activation, and optionally the input added to the result.
+//
+// It also runs a memory whose gates another kernel made (gated_scan): S <- g S + b k v^T per head and token with g and b of every
+// token given as logarithms and running maxima, and beside S a vector n that takes the keys alone (a column of values that are all
+// one, kept in its own place of the slot); the read-outs come with n . q behind them.
 #include "common.cuh"
 
 namespace b200 {
@@ -466,6 +470,62 @@ linear_scan_prepare_kernel(LinearPrepareArgs a) {
     }
 }
 
+// The rows of a memory with given gates: `gates` holds, in planes of [heads][T], what the gates kernel leaves (plane 1: the log
+// input gate i, 2: the running maximum m, 3: the log forget gate f), start_m [n_seqs][heads] the maximum before the step.  Decay
+// e^(f + m_(t-1) - m_t), write strength e^(i - m_t); behind the d_v values stands a one.
+struct GatedPrepareArgs {
+    const void* q;
+    int ld_q;
+    const void* k;
+    int ld_k;
+    const void* v;
+    int ld_v;
+    const float* gates;
+    const float* start_m;
+    const int* seq_ids;
+    const int* cu_seqlens;
+    float* rows;
+    int n_tokens, heads, d_k, d_v, d_pad, row;
+    float q_scale;
+};
+
+template <typename T>
+__global__ void __launch_bounds__(128)
+gated_scan_prepare_kernel(GatedPrepareArgs a) {
+    const long long unit = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);
+    const int lane = threadIdx.x & 31;
+    if (unit >= (long long)a.n_tokens * a.heads) return;
+    const size_t t = (size_t)(unit / a.heads);
+    const int h = (int)(unit % a.heads);
+    const T* qr = (const T*)a.q + t * a.ld_q + (size_t)h * a.d_k;
+    const T* kr = (const T*)a.k + t * a.ld_k + (size_t)h * a.d_k;
+    const T* vr = (const T*)a.v + t * a.ld_v + (size_t)h * a.d_v;
+    float* out = a.rows + ((size_t)h * a.n_tokens + t) * a.row;
+    const size_t plane = (size_t)a.heads * a.n_tokens;
+    const float* G = a.gates + (size_t)h * a.n_tokens + t;
+    const int seq = a.seq_ids[t];
+    const float m = G[2 * plane], before = (int)t == a.cu_seqlens[seq] ? a.start_m[(size_t)seq * a.heads + h] : *(G + 2 * plane - 1);
+    const float keep = expf(G[3 * plane] + before - m), take = expf(G[plane] - m);
+    float qk = 0.f;
+    for (int i = lane; i < a.d_pad; i += 32) {
+        const bool in = i < a.d_k;
+        const float qv = in ? to_f32<T>(qr[i]) * a.q_scale : 0.f, kv = in ? to_f32<T>(kr[i]) : 0.f;
+        qk += qv * kv;
+        out[i] = qv;
+        out[a.d_pad + i] = kv;
+        out[2 * a.d_pad + i] = in ? keep : 0.f;
+    }
+    qk = warp_sum(qk);
+    for (int j = lane; j < a.d_v; j += 32) out[3 * a.d_pad + j] = to_f32<T>(vr[j]);
+    if (lane == 0) {
+        float* behind = out + 3 * a.d_pad + a.d_v;
+        behind[0] = 1.f;
+        behind[1] = take;
+        behind[2] = qk;
+        behind[3] = 0.f;
+    }
+}
+
 struct ScanArgs {
     const float* rows;      // [heads, T, row] as delta_rule_prepare leaves them
     float* state;           // per slot: [heads][d_k][d_v]
@@ -474,6 +534,8 @@ struct ScanArgs {
     const int* cu_seqlens;
     float* out;             // [T, heads d_v] 32-bit
     int n_tokens, heads, d_k, d_v, row;
+    long long sum_off;      // >= 0: column d_v - 1 is a vector per head at slot + sum_off + h sum_stride, the others [d_k][d_v - 1] per head
+    int sum_stride;
 };
 
 __device__ __forceinline__ void copy_async_16(float* dst, const float* src) {
@@ -498,7 +560,10 @@ delta_rule_scan_kernel(ScanArgs a) {
     const bool live = col < a.d_v;
     const int v_at = 3 * dpad + min(col, a.d_v - 1), b_at = 3 * dpad + a.d_v;
     const int first = a.cu_seqlens[seq], n = a.cu_seqlens[seq + 1] - first;
-    float* S_g = a.state + (size_t)a.slots[seq] * a.slot_stride + (size_t)h * a.d_k * a.d_v;
+    const bool apart = a.sum_off >= 0, sum_col = apart && col == a.d_v - 1;
+    const int ld_s = sum_col ? 1 : apart ? a.d_v - 1 : a.d_v;
+    float* S_g = a.state + (size_t)a.slots[seq] * a.slot_stride +
+                 (sum_col ? (size_t)a.sum_off + (size_t)h * a.sum_stride : (size_t)h * a.d_k * ld_s + col);    // this column's row 0
     const float* rows = a.rows + ((size_t)h * a.n_tokens + first) * a.row;
 
     auto fetch = [&](int base, float* buf) {
@@ -514,7 +579,7 @@ delta_rule_scan_kernel(ScanArgs a) {
 #pragma unroll
     for (int i = 0; i < RPT; ++i) {
         const int rw = (i >> 2) * (4 * R) + 4 * r + (i & 3);
-        S[i] = (live && rw < a.d_k) ? S_g[(size_t)rw * a.d_v + col] : 0.f;
+        S[i] = (live && rw < a.d_k) ? S_g[(size_t)rw * ld_s] : 0.f;
     }
 
     fetch(0, smem);
@@ -570,7 +635,7 @@ delta_rule_scan_kernel(ScanArgs a) {
 #pragma unroll
     for (int i = 0; i < RPT; ++i) {
         const int rw = (i >> 2) * (4 * R) + 4 * r + (i & 3);
-        if (live && rw < a.d_k) S_g[(size_t)rw * a.d_v + col] = S[i];
+        if (live && rw < a.d_k) S_g[(size_t)rw * ld_s] = S[i];
     }
 }
 
@@ -772,7 +837,7 @@ extern "C" int b200_delta_rule_scan(const void* qkv, int ld_qkv, const void* bet
     const long long units = (long long)n_tokens * heads;
     B200_DISPATCH_DTYPE(dtype, T,
         b200::delta_rule_prepare_kernel<T><<<(unsigned)((units + 3) / 4), 128, 0, stream>>>(p));
-    b200::ScanArgs a = {scratch, state, (size_t)slot_stride, slots, cu_seqlens, out, n_tokens, heads, d_k, d_v, row};
+    b200::ScanArgs a = {scratch, state, (size_t)slot_stride, slots, cu_seqlens, out, n_tokens, heads, d_k, d_v, row, -1, 0};
     return b200::launch_scan_rows<false>(a, rpt, lanes, n_seqs, stream);
 }
 
@@ -800,6 +865,27 @@ extern "C" int b200_linear_scan(const void* q, int ld_q, const void* k, int ld_k
     const long long units = (long long)n_tokens * heads;
     B200_DISPATCH_DTYPE(dtype, T,
         b200::linear_scan_prepare_kernel<T><<<(unsigned)((units + 3) / 4), 128, 0, stream>>>(p));
-    b200::ScanArgs a = {scratch, state, (size_t)slot_stride, slots, cu_seqlens, out, n_tokens, heads, d_k, d_v, row};
+    b200::ScanArgs a = {scratch, state, (size_t)slot_stride, slots, cu_seqlens, out, n_tokens, heads, d_k, d_v, row, -1, 0};
+    return b200::launch_scan_rows<true>(a, rpt, lanes, n_seqs, stream);
+}
+
+// A memory with given gates over a packed step (see GatedPrepareArgs): out float32 [T, heads, d_v + 1], the read-outs with n . q
+// behind them; S at slot + 0, head h's n at slot + sum_off + h sum_stride.  scratch as b200_delta_rule_row(d_k, d_v + 1) says.
+extern "C" int b200_gated_scan(const void* q, int ld_q, const void* k, int ld_k, const void* v, int ld_v, const float* gates,
+                               const float* start_m, float* state, long long slot_stride, long long sum_off, int sum_stride,
+                               const int* slots, const int* seq_ids, const int* cu_seqlens, float* out, float* scratch, int dtype,
+                               int n_tokens, int n_seqs, int heads, int d_k, int d_v, float q_scale, cudaStream_t stream) {
+    if (n_seqs <= 0 || n_tokens <= 0) return 0;
+    if (heads < 1 || d_k < 1 || d_v < 1 || n_seqs > 65535 || heads > 65535 || !scratch || sum_off < 0) return b200::kErrBadArgument;
+    int rpt = 0, lanes = 0;
+    if (!b200_delta_rule_plan(d_k, &rpt, &lanes)) return b200::kErrUnsupportedSize;
+    const int row = b200_delta_rule_row(d_k, d_v + 1);
+    if ((uintptr_t)scratch % 16) return b200::kErrBadArgument;
+    b200::GatedPrepareArgs p = {q, ld_q, k, ld_k, v, ld_v, gates, start_m, seq_ids, cu_seqlens, scratch, n_tokens, heads, d_k, d_v,
+                                rpt * lanes, row, q_scale};
+    const long long units = (long long)n_tokens * heads;
+    B200_DISPATCH_DTYPE(dtype, T,
+        b200::gated_scan_prepare_kernel<T><<<(unsigned)((units + 3) / 4), 128, 0, stream>>>(p));
+    b200::ScanArgs a = {scratch, state, (size_t)slot_stride, slots, cu_seqlens, out, n_tokens, heads, d_k, d_v + 1, row, sum_off, sum_stride};
     return b200::launch_scan_rows<true>(a, rpt, lanes, n_seqs, stream);
 }

@@ -9,7 +9,8 @@
 //   depth_average      level[n] = x ;  x <- sum_(j <= n) c[j] level[j] ;  xc = x (optional): every layer's result is
 //                      kept for the pass, and what the next layer reads is a learned mix of all of them
 //   cast_rows          xc = x in the run's type (what a product over the stream itself reads)
-//   bias_act_rows      u <- act(u + bias) in place on a product's result; act: the square of max(., 0)
+//   bias_act_rows      act(u + bias) of a product's result, in place or into columns of another buffer; act: the square of max(., 0);
+//                      optionally times the sigmoid of one number per token
 //   token_gate_rows    g[t, j] = gelu_tanh(a[t, j]) * table[token[t], j]: a few numbers per token id that the stream gates
 //
 // Every kernel here is launched with programmatic dependent launch and waits for its predecessor before it touches memory.
@@ -300,15 +301,25 @@ cast_rows_kernel(const float* __restrict__ x, TR* __restrict__ xc, size_t total)
         xc[i] = from_f32<TR>(x[i]);
 }
 
-template <typename TR>
+template <typename TR, int VEC>
 __global__ void __launch_bounds__(256)
-bias_act_rows_kernel(TR* __restrict__ u, int ld, const float* __restrict__ bias, int n) {
+bias_act_rows_kernel(const TR* u, int ld, const float* __restrict__ bias, TR* out, int ld_out, const TR* gate, int ld_gate, int n) {
     pdl_launch_dependents();
     pdl_wait();
-    TR* ur = u + (size_t)blockIdx.x * ld;
-    for (int e = blockIdx.y * blockDim.x + threadIdx.x; e < n; e += gridDim.y * blockDim.x) {
-        const float z = fmaxf(to_f32<TR>(ur[e]) + (bias ? bias[e] : 0.f), 0.f);
-        ur[e] = from_f32<TR>(z * z);
+    const TR* ur = u + (size_t)blockIdx.x * ld;
+    TR* o = out + (size_t)blockIdx.x * ld_out;
+    const float g = gate ? 1.0f / (1.0f + expf(-to_f32<TR>(gate[(size_t)blockIdx.x * ld_gate]))) : 1.0f;
+    for (int e = (blockIdx.y * blockDim.x + threadIdx.x) * VEC; e < n; e += gridDim.y * blockDim.x * VEC) {
+        alignas(16) TR x[VEC];
+        if constexpr (VEC > 1) *reinterpret_cast<uint4*>(x) = *reinterpret_cast<const uint4*>(ur + e);
+        else x[0] = ur[e];
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) {
+            const float z = fmaxf(to_f32<TR>(x[i]) + (bias ? bias[e + i] : 0.f), 0.f);
+            x[i] = from_f32<TR>(z * z * g);
+        }
+        if constexpr (VEC > 1) *reinterpret_cast<uint4*>(o + e) = *reinterpret_cast<uint4*>(x);
+        else o[e] = x[0];
     }
 }
 
@@ -408,14 +419,22 @@ extern "C" int b200_cast_rows(const float* x, void* xc, int dtype, long long tot
 }
 
 // act 0: max(u + bias, 0)^2
-extern "C" int b200_bias_act_rows(void* u, int ld, int dtype, const float* bias, int n_tokens, int n, int act,
-                                  cudaStream_t stream) {
+// out [T][ld_out] may be u itself, or columns of a wider buffer; gate [T][ld_gate] (null: none): column 0, before its sigmoid, is a
+// factor on the token's row.
+extern "C" int b200_bias_act_rows(const void* u, int ld, int dtype, const float* bias, void* out, int ld_out, const void* gate, int ld_gate,
+                                  int n_tokens, int n, int act, cudaStream_t stream) {
     if (act != 0) return b200::kErrBadArgument;
     if (n_tokens <= 0 || n <= 0) return 0;
-    const int ny = (n + 1023) / 1024;
+    const int vec = dtype == b200::kF32 ? 4 : 8;
+    const bool wide = n % vec == 0 && ld % vec == 0 && ld_out % vec == 0 && (((uintptr_t)u | (uintptr_t)out) & 15) == 0;
+    const int per = 256 * (wide ? vec : 1), ny = (n + per - 1) / per;
+    const dim3 grid(n_tokens, ny > 64 ? 64 : ny);
     B200_DISPATCH_DTYPE(dtype, T,
-        return b200::launch_pdl(b200::bias_act_rows_kernel<T>, dim3(n_tokens, ny > 64 ? 64 : ny), dim3(256), 0, stream, (T*)u, ld,
-                                bias, n));
+        if (wide)
+            return b200::launch_pdl(b200::bias_act_rows_kernel<T, 16 / (int)sizeof(T)>, grid, dim3(256), 0, stream, (const T*)u, ld, bias,
+                                    (T*)out, ld_out, (const T*)gate, ld_gate, n);
+        return b200::launch_pdl(b200::bias_act_rows_kernel<T, 1>, grid, dim3(256), 0, stream, (const T*)u, ld, bias, (T*)out, ld_out,
+                                (const T*)gate, ld_gate, n));
     return 0;
 }
 

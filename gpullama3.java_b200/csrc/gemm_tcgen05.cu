@@ -90,6 +90,7 @@ struct RopeEpilogue {
     float gate_limit, gate_slope;
     const float* bias;         // [N] float32 or null: joins every sum before the store, residual and gated epilogues (not EPI 3)
     int silu_cols;             // EPI 0: columns below this one are stored as silu(sum) (projections that are used activated)
+    int squared_relu;          // EPI 0: 1: every column is stored as max(sum, 0)^2
 };
 
 __device__ __forceinline__ float gated_clamped(float gate, float up, float limit, float slope) {
@@ -235,6 +236,13 @@ __device__ __forceinline__ void epilogue_tile(uint32_t acc, int quarter, int lan
             } else {
 #pragma unroll
                 for (int j = 0; j < 32; ++j) if (n0 + c0 + j < rope.silu_cols) v[j] = v[j] / (1.0f + expf(-v[j]));
+            }
+        }
+        if (EPI == 0 && rope.squared_relu) {
+#pragma unroll
+            for (int j = 0; j < 32; ++j) {
+                const float z = fmaxf(v[j], 0.f);
+                v[j] = z * z;
             }
         }
         if (EPI == 1 && reduce_c) {
@@ -1151,7 +1159,8 @@ static int launch_grouped(const void* A, int lda, const void* W, void* C, int ld
 
 // One product per group over the group's run of rows (see gemm_tcgen05_grouped_kernel): A [total_rows, K] bfloat16, W
 // [n_groups, N, K] bfloat16 and dense, offsets [n_groups + 1] on the device, C [total_rows, N] float32 (epilogue 0) or
-// [total_rows, N / 2] bfloat16 (gated epilogues 2, 3, 4 with gate_limit and gate_slope).
+// [total_rows, N / 2] bfloat16 (gated epilogues 2, 3, 4 with gate_limit and gate_slope); epilogue 5: C [total_rows, N] bfloat16 holds
+// max(sum, 0)^2.
 extern "C" int b200_gemm_tcgen05_grouped(const void* A, int lda, const void* W, void* C, int c_dtype, int ldc, int total_rows,
                                          int N, int K, int n_groups, const int* offsets, int epilogue, float gate_limit,
                                          float gate_slope, cudaStream_t stream) {
@@ -1167,6 +1176,12 @@ extern "C" int b200_gemm_tcgen05_grouped(const void* A, int lda, const void* W, 
         gated.gate_slope = gate_slope;
         if (N >= 1024) return launch_grouped<256, 4, 2, __nv_bfloat16>(A, lda, W, C, ldc, total_rows, N, K, n_groups, offsets, stream, gated);
         return launch_grouped<128, 6, 2, __nv_bfloat16>(A, lda, W, C, ldc, total_rows, N, K, n_groups, offsets, stream, gated);
+    }
+    if (epilogue == 5) {
+        if (c_dtype != kBF16) return kErrBadArgument;
+        gated.squared_relu = 1;
+        if (N >= 1024) return launch_grouped<256, 4, 0, __nv_bfloat16>(A, lda, W, C, ldc, total_rows, N, K, n_groups, offsets, stream, gated);
+        return launch_grouped<128, 6, 0, __nv_bfloat16>(A, lda, W, C, ldc, total_rows, N, K, n_groups, offsets, stream, gated);
     }
     if (epilogue != 0 || c_dtype != kF32) return kErrBadArgument;
     if (N >= 1024) return launch_grouped<256, 4, 0, float>(A, lda, W, C, ldc, total_rows, N, K, n_groups, offsets, stream, gated);

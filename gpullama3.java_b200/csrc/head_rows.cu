@@ -15,7 +15,8 @@
 //                                                   pairs, the angle, its cosine and sine in 32 bits; `mul` then also carries
 //                                                   a factor on cosine and sine)
 //     or, over halves: (z[i], z[i + n]) <- turned by position * inv_freq[f + i] for i < n, the columns from 2 n on as they
-//                                                   are; every segment with frequencies (f) and pairs (n) of its own
+//                                                   are; every segment with frequencies (f), pairs (n) and a factor on cosine
+//                                                   and sine of its own
 // A segment's rows need not lie back to back (`src_stride`: a part of every head of a wider projection; 0 as a stride:
 // every row reads the same numbers, one row shared by all heads) nor be written back to back (`dst_stride`), and a row may
 // fill only some columns of a cache row (`dst_off` columns in, `cache_dim` the cache's row size), so that two segments can
@@ -31,7 +32,7 @@
 namespace b200 {
 
 constexpr int kRowSegments = 6;
-constexpr int kSegmentWords = 20;   // 32-bit words of one segment record at the C interface (19 used)
+constexpr int kSegmentWords = 20;   // 32-bit words of one segment record at the C interface
 constexpr int kRowThreads = 128;
 
 struct RowSegment {
@@ -48,7 +49,8 @@ struct RowSegment {
     int src_stride;   // numbers between two rows of the source (-1: d)
     int dst_stride;   // numbers between two rows written to dst (-1: d_pad)
     int cache_dim;    // row size of the cache the segment goes into (-1: d_pad); the segment starts dst_off columns in
-    int pairs, freq_off;   // rotate 2 alone reads these
+    int pairs, freq_off;   // rotate 2 alone reads these, and
+    float turn_mul;        // the factor on its cosines and sines
     int lead;         // zeros written in front of the row: of the d_pad numbers the first `lead` are zero, then the d, then zeros
 };
 struct MixSource {
@@ -123,6 +125,7 @@ __device__ __forceinline__ void head_row(const T* __restrict__ src, int ld_src, 
             const float u = value(i), v = value(i + n);
             float sn, cs;
             sincosf(pos * cache.inv_freq[g.freq_off + i], &sn, &cs);
+            sn *= g.turn_mul; cs *= g.turn_mul;
             o[(size_t)i * step] = from_f32<T>(u * cs - v * sn);
             o[(size_t)(i + n) * step] = from_f32<T>(v * cs + u * sn);
         }
@@ -262,7 +265,7 @@ head_rows_tile_kernel(const T* __restrict__ src, int ld_src, T* __restrict__ dst
                 const float2* a = turn + tt * n_freqs + g.freq_off + c0;
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
-                    const float u = z[e], v = z[4 + e];
+                    const float u = z[e] * g.turn_mul, v = z[4 + e] * g.turn_mul;
                     z[e] = u * a[e].x - v * a[e].y;
                     z[4 + e] = v * a[e].x + u * a[e].y;
                 }
@@ -335,8 +338,8 @@ head_rows_token_kernel(const T* __restrict__ src, int ld_src, T* __restrict__ ds
 }  // namespace b200
 
 // `segments`: n_segments records of twenty 32-bit words each (src_off, n_rows, d, dst_off, d_pad, bias_off, norm,
-// weight_off, mul as float bits, target, weight_per_row, mix_off, rotate, src_stride, dst_stride, cache_dim, lead, pairs, freq_off; the rest
-// unused), read on the host.  Segments with a cache target need positions, seq_ids,
+// weight_off, mul as float bits, target, weight_per_row, mix_off, rotate, src_stride, dst_stride, cache_dim, lead, pairs, freq_off,
+// turn_mul as float bits), read on the host.  Segments with a cache target need positions, seq_ids,
 // page_table and the pools; their n_rows is the number of kv heads of the cache entry and d_pad its head size.
 extern "C" int b200_head_rows(const void* src, int ld_src, void* dst, int ld_dst, int dtype, const float* bias,
                               const float* weight, const int* segments, int n_segments, int n_tokens, float eps,
@@ -360,6 +363,8 @@ extern "C" int b200_head_rows(const void* src, int ld_src, void* dst, int ld_dst
         g.mix_off = p[11];
         g.rotate = p[12]; g.src_stride = p[13]; g.dst_stride = p[14]; g.cache_dim = p[15]; g.lead = p[16];
         g.pairs = p[17]; g.freq_off = p[18];
+        u.i = p[19];
+        g.turn_mul = u.f;
         if (g.lead < 0 || g.lead + g.d > g.d_pad) return b200::kErrBadArgument;
         if (g.rotate && (!inv_freq || !positions || g.mix_off >= 0)) return b200::kErrBadArgument;
         if (g.rotate == 1 && g.d % 2) return b200::kErrBadArgument;

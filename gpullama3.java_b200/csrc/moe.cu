@@ -1,16 +1,18 @@
 // A routed feed-forward (mixture of experts): the router, and the experts for steps of few tokens.
 //
-//   moe_route     per token: logits z = W_r h (+ bias) (32-bit sums, W_r kept in 32 bits), scores s = softmax(z) over all experts.
+//   moe_route     per token: logits z = W_r h (+ bias) (32-bit sums, W_r kept in 32 bits), scores s = softmax(z) over all experts, or
+//                 s = sigmoid(z) of each; experts are chosen by s (+ correction), weighed by s alone.
 //                 The experts form `n_groups` equal groups of neighbours; a group's score is its best expert's score, and
 //                 only experts of the `keep_groups` best groups may be chosen.  The `top` allowed experts with the
 //                 largest scores are chosen (ties: the lower index); their weights are their scores over the sum of
-//                 the chosen scores (+ norm_eps).  A CTA per token.
+//                 the chosen scores (+ norm_eps), times `scale`.  A CTA per token.
 //   moe_group     the (token, choice) pairs ordered by expert (counting sort; the order inside an expert's run does not
 //                 change any result, a row of a product depends on its own input row only).
 //   moe_rows      steps of few tokens: every expert's rows as a weight-streaming product whose row counts are read on
 //                 the device, so a decode step's launches do not depend on the routing; an expert's weights are read once
 //                 for all tokens that chose it (in groups of eight), an expert nobody chose is not read.  Used twice:
-//                 gate and up rows with the gated epilogue (the same codes as the products' gated epilogues), then down.
+//                 gate and up rows with the gated epilogue (the same codes as the products' gated epilogues), or up rows alone with the
+//                 square of max(., 0), then down.
 //                 bfloat16 runs on the tensor cores (mma.sync, the eight rows as a tile's columns), float32 on the FMA pipe.
 //   moe_gather    prompts: the inputs copied into the order of their experts, so that each expert's rows are one dense
 //                 product for the tensor-core kernels.
@@ -73,6 +75,9 @@ struct RouteArgs {
     int n_tokens, width, n_experts, n_groups, keep_groups, top;
     float norm_eps;
     const float* bias;      // [n_experts] added to the logits, or null
+    int sigmoid_scores;     // 1: s = sigmoid(z)
+    const float* correction;   // [n_experts] added to the scores for the choice alone, or null
+    float scale;
 };
 
 constexpr int kRouteThreads = 128;
@@ -85,8 +90,9 @@ moe_route_kernel(RouteArgs a) {
     extern __shared__ float smem[];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     float* x = smem;                       // the token's input
-    float* s = x + a.width;                // logits, then scores; chosen or barred ones turn negative
-    float* gs = s + a.n_experts;           // group scores
+    float* s = x + a.width;                // logits, then scores
+    float* c = s + a.n_experts;            // what the choice goes by; -inf: chosen already, or barred
+    float* gs = c + a.n_experts;           // group scores
     const int t = blockIdx.x;
     const T* hr = (const T*)a.h + (size_t)t * a.ld_h;
     for (int k = threadIdx.x; k < a.width; k += kRouteThreads) x[k] = to_f32<T>(hr[k]);
@@ -99,14 +105,16 @@ moe_route_kernel(RouteArgs a) {
     }
     __syncthreads();
     if (warp != 0) return;
-    float m = -INFINITY;
-    for (int e = lane; e < a.n_experts; e += 32) m = fmaxf(m, s[e]);
-    m = warp_max(m);
-    float sum = 0.f;
-    for (int e = lane; e < a.n_experts; e += 32) sum += expf(s[e] - m);
-    sum = warp_sum(sum);
+    float m = -INFINITY, sum = 0.f;
+    if (!a.sigmoid_scores) {
+        for (int e = lane; e < a.n_experts; e += 32) m = fmaxf(m, s[e]);
+        m = warp_max(m);
+        for (int e = lane; e < a.n_experts; e += 32) sum += expf(s[e] - m);
+        sum = warp_sum(sum);
+    }
     for (int e = lane; e < a.n_experts; e += 32) {
-        s[e] = expf(s[e] - m) / sum;
+        s[e] = a.sigmoid_scores ? 1.0f / (1.0f + expf(-s[e])) : expf(s[e] - m) / sum;
+        c[e] = s[e] + (a.correction ? a.correction[e] : 0.f);
         if (a.scores) a.scores[(size_t)t * a.n_experts + e] = s[e];
     }
     __syncwarp();
@@ -114,14 +122,14 @@ moe_route_kernel(RouteArgs a) {
     const int per = a.n_experts / a.n_groups;
     if (a.keep_groups < a.n_groups) {
         for (int g = lane; g < a.n_groups; g += 32) {
-            float best = -1.f;
-            for (int i = 0; i < per; ++i) best = fmaxf(best, s[g * per + i]);
+            float best = -INFINITY;
+            for (int i = 0; i < per; ++i) best = fmaxf(best, c[g * per + i]);
             gs[g] = best;
         }
         __syncwarp();
         for (int r = 0; r < a.keep_groups; ++r) {
-            float bv = -2.f;
-            int bi = 0x7fffffff;
+            float bv = -INFINITY;
+            int bi = a.n_groups - 1;
             for (int g = lane; g < a.n_groups; g += 32)
                 if (gs[g] > bv) { bv = gs[g]; bi = g; }
 #pragma unroll
@@ -130,11 +138,11 @@ moe_route_kernel(RouteArgs a) {
                 const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
                 if (ov > bv || (ov == bv && oi < bi)) { bv = ov; bi = oi; }
             }
-            if (lane == 0) gs[bi] = -3.f;    // taken
+            if (lane == 0) gs[bi] = -INFINITY;    // taken
             __syncwarp();
         }
         for (int e = lane; e < a.n_experts; e += 32)
-            if (gs[e / per] != -3.f) s[e] = -1.f - s[e];   // barred: negative
+            if (gs[e / per] != -INFINITY) c[e] = -INFINITY;   // barred
         __syncwarp();
     }
     // the `top` best allowed experts, one after the other
@@ -142,24 +150,24 @@ moe_route_kernel(RouteArgs a) {
     float my_w = 0.f;
     int my_e = 0;
     for (int r = 0; r < a.top; ++r) {
-        float bv = -1.f;
-        int bi = 0x7fffffff;
+        float bv = -INFINITY;
+        int bi = a.n_experts - 1;      // (stays inside the experts even if no score compares: logits that are not numbers)
         for (int e = lane; e < a.n_experts; e += 32)
-            if (s[e] > bv) { bv = s[e]; bi = e; }
+            if (c[e] > bv) { bv = c[e]; bi = e; }
 #pragma unroll
         for (int o = 16; o > 0; o >>= 1) {
             const float ov = __shfl_xor_sync(0xffffffffu, bv, o);
             const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
             if (ov > bv || (ov == bv && oi < bi)) { bv = ov; bi = oi; }
         }
-        chosen_sum += bv;
-        if (lane == r) { my_w = bv; my_e = bi; }
-        if (lane == 0) s[bi] = -1.f;
+        chosen_sum += s[bi];
+        if (lane == r) { my_w = s[bi]; my_e = bi; }
+        if (lane == 0) c[bi] = -INFINITY;
         __syncwarp();
     }
     if (lane < a.top) {
         a.chosen[(size_t)t * a.top + lane] = my_e;
-        a.weights[(size_t)t * a.top + lane] = my_w / (chosen_sum + a.norm_eps);
+        a.weights[(size_t)t * a.top + lane] = my_w / (chosen_sum + a.norm_eps) * a.scale;
     }
 }
 
@@ -183,12 +191,22 @@ struct RowsArgs {
     int top;
     const void* w;          // [n_experts][n_out (2 n_out when gated: gate and up rows interleaved)][K]
     const int* offsets;     // [n_experts + 1]: expert e owns places offsets[e] .. offsets[e + 1] - 1
-    void* out;              // gated: [.][ld_out] of the run's type; plain: 32-bit
+    void* out;              // gated or activated: [.][ld_out] of the run's type; plain: 32-bit
     int ld_out;
     int K, n_out, units_per_cta;
-    int act;
+    int act;                // gated: the gate's activation; plain: 3 the square of max(., 0), else none
     float limit, slope;
 };
+
+constexpr int kActSquaredRelu = 3;
+template <typename T> __device__ __forceinline__ void store_plain(const RowsArgs& r, size_t at, float v) {
+    if (r.act == kActSquaredRelu) {
+        const float z = fmaxf(v, 0.f);
+        ((T*)r.out)[at] = from_f32<T>(z * z);
+    } else {
+        ((float*)r.out)[at] = v;
+    }
+}
 
 __device__ __forceinline__ uint4 load_streamed(const void* p) {    // weights pass once: they need not stay in L1
     uint4 v;
@@ -305,8 +323,8 @@ moe_rows_kernel(RowsArgs r) {
                         if (GATED) {
                             ((T*)r.out)[at + row0 / 2] = from_f32<T>(gated_value(s0, s1, r.act, r.limit, r.slope));
                         } else {
-                            ((float*)r.out)[at + row0] = s0;
-                            if (second) ((float*)r.out)[at + row0 + 1] = s1;
+                            store_plain<T>(r, at + row0, s0);
+                            if (second) store_plain<T>(r, at + row0 + 1, s1);
                         }
                     }
                 }
@@ -412,7 +430,7 @@ moe_rows_mma_kernel(RowsArgs r, int k_parts) {
 #pragma unroll
                 for (int i = 0; i < 4; ++i) {
                     const int m = 2 * t + (i & 1), row = row0 + g + (i >> 1) * 8;
-                    if (m < cnt && row < n_rows) ((float*)r.out)[(size_t)(g0 + m) * r.ld_out + row] = d[i];
+                    if (m < cnt && row < n_rows) store_plain<__nv_bfloat16>(r, (size_t)(g0 + m) * r.ld_out + row, d[i]);
                 }
             }
         }
@@ -501,14 +519,14 @@ extern "C" int b200_moe_table_route(const int* tokens, const int* table, int* ch
 
 extern "C" int b200_moe_route(const void* h, int ld_h, int dtype, const float* router, int* chosen, float* weights,
                               float* scores, int n_tokens, int width, int n_experts, int n_groups, int keep_groups, int top,
-                              float norm_eps, const float* bias, cudaStream_t stream) {
+                              float norm_eps, const float* bias, int sigmoid_scores, const float* correction, float scale, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (n_experts < 1 || n_experts > b200::kMaxExperts || top < 1 || top > 32 || top > n_experts || n_groups < 1 ||
         n_experts % n_groups || keep_groups < 1 || keep_groups > n_groups || top > keep_groups * (n_experts / n_groups))
         return b200::kErrBadArgument;
-    const size_t smem = sizeof(float) * ((size_t)width + n_experts + n_groups);
+    const size_t smem = sizeof(float) * ((size_t)width + 2 * (size_t)n_experts + n_groups);
     if (smem > 200 * 1024) return b200::kErrUnsupportedSize;
-    const b200::RouteArgs a = {h, ld_h, router, chosen, weights, scores, n_tokens, width, n_experts, n_groups, keep_groups, top, norm_eps, bias};
+    const b200::RouteArgs a = {h, ld_h, router, chosen, weights, scores, n_tokens, width, n_experts, n_groups, keep_groups, top, norm_eps, bias, sigmoid_scores, correction, scale};
     B200_DISPATCH_DTYPE(dtype, T,
         auto kernel = b200::moe_route_kernel<T>;
         if (smem > 48 * 1024) {
@@ -520,12 +538,13 @@ extern "C" int b200_moe_route(const void* h, int ld_h, int dtype, const float* r
 }
 
 // One product per expert over the places offsets[e] .. offsets[e + 1] - 1 (see moe_rows_kernel).  gated: w holds gate
-// and up rows interleaved and `out` is of the run's type; else `out` is 32-bit.  act: 0 SiLU, 1 GELU (tanh form), 2 clamped.
+// and up rows interleaved and `out` is of the run's type, act: 0 SiLU, 1 GELU (tanh form), 2 clamped; else `out` is 32-bit, or with act 3 of the run's
+// type and holds the square of max(., 0).
 extern "C" int b200_moe_rows(const void* a, int ld_a, int dtype, const int* order, int top, const void* w, const int* offsets,
                              void* out, int ld_out, int n_experts, int K, int n_out, int gated, int act, float limit,
                              float slope, cudaStream_t stream) {
     if (n_experts <= 0 || n_out <= 0) return 0;
-    if (K < 1 || act < 0 || act > 2 || (order && top < 1) || n_experts > 65535) return b200::kErrBadArgument;
+    if (K < 1 || act < 0 || act > (gated ? 2 : 3) || (order && top < 1) || n_experts > 65535) return b200::kErrBadArgument;
     const size_t el = dtype == b200::kF32 ? 4 : 2;
     const size_t smem = (size_t)b200::kRowsTokens * K * el;
     if (smem > 200 * 1024) return b200::kErrUnsupportedSize;
