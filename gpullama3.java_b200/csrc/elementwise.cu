@@ -163,7 +163,7 @@ __global__ void gate_rows_kernel(T* __restrict__ x, int ld_x, const T* __restric
 
 template <typename T>
 __global__ void __launch_bounds__(128)
-differential_heads_kernel(const T* __restrict__ maps, const T* __restrict__ gate, int ld_gate, T* __restrict__ out,
+differential_heads_kernel(const T* __restrict__ maps, const T* __restrict__ gate, int ld_gate, T* __restrict__ out, int ld_out,
                           int n_heads, int d, int d_pad, int n_rows, float lambda, float post, float eps) {
     pdl_launch_dependents();
     pdl_wait();
@@ -180,7 +180,7 @@ differential_heads_kernel(const T* __restrict__ maps, const T* __restrict__ gate
     ss = warp_sum(ss);
     const float scale = post / sqrtf(ss / (float)d + eps);
     const T* g = gate ? gate + (size_t)t * ld_gate + (size_t)h * d : nullptr;
-    T* o_row = out + (size_t)row * d;
+    T* o_row = out + (size_t)t * ld_out + (size_t)h * d;
     for (int e = lane; e < d; e += 32) {
         float o = (to_f32<T>(a1[e]) - lambda * to_f32<T>(a2[e])) * scale;
         if (g) o *= 1.0f / (1.0f + expf(-to_f32<T>(g[e])));
@@ -303,17 +303,17 @@ extern "C" int b200_scale_rows(float* x, long long n, float s, cudaStream_t stre
     return b200::launch_status();
 }
 
-// maps [T][2 n_heads][d_pad], gate [T][ld_gate] (or null), out [T][n_heads d], all of the run's type
-extern "C" int b200_differential_heads(const void* maps, const void* gate, int ld_gate, void* out, int dtype, int n_tokens,
+// maps [T][2 n_heads][d_pad], gate [T][ld_gate] (or null), out [T][ld_out >= n_heads d], all of the run's type
+extern "C" int b200_differential_heads(const void* maps, const void* gate, int ld_gate, void* out, int ld_out, int dtype, int n_tokens,
                                        int n_heads, int d, int d_pad, float lambda, float post, float eps,
                                        cudaStream_t stream) {
     if (n_tokens <= 0 || n_heads <= 0) return 0;
-    if (d < 1 || d_pad < d || (gate && ld_gate < n_heads * d)) return b200::kErrBadArgument;
+    if (d < 1 || d_pad < d || ld_out < n_heads * d || (gate && ld_gate < n_heads * d)) return b200::kErrBadArgument;
     const long long rows = (long long)n_tokens * n_heads;
     if (rows > 0x7fffffffLL) return b200::kErrUnsupportedSize;
     B200_DISPATCH_DTYPE(dtype, T,
         return b200::launch_pdl(b200::differential_heads_kernel<T>, dim3((int)((rows + 3) / 4)), dim3(128), 0, stream,
-                                (const T*)maps, (const T*)gate, ld_gate, (T*)out, n_heads, d, d_pad, (int)rows, lambda, post, eps));
+                                (const T*)maps, (const T*)gate, ld_gate, (T*)out, ld_out, n_heads, d, d_pad, (int)rows, lambda, post, eps));
     return 0;
 }
 

@@ -189,7 +189,7 @@ class CausalLM:
             mark = ws.mark() if ws is not None else 0
             if entry.enters is not None and handed is None:
                 self.pass_offsets.add_to(residual, entry.enters)
-            if block.takes_scaled_rows(ctx):
+            if block.takes_scaled_rows(ctx) or block.leaves_scaled_rows(ctx):
                 nxt = self.blocks[self.schedule[k + 1].layer] if k + 1 < len(self.schedule) else None
                 then = nxt.first_norm() if nxt is not None and nxt.takes_scaled_rows(ctx) else None
                 if then is not None and self.schedule[k + 1].enters is not None:

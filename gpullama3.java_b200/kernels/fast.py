@@ -64,10 +64,11 @@ def try_decode_attention_with_rope(qkv, out, ctx, page_table, cache, mixer, writ
 
 def try_attention(qkv, out, ctx, page_table, cache, mixer, gate=None) -> bool:
     if getattr(mixer, "has_terms", False):
-        # kept first positions, runs of positions, distance penalty, sink, output gate: the span kernel for decode steps, for
-        # prompts the tcgen05 kernel where runs and sink are all there is (heads of 64 and 128), else the flash kernel
+        # kept first positions, runs of positions, distance penalty, sink, output gate, soft cap: the span kernel for decode steps,
+        # for prompts the tcgen05 kernel without kept positions and penalty (heads of 64 and 128), else the flash kernel
         chunk = getattr(mixer, "chunk", None) or 0
-        terms = dict(keep_first=mixer.keep_first, chunk=chunk, slopes=mixer.slopes, sinks=mixer.sinks, gate=gate)
+        terms = dict(keep_first=mixer.keep_first, chunk=chunk, slopes=mixer.slopes, sinks=mixer.sinks, gate=gate,
+                     softcap=getattr(mixer, "softcap", None) or 0.0)
         if qkv.dtype != torch.bfloat16 or mixer.head_dim not in (32, 64, 96, 128):
             return False
         if ctx.all_decode and ops.attention_decode_supported(qkv.dtype, mixer.n_heads, mixer.n_kv_heads, mixer.head_dim):
@@ -77,9 +78,10 @@ def try_attention(qkv, out, ctx, page_table, cache, mixer, gate=None) -> bool:
             return True
         if qkv.shape[1] % 8 or (qkv.data_ptr() & 15):
             return False
-        if not mixer.keep_first and mixer.slopes is None and gate is None and ops.attention_prefill_tc(
+        if not mixer.keep_first and mixer.slopes is None and ops.attention_prefill_tc(
                 qkv, qkv.shape[1], out, ctx.cu_seqlens, ctx.kv_lens, page_table, cache.k, cache.v, ctx.n_seqs, ctx.max_q_len,
-                mixer.n_heads, mixer.n_kv_heads, mixer.head_dim, mixer.window or 0, chunk=chunk, sinks=mixer.sinks):
+                mixer.n_heads, mixer.n_kv_heads, mixer.head_dim, mixer.window or 0, chunk=chunk, sinks=mixer.sinks, gate=gate,
+                softcap=terms["softcap"]):
             return True
         ops.attention_prefill(qkv, qkv.shape[1], out, ctx.cu_seqlens, ctx.kv_lens, page_table, cache.k, cache.v,
                               ctx.n_seqs, ctx.max_q_len, mixer.n_heads, mixer.n_kv_heads, mixer.head_dim,

@@ -40,7 +40,7 @@ _SIGNATURES = {
                                              c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int]),
     "b200_attention_paged": ("attention_generic", [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
                                                    c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
-                                                   c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int]),
+                                                   c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_float]),
     "b200_gemm_generic": ("gemm_generic", [c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_void_p, c_int, c_int,
                                            c_int, c_int, c_int, c_int, c_float, c_float, c_void_p, c_int]),
     "b200_gemm_generic_batched": ("gemm_generic", [c_void_p, c_int, c_int, ctypes.c_longlong, c_void_p, c_int, c_int,
@@ -66,16 +66,18 @@ _SIGNATURES = {
                                                    c_int, c_int, c_int]),
     "b200_attention_decode_terms": ("attention_decode", [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
                                                          c_void_p, c_void_p, ctypes.c_longlong, c_int, c_int, c_int, c_int,
-                                                         c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int]),
+                                                         c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int,
+                                                         c_float]),
     "b200_attention_prefill": ("attention_prefill", [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
                                                      c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
-                                                     c_int, c_void_p, c_void_p, c_void_p, c_int]),
+                                                     c_int, c_void_p, c_void_p, c_void_p, c_int, c_float]),
     "b200_attention_decode_rope": ("attention_decode", [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
                                                         c_void_p, c_void_p, ctypes.c_longlong, c_int, c_int, c_int,
                                                         c_int, c_int, c_int, c_void_p, c_int, c_int, c_int]),
     "b200_attention_prefill_tc": ("attention_prefill_tcgen05", [c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p,
                                                                 c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int,
-                                                                c_int, c_int, c_int, c_int, c_int, c_void_p]),
+                                                                c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int,
+                                                                c_float]),
     "b200_random_fill": ("random_init", [c_void_p, c_int, ctypes.c_longlong, ctypes.c_ulonglong, c_float, c_float]),
     "b200_streams_combine": ("streams", [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int]),
     "b200_streams_read_norm": ("streams", [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int,
@@ -111,6 +113,13 @@ _SIGNATURES = {
                                          c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int,
                                          c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_int, c_int, c_void_p,
                                          c_int, c_float, c_float]),
+    "b200_gated_scan": ("delta_rule", [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
+                                       ctypes.c_longlong, ctypes.c_longlong, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                                       c_int, c_int, c_int, c_int, c_int, c_int, c_float]),
+    "b200_matrix_memory": ("matrix_memory", [c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int,
+                                             c_void_p, c_void_p, c_float, c_void_p, ctypes.c_longlong, c_int, c_void_p, c_void_p,
+                                             c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float,
+                                             c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_float]),
     "b200_moe_table_route": ("moe", [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int]),
     "b200_layernorm": ("norm", [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_float]),
     "b200_causal_conv_silu": ("delta_rule", [c_void_p, c_int, c_void_p, c_void_p, ctypes.c_longlong, c_void_p, c_void_p,
@@ -119,21 +128,22 @@ _SIGNATURES = {
                                             ctypes.c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
                                             c_int, c_int, c_int, c_int, c_float, c_float, c_int]),
     "b200_moe_route": ("moe", [c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
-                               c_int, c_int, c_float, c_void_p]),
+                               c_int, c_int, c_float, c_void_p, c_int, c_void_p, c_float]),
     "b200_moe_rows": ("moe", [c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
                               c_int, c_int, c_int, c_float, c_float]),
     "b200_moe_group": ("moe", [c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p]),
     "b200_moe_gather": ("moe", [c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int]),
     "b200_moe_combine": ("moe", [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int]),
-    "b200_differential_heads": ("elementwise", [c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float,
-                                                c_float, c_float]),
+    "b200_differential_heads": ("elementwise", [c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
+                                                c_float, c_float, c_float]),
     "b200_gated_norm_step": ("gated_residual", [c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
                                                 c_void_p, c_int, c_int, c_int, c_float, c_int, c_void_p, ctypes.c_longlong, c_int,
                                                 c_void_p, c_void_p, c_void_p, ctypes.c_longlong, c_void_p, c_int, c_int, c_void_p]),
     "b200_depth_average": ("gated_residual", [c_void_p, ctypes.c_longlong, c_int, c_void_p, c_void_p, c_void_p, c_int,
                                               ctypes.c_longlong]),
     "b200_cast_rows": ("gated_residual", [c_void_p, c_void_p, c_int, ctypes.c_longlong]),
-    "b200_bias_act_rows": ("gated_residual", [c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_int]),
+    "b200_bias_act_rows": ("gated_residual", [c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int,
+                                              c_int]),
     "b200_token_gate_rows": ("gated_residual", [c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_int,
                                                 c_int, c_int, c_int]),
     "b200_argmax_rows": ("sampling", [c_void_p, c_int, c_void_p, c_int, c_int]),
@@ -321,14 +331,15 @@ def attention_paged(q: torch.Tensor, q_row_stride: int, out: torch.Tensor, posit
                     seq_ids: torch.Tensor, page_table: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor,
                     n_heads: int, n_kv_heads: int, head_dim: int, window: int = 0, n_splits: int = 1, *,
                     keep_first: int = 0, chunk: int = 0, slopes: torch.Tensor | None = None,
-                    sinks: torch.Tensor | None = None, gate: torch.Tensor | None = None) -> None:
+                    sinks: torch.Tensor | None = None, gate: torch.Tensor | None = None, softcap: float = 0.0) -> None:
     """Causal grouped-query attention of every token of ``q`` over the cached keys 0..position of
     its sequence.  q: rows of ``q_row_stride`` elements whose first H*D are the rotated queries.
     ``n_splits`` > 1 cuts every token's keys into that many spans, one CTA each, merged by a second kernel (a decode
     step: few tokens, long rows of keys).  ``keep_first``: positions below it stay visible behind the window;
     ``slopes`` float32 [H]: score -= slopes[h] * distance; ``sinks`` float32 [H]: exp(sinks[h]) joins the softmax's
     denominator; ``gate`` [T, >= H] of q's dtype: head outputs are multiplied by sigmoid(gate[t, h]).  ``chunk`` (in place of a
-    window): positions are cut into runs of that many, counted from 0, and a query sees the keys of its own run."""
+    window): positions are cut into runs of that many, counted from 0, and a query sees the keys of its own run.  ``softcap`` > 0:
+    score <- softcap * tanh(score / softcap), before the penalty; the sink is not capped."""
     _dev(q, out, positions, seq_ids, page_table, k_pool, v_pool)
     assert out.is_contiguous() and out.shape[1] == n_heads * head_dim and out.dtype == q.dtype == k_pool.dtype
     assert tuple(k_pool.shape[1:]) == (n_kv_heads, PAGE_TOKENS, head_dim)
@@ -345,12 +356,13 @@ def attention_paged(q: torch.Tensor, q_row_stride: int, out: torch.Tensor, posit
         q.data_ptr(), q_row_stride, out.data_ptr(), dtype_code(q.dtype), positions.data_ptr(), seq_ids.data_ptr(),
         page_table.data_ptr(), page_table.shape[1], k_pool.data_ptr(), v_pool.data_ptr(), out.shape[0], n_heads,
         n_kv_heads, head_dim, int(window), int(n_splits), scratch.data_ptr() if scratch is not None else None,
-        int(keep_first), int(chunk), ptr(slopes), ptr(sinks), ptr(gate), gate.stride(0) if gate is not None else 0, _stream()),
-        "attention_paged")
+        int(keep_first), int(chunk), ptr(slopes), ptr(sinks), ptr(gate), gate.stride(0) if gate is not None else 0,
+        float(softcap), _stream()), "attention_paged")
 
 
 # --------------------------------------------------------------------------- matrix products
 EPILOGUE_STORE, EPILOGUE_RESIDUAL_ADD, EPILOGUE_GATED_SILU, EPILOGUE_GATED_GELU_TANH, EPILOGUE_GATED_CLAMPED = 0, 1, 2, 3, 4
+EPILOGUE_SQUARED_RELU = 5   # the grouped product alone has it
 GATED_EPILOGUES = (EPILOGUE_GATED_SILU, EPILOGUE_GATED_GELU_TANH, EPILOGUE_GATED_CLAMPED)
 # the gated epilogues' activations: silu(g) u, gelu_tanh(g) u, and the clamped form g' sigmoid(slope g') (u' + 1) with
 # g' = min(g, limit), u' = clamp(u, -limit, limit), whose two numbers travel with the call (``gate_args``)
@@ -504,7 +516,7 @@ def gemm_tcgen05_grouped(a: torch.Tensor, w: torch.Tensor, offsets: torch.Tensor
                          epilogue: int = EPILOGUE_STORE, gate_args: tuple[float, float] = (0.0, 0.0)) -> bool:
     """One product per group in one launch on tcgen05 tensor cores: c[p] = a[p] @ w[g].T for the rows p = offsets[g] ..
     offsets[g + 1] - 1 (offsets int32 [G + 1] on the device, read there).  a [P, K] and w [G, N, K] bfloat16; c [P, N]
-    float32 (store) or [P, N / 2] bfloat16 (gated epilogues).  Returns False, having done nothing, for operands it
+    float32 (store), bfloat16 (``EPILOGUE_SQUARED_RELU``: max(., 0)^2) or [P, N / 2] bfloat16 (gated epilogues).  Returns False, having done nothing, for operands it
     does not take."""
     P, K = a.shape
     G, N, Kw = w.shape
@@ -512,7 +524,8 @@ def gemm_tcgen05_grouped(a: torch.Tensor, w: torch.Tensor, offsets: torch.Tensor
             or a.stride(0) % 8 or not w.is_contiguous() or (a.data_ptr() | w.data_ptr()) & 15):
         return False
     gated = epilogue in GATED_EPILOGUES
-    if (gated and (c.dtype != torch.bfloat16 or N % 2)) or (not gated and (epilogue != EPILOGUE_STORE or c.dtype != torch.float32)):
+    stored = {EPILOGUE_STORE: torch.float32, EPILOGUE_SQUARED_RELU: torch.bfloat16}
+    if (gated and (c.dtype != torch.bfloat16 or N % 2)) or (not gated and stored.get(epilogue) != c.dtype):
         return False
     _dev(a, w, offsets, c)
     assert Kw == K and offsets.dtype == torch.int32 and offsets.numel() == G + 1 and c.stride(1) == 1
@@ -707,11 +720,11 @@ def attention_decode(q: torch.Tensor, q_row_stride: int, out: torch.Tensor, kv_l
                      n_kv_heads: int, head_dim: int, window: int, n_splits: int,
                      scratch: torch.Tensor | None = None, early_start: bool = True, *, keep_first: int = 0, chunk: int = 0,
                      slopes: torch.Tensor | None = None, sinks: torch.Tensor | None = None,
-                     gate: torch.Tensor | None = None) -> None:
+                     gate: torch.Tensor | None = None, softcap: float = 0.0) -> None:
     """One query token per sequence (row i of q belongs to sequence i) over kv_lens[i] cached keys.
     ``scratch``: float32 workspace for the spans' partial results (allocated here when absent).
-    ``early_start``: see ``attention_decode_early_start``.  ``keep_first``, ``chunk``, ``slopes``, ``sinks``, ``gate``:
-    as for ``attention_paged``."""
+    ``early_start``: see ``attention_decode_early_start``.  ``keep_first``, ``chunk``, ``slopes``, ``sinks``, ``gate``,
+    ``softcap``: as for ``attention_paged``."""
     _dev(q, out, kv_lens, page_table, k_pool, v_pool)
     n_seqs = out.shape[0]
     assert q.dtype == out.dtype == k_pool.dtype == torch.bfloat16 and out.is_contiguous()
@@ -720,7 +733,7 @@ def attention_decode(q: torch.Tensor, q_row_stride: int, out: torch.Tensor, kv_l
     need = n_seqs * n_heads * n_splits * (head_dim + 2) if n_splits > 1 else 0
     if need and (scratch is None or scratch.numel() < need):
         scratch = torch.empty(need, dtype=torch.float32, device=q.device)
-    if keep_first or chunk or slopes is not None or sinks is not None or gate is not None:
+    if keep_first or chunk or slopes is not None or sinks is not None or gate is not None or softcap:
         _dev(slopes, sinks, gate)
         for t in (slopes, sinks):
             assert t is None or (t.dtype == torch.float32 and t.is_contiguous() and t.numel() == n_heads)
@@ -730,7 +743,7 @@ def attention_decode(q: torch.Tensor, q_row_stride: int, out: torch.Tensor, kv_l
             q.data_ptr(), q_row_stride, out.data_ptr(), kv_lens.data_ptr(), page_table.data_ptr(), page_table.shape[1],
             k_pool.data_ptr(), v_pool.data_ptr(), scratch.data_ptr() if need else None, scratch.numel() if need else 0,
             n_seqs, n_heads, n_kv_heads, head_dim, int(window), n_splits, 1 if early_start else 0, int(keep_first), int(chunk),
-            ptr(slopes), ptr(sinks), ptr(gate), gate.stride(0) if gate is not None else 0, _stream()),
+            ptr(slopes), ptr(sinks), ptr(gate), gate.stride(0) if gate is not None else 0, float(softcap), _stream()),
             "attention_decode_terms" if early_start else "attention_decode_terms:late")
         return
     _check(_fn("b200_attention_decode")(
@@ -744,10 +757,10 @@ def attention_prefill(q: torch.Tensor, q_row_stride: int, out: torch.Tensor, cu_
                       kv_lens: torch.Tensor, page_table: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor,
                       n_seqs: int, max_q_len: int, n_heads: int, n_kv_heads: int, head_dim: int, window: int, *,
                       keep_first: int = 0, chunk: int = 0, slopes: torch.Tensor | None = None, sinks: torch.Tensor | None = None,
-                      gate: torch.Tensor | None = None) -> None:
+                      gate: torch.Tensor | None = None, softcap: float = 0.0) -> None:
     """Causal attention of packed query tokens: sequence i owns rows cu_seqlens[i]..cu_seqlens[i+1],
     which are its last positions (kv_lens[i] - q_len .. kv_lens[i] - 1); keys come from the cache.
-    ``keep_first``, ``chunk``, ``slopes``, ``sinks``, ``gate``: as for ``attention_paged``."""
+    ``keep_first``, ``chunk``, ``slopes``, ``sinks``, ``gate``, ``softcap``: as for ``attention_paged``."""
     _dev(q, out, cu_seqlens, kv_lens, page_table, k_pool, v_pool, slopes, sinks, gate)
     for t in (slopes, sinks):
         assert t is None or (t.dtype == torch.float32 and t.is_contiguous() and t.numel() == n_heads)
@@ -760,19 +773,20 @@ def attention_prefill(q: torch.Tensor, q_row_stride: int, out: torch.Tensor, cu_
         q.data_ptr(), q_row_stride, out.data_ptr(), cu_seqlens.data_ptr(), kv_lens.data_ptr(), page_table.data_ptr(),
         page_table.shape[1], k_pool.data_ptr(), v_pool.data_ptr(), n_seqs, max_q_len, n_heads, n_kv_heads, head_dim,
         int(window), int(keep_first), int(chunk), ptr(slopes), ptr(sinks), ptr(gate),
-        gate.stride(0) if gate is not None else 0, _stream()), "attention_prefill")
+        gate.stride(0) if gate is not None else 0, float(softcap), _stream()), "attention_prefill")
 
 
 def attention_prefill_tc(q: torch.Tensor, q_row_stride: int, out: torch.Tensor, cu_seqlens: torch.Tensor,
                          kv_lens: torch.Tensor, page_table: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor,
                          n_seqs: int, max_q_len: int, n_heads: int, n_kv_heads: int, head_dim: int, window: int, *,
-                         chunk: int = 0, sinks: torch.Tensor | None = None) -> bool:
-    """``attention_prefill`` on tcgen05 tensor cores (head_dim 64 or 128), with ``chunk`` and ``sinks`` but none of the other
-    terms.  Returns False, having done
-    nothing, for sizes it does not take."""
+                         chunk: int = 0, sinks: torch.Tensor | None = None, gate: torch.Tensor | None = None,
+                         softcap: float = 0.0) -> bool:
+    """``attention_prefill`` on tcgen05 tensor cores (head_dim 64 or 128), with ``chunk``, ``sinks``, ``gate`` and ``softcap`` but
+    none of the other terms.  Returns False, having done nothing, for sizes it does not take."""
     if head_dim not in (64, 128) or q.dtype != torch.bfloat16 or q_row_stride % 8 or (q.data_ptr() | out.data_ptr()) & 15:
         return False
-    _dev(q, out, cu_seqlens, kv_lens, page_table, k_pool, v_pool, sinks)
+    _dev(q, out, cu_seqlens, kv_lens, page_table, k_pool, v_pool, sinks, gate)
+    assert gate is None or (gate.dtype == torch.bfloat16 and gate.stride(1) == 1 and gate.shape[1] >= n_heads)
     assert sinks is None or (sinks.dtype == torch.float32 and sinks.is_contiguous() and sinks.numel() == n_heads)
     assert out.dtype == k_pool.dtype == torch.bfloat16 and out.is_contiguous() and k_pool.is_contiguous()
     assert tuple(k_pool.shape[1:]) == (n_kv_heads, PAGE_TOKENS, head_dim)
@@ -781,7 +795,8 @@ def attention_prefill_tc(q: torch.Tensor, q_row_stride: int, out: torch.Tensor, 
         q.data_ptr(), q_row_stride, out.shape[0], out.data_ptr(), cu_seqlens.data_ptr(), kv_lens.data_ptr(),
         page_table.data_ptr(), page_table.shape[1], k_pool.data_ptr(), v_pool.data_ptr(), k_pool.shape[0], n_seqs,
         max_q_len, n_heads, n_kv_heads, head_dim, int(window), int(chunk), sinks.data_ptr() if sinks is not None else None,
-        _stream()), "attention_prefill_tc")
+        gate.data_ptr() if gate is not None else None, gate.stride(0) if gate is not None else 0, float(softcap), _stream()),
+        "attention_prefill_tc")
     return True
 
 
@@ -893,7 +908,7 @@ def head_row_segment(src_off: int, n_rows: int, d: int, dst_off: int, d_pad: int
                      norm: bool | int = False, weight_off: int = -1, mul: float = 1.0, target: int = TO_ROWS,
                      weight_per_row: bool = False, mix_off: int = -1, rotate: bool = False, src_stride: int = -1,
                      dst_stride: int = -1, cache_dim: int = -1, lead: int = 0, half_pairs: int | None = None,
-                     freq_off: int = 0) -> list[int]:
+                     freq_off: int = 0, turn_mul: float = 1.0) -> list[int]:
     """One segment of ``head_rows``: ``n_rows`` rows of ``d`` numbers from column ``src_off`` on, each (+ bias)
     (normalised) (* weight) * mul, written ``d_pad`` wide (zeros behind the ``d``) from column ``dst_off`` on, or with
     ``target`` TO_CACHE_KEYS / TO_CACHE_VALUES into the cache page of the token's position (``n_rows`` = the cache
@@ -906,12 +921,13 @@ def head_row_segment(src_off: int, n_rows: int, d: int, dst_off: int, d_pad: int
     the ``d_pad`` columns from ``dst_off`` on of every cache row.  ``lead``: how many of the ``d_pad`` numbers written are
     zeros in front of the row's ``d`` (the rest of the zeros follow it).  ``half_pairs`` n (in place of ``rotate``): the
     row's pairs (i, i + n), i < n, are turned by the token's position times the frequencies from ``freq_off`` on; the columns
-    from 2 n on pass."""
+    from 2 n on pass; ``turn_mul``: a factor on their cosines and sines."""
     import struct
 
+    bits = lambda x: struct.unpack("<i", struct.pack("<f", float(x)))[0]
     return [src_off, n_rows, d, dst_off, d if d_pad is None else d_pad, bias_off, int(norm), weight_off,
-            struct.unpack("<i", struct.pack("<f", float(mul)))[0], target, 1 if weight_per_row else 0, mix_off,
-            2 if half_pairs else 1 if rotate else 0, src_stride, dst_stride, cache_dim, int(lead), int(half_pairs or 0), int(freq_off), 0]
+            bits(mul), target, 1 if weight_per_row else 0, mix_off,
+            2 if half_pairs else 1 if rotate else 0, src_stride, dst_stride, cache_dim, int(lead), int(half_pairs or 0), int(freq_off), bits(turn_mul)]
 
 
 def head_rows(src: torch.Tensor, dst: torch.Tensor | None, segments, eps: float = 0.0, bias: torch.Tensor | None = None,
@@ -1018,14 +1034,15 @@ def scale_rows(logits: torch.Tensor, scale: float) -> None:
 def differential_heads(maps: torch.Tensor, gate: torch.Tensor | None, out: torch.Tensor, n_heads: int, d: int, d_pad: int,
                        weight: float, post: float, eps: float) -> None:
     """maps [T, 2 n_heads d_pad]: heads (2h, 2h + 1) are two attention maps' results over the same values.  out[t, h] =
-    post * o / sqrt(mean(o^2) + eps) * sigmoid(gate[t, h]) over the first ``d`` numbers, o = map 1 - weight * map 2."""
+    post * o / sqrt(mean(o^2) + eps) * sigmoid(gate[t, h]) over the first ``d`` numbers, o = map 1 - weight * map 2; ``out`` may be
+    columns of a wider buffer."""
     _dev(maps, gate, out)
-    assert maps.is_contiguous() and out.is_contiguous() and maps.dtype == out.dtype
+    assert maps.is_contiguous() and out.stride(1) == 1 and maps.dtype == out.dtype
     assert maps.shape[1] == 2 * n_heads * d_pad and out.shape[1] == n_heads * d and maps.shape[0] == out.shape[0]
     assert gate is None or (gate.dtype == out.dtype and gate.stride(1) == 1 and gate.shape[1] >= n_heads * d)
     _check(_fn("b200_differential_heads")(maps.data_ptr(), gate.data_ptr() if gate is not None else None,
-                                          gate.stride(0) if gate is not None else 0, out.data_ptr(), dtype_code(out.dtype),
-                                          out.shape[0], int(n_heads), int(d), int(d_pad), float(weight), float(post), float(eps),
+                                          gate.stride(0) if gate is not None else 0, out.data_ptr(), out.stride(0),
+                                          dtype_code(out.dtype), out.shape[0], int(n_heads), int(d), int(d_pad), float(weight), float(post), float(eps),
                                           _stream()), "differential_heads")
 
 
@@ -1099,12 +1116,19 @@ def cast_rows(x: torch.Tensor, out: torch.Tensor) -> None:
 UNGATED_ACTIVATIONS = {"relu_squared": 0}
 
 
-def bias_act_rows(u: torch.Tensor, bias: torch.Tensor | None, activation: str = "relu_squared") -> None:
-    """u <- act(u + bias) in place on a product's result [T, n]; ``relu_squared``: max(., 0)^2, evaluated in 32 bits."""
-    _dev(u, bias)
+def bias_act_rows(u: torch.Tensor, bias: torch.Tensor | None, activation: str = "relu_squared", out: torch.Tensor | None = None,
+                  gate: torch.Tensor | None = None) -> None:
+    """act(u + bias) of a product's result [T, n], in place or into ``out`` [T, n] (columns of a wider buffer, if need be);
+    ``relu_squared``: max(., 0)^2, evaluated in 32 bits.  ``gate`` [T, >= 1]: row t is multiplied by sigmoid(gate[t, 0])."""
+    out = u if out is None else out
+    _dev(u, bias, out, gate)
     assert u.stride(1) == 1 and (bias is None or (bias.dtype == torch.float32 and bias.is_contiguous() and bias.numel() == u.shape[1]))
+    assert out.dtype == u.dtype and out.stride(1) == 1 and out.shape == u.shape
+    assert gate is None or (gate.dtype == u.dtype and gate.shape[0] == u.shape[0])
     _check(_fn("b200_bias_act_rows")(u.data_ptr(), u.stride(0), dtype_code(u.dtype), bias.data_ptr() if bias is not None else None,
-                                     u.shape[0], u.shape[1], UNGATED_ACTIVATIONS[activation], _stream()), "bias_act_rows")
+                                     out.data_ptr(), out.stride(0), gate.data_ptr() if gate is not None else None,
+                                     gate.stride(0) if gate is not None else 0, u.shape[0], u.shape[1], UNGATED_ACTIVATIONS[activation],
+                                     _stream()), "bias_act_rows")
 
 
 def token_gate_rows(a: torch.Tensor, tokens: torch.Tensor, table: torch.Tensor, out: torch.Tensor, n: int) -> None:
@@ -1341,6 +1365,94 @@ def fixed_decay(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.
         rows.stride(0) if rows is not None else 0, float(eps), float(mul), _stream()), "fixed_decay" if not single else "fixed_decay:step")
 
 
+MAX_MEMORY_KEYS = 512   # matrix_memory.cu
+
+
+def matrix_memory_copies(d_v: int) -> int:
+    """How many copies of its key sum and its running maximum a head keeps: the slices of its columns that the one-token kernel
+    takes (64 or 128 in fours, else 32)."""
+    return -(-d_v // (32 if d_v % 4 else 64 if d_v <= 64 else 128))
+
+
+def matrix_memory_state(heads: int, d_k: int, d_v: int) -> int:
+    """Floats of state per sequence: S [d_k, d_v], then n [copies, d_k], then m [copies] of every head, to a multiple of 4."""
+    copies = matrix_memory_copies(d_v)
+    return -(-heads * (d_k * d_v + copies * (d_k + 1)) // 4) * 4
+
+
+def matrix_memory_finishes(dtype: torch.dtype, all_single: bool, d_k: int, d_v: int) -> bool:
+    """Whether a CTA of ``matrix_memory`` has all of a head's values, so that it can also norm and gate them."""
+    if all_single:
+        return matrix_memory_copies(d_v) == 1
+    return dtype == torch.bfloat16 and d_v <= int(library("matrix_memory").b200_matrix_memory_columns(c_int(d_k), c_int(d_v)))
+
+
+def matrix_memory(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, log_gates, cap: float, state: torch.Tensor, slots: torch.Tensor,
+                  seq_ids: torch.Tensor, cu_seqlens: torch.Tensor, heads: int, d_k: int, d_v: int, max_q_len: int, *,
+                  q_scale: float = 1.0, out: torch.Tensor | None = None, finish=None, alloc=None) -> None:
+    """Per head over a packed step, with i = cap tanh((z_i + b_i) / cap) and f = log sigmoid(cap tanh((z_f + b_f) / cap)):
+    m <- max(f + m, i), S <- e^(f + m_old - m) S + e^(i - m) k v^T, n alike with k alone, o = S^T (q_scale q) / (max(|n . q_scale q|,
+    e^(-m)) + 1e-6); S, n and m in the float32 [slots, >= matrix_memory_state(...)] ``state`` at the sequence's slot, updated in place.
+    ``log_gates`` = (z_i [T, >= heads], z_f, b_i float32 [heads], b_f).  q, k [T, >= heads d_k], v [T, >= heads d_v], z of one type.
+    Steps of one token per sequence take one kernel; longer ones the run kernels (bfloat16, keys whose tiles fit an SM) or the
+    token-by-token scan.  ``out`` float32 [T, heads d_v], or ``finish`` = (rows [T, heads d_v], gate [T, >= heads d_v], activation, eps,
+    weight float32 [heads d_v] or None) where ``matrix_memory_finishes``: rows = o / sqrt(mean(o^2) + eps) per head * weight *
+    act(gate), rows being columns of a wider buffer."""
+    z_i, z_f, b_i, b_f = log_gates
+    _dev(q, k, v, z_i, z_f, b_i, b_f, state, slots, seq_ids, cu_seqlens, out)
+    T = q.shape[0]
+    assert q.dtype == k.dtype == v.dtype == z_i.dtype == z_f.dtype
+    assert all(t.stride(1) == 1 for t in (q, k, v, z_i, z_f, state))
+    assert q.shape[1] >= heads * d_k and k.shape[1] >= heads * d_k and v.shape[1] >= heads * d_v
+    assert z_i.shape[1] >= heads and z_f.shape[1] >= heads
+    for b in (b_i, b_f):
+        assert b.dtype == torch.float32 and b.is_contiguous() and b.numel() == heads
+    assert state.dtype == torch.float32 and state.shape[1] >= matrix_memory_state(heads, d_k, d_v)
+    n_seqs, copies = slots.numel(), matrix_memory_copies(d_v)
+    single = T == n_seqs
+    rows = gate = weight = None
+    act, eps = "sigmoid", 0.0
+    if finish is not None:
+        rows, gate, act, eps, weight = finish
+        _dev(rows, gate, weight)
+        assert out is None and rows.dtype == gate.dtype == q.dtype and rows.stride(1) == gate.stride(1) == 1
+        assert tuple(rows.shape) == (T, heads * d_v) and gate.shape[0] == T and gate.shape[1] >= heads * d_v
+        assert weight is None or (weight.dtype == torch.float32 and weight.is_contiguous() and weight.numel() == heads * d_v)
+    else:
+        assert out.dtype == torch.float32 and out.is_contiguous() and tuple(out.shape) == (T, heads * d_v)
+    ptr = lambda t: t.data_ptr() if t is not None else None
+    take = lambda shape: alloc(shape, torch.float32) if alloc is not None else torch.empty(shape, dtype=torch.float32, device=q.device)
+    lib = library("matrix_memory")
+    runs = not single and q.dtype == torch.bfloat16 and int(lib.b200_matrix_memory_columns(c_int(d_k), c_int(d_v))) > 0
+    scratch = scanned = None
+    if not single:
+        floats, more = (lib.b200_matrix_memory_scratch, (d_k, d_v)) if runs else (lib.b200_matrix_memory_gate_floats, ())
+        floats.restype = ctypes.c_longlong
+        scratch = take((int(floats(*(c_int(x) for x in (T, n_seqs, heads, *more)))),))
+
+    def call(stage, name):
+        _check(_fn("b200_matrix_memory")(
+            stage, q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0), z_i.data_ptr(), z_i.stride(0),
+            z_f.data_ptr(), z_f.stride(0), b_i.data_ptr(), b_f.data_ptr(), float(cap), state.data_ptr(), state.stride(0), copies,
+            slots.data_ptr(), cu_seqlens.data_ptr(), ptr(out), ptr(scratch), ptr(scanned), dtype_code(q.dtype), T, n_seqs,
+            int(max_q_len), heads, d_k, d_v, float(q_scale), ptr(weight), ptr(gate), gate.stride(0) if gate is not None else 0,
+            GATE_ACTIVATIONS[act], ptr(rows), rows.stride(0) if rows is not None else 0, float(eps), _stream()), name)
+
+    if single or runs:
+        call(0, "matrix_memory:step" if single else "matrix_memory")
+        return
+    assert out is not None, "the token-by-token scan leaves its heads unfinished"
+    call(1, "matrix_memory:gates")
+    scanned = take((T, heads, d_v + 1))
+    scan_rows = take((heads, T, int(library("delta_rule").b200_delta_rule_row(c_int(d_k), c_int(d_v + 1)))))
+    _check(_fn("b200_gated_scan")(
+        q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0), scratch.data_ptr(),
+        scratch.data_ptr() + 4 * (4 * heads * T), state.data_ptr(), state.stride(0), heads * d_k * d_v, copies * d_k, slots.data_ptr(),
+        seq_ids.data_ptr(), cu_seqlens.data_ptr(), scanned.data_ptr(), scan_rows.data_ptr(), dtype_code(q.dtype), T, n_seqs, heads,
+        d_k, d_v, float(q_scale), _stream()), "gated_scan")
+    call(2, "matrix_memory:divide")
+
+
 def delta_rule_supported(d_k: int) -> bool:
     lib = library("delta_rule")
     a, b = c_int(0), c_int(0)
@@ -1375,14 +1487,20 @@ def delta_rule_scan(qkv: torch.Tensor, beta: torch.Tensor, decay: torch.Tensor, 
 
 # --------------------------------------------------------------------------- routed feed-forward (mixture of experts)
 MAX_EXPERTS, MAX_EXPERTS_PER_TOKEN = 1024, 32   # moe.cu
+ROUTER_SCORES = {"softmax": 0, "sigmoid": 1}
+ACT_SQUARED_RELU = 3
 
 
 def moe_route(h: torch.Tensor, router: torch.Tensor, chosen: torch.Tensor, weights: torch.Tensor, n_groups: int,
-              keep_groups: int, norm_eps: float, scores: torch.Tensor | None = None, bias: torch.Tensor | None = None) -> None:
+              keep_groups: int, norm_eps: float, scores: torch.Tensor | None = None, bias: torch.Tensor | None = None, *,
+              score: str = "softmax", correction: torch.Tensor | None = None, scale: float = 1.0) -> None:
     """Per token of h [T, width]: softmax scores over router [E, width] (float32; ``bias`` float32 [E] joins the logits), the ``top`` = chosen.shape[1] best
     experts among the ``keep_groups`` best of ``n_groups`` groups of neighbours into chosen int32 [T, top], and
-    their scores over the chosen scores' sum (+ norm_eps) into weights float32 [T, top]."""
-    _dev(h, router, chosen, weights, scores)
+    their scores over the chosen scores' sum (+ norm_eps) into weights float32 [T, top].  ``score`` "sigmoid": every expert's
+    score is the sigmoid of its own logit; ``correction`` float32 [E] joins the scores for the choice alone; ``scale``: a last
+    factor on the weights."""
+    _dev(h, router, chosen, weights, scores, correction)
+    assert correction is None or (correction.dtype == torch.float32 and correction.is_contiguous() and correction.numel() == router.shape[0])
     T, width = h.shape
     E = router.shape[0]
     assert router.dtype == torch.float32 and router.is_contiguous() and router.shape[1] == width and h.stride(1) == 1
@@ -1394,7 +1512,8 @@ def moe_route(h: torch.Tensor, router: torch.Tensor, chosen: torch.Tensor, weigh
     _check(_fn("b200_moe_route")(h.data_ptr(), h.stride(0), dtype_code(h.dtype), router.data_ptr(), chosen.data_ptr(),
                                  weights.data_ptr(), scores.data_ptr() if scores is not None else None, T, width, E,
                                  int(n_groups), int(keep_groups), chosen.shape[1], float(norm_eps),
-                                 bias.data_ptr() if bias is not None else None, _stream()), "moe_route")
+                                 bias.data_ptr() if bias is not None else None, ROUTER_SCORES[score],
+                                 correction.data_ptr() if correction is not None else None, float(scale), _stream()), "moe_route")
 
 
 def moe_table_route(tokens: torch.Tensor, table: torch.Tensor, chosen: torch.Tensor, weights: torch.Tensor,
@@ -1419,17 +1538,20 @@ def moe_rows(a: torch.Tensor, w: torch.Tensor, offsets: torch.Tensor, out: torch
     """One weight-streaming product per expert: out[p] = a[row(p)] @ w[e].T for the places p = offsets[e] ..
     offsets[e + 1] - 1 of expert e, row(p) = order[p] // top when ``order`` is given, p otherwise.  With ``activation``
     w [E, 2 n, K] holds gate and up rows interleaved and out [P, n] (a's dtype) receives the gated values; without, w
-    [E, n, K] and out [P, n] float32.  The row counts are read on the device."""
+    [E, n, K] and out [P, n] float32.  With one of ``UNGATED_ACTIVATIONS`` w [E, n, K] and out [P, n] (a's dtype) receives the
+    activated values.  The row counts are read on the device."""
     _dev(a, w, offsets, out, order)
     E, rows, K = w.shape
-    gated = activation is not None
+    ungated = activation in UNGATED_ACTIVATIONS
+    gated = activation is not None and not ungated
     n_out = rows // 2 if gated else rows
     assert a.dtype == w.dtype and w.is_contiguous() and a.stride(1) == 1 and a.shape[1] == K and out.stride(1) == 1
-    assert out.shape[1] == n_out and out.dtype == (a.dtype if gated else torch.float32)
+    assert out.shape[1] == n_out and out.dtype == (a.dtype if gated or ungated else torch.float32)
     assert offsets.dtype == torch.int32 and offsets.numel() == E + 1 and (order is None or order.dtype == torch.int32)
     _check(_fn("b200_moe_rows")(a.data_ptr(), a.stride(0), dtype_code(a.dtype), order.data_ptr() if order is not None else None,
                                 int(top), w.data_ptr(), offsets.data_ptr(), out.data_ptr(), out.stride(0), E, K, n_out,
-                                1 if gated else 0, ACTIVATION_CODES[activation] if gated else 0, float(gate_args[0]),
+                                1 if gated else 0, ACTIVATION_CODES[activation] if gated else ACT_SQUARED_RELU if ungated else 0,
+                                float(gate_args[0]),
                                 float(gate_args[1]), _stream()), "moe_rows")
 
 

@@ -20,7 +20,7 @@ from .position import YarnRotaryPositionEncoding
 from .feed_forward import DenseFeedForward
 from .differential_attention import DifferentialAttention
 from .gated_residual import GatedResidualBlock
-from .linear_recurrence import FixedDecayAttention
+from .linear_recurrence import FixedDecayAttention, MatrixMemory
 from .chunked_attention import ChunkedAttention
 from .parallel import ParallelBlock, ParallelMixers
 
@@ -32,4 +32,4 @@ __all__ = ["Block", "FeedForward", "Mixer", "Norm", "Part", "PartRegistryError",
            "ChannelDeltaRule", "HeadDeltaRule", "LayerNorm", "RoutedFeedForward", "GatedLinearAttention",
            "StateSpaceDuality", "SandwichBlock", "YarnRotaryPositionEncoding", "DenseFeedForward",
            "DifferentialAttention", "GatedResidualBlock", "FixedDecayAttention", "ChunkedAttention", "ParallelBlock",
-           "ParallelMixers"]
+           "ParallelMixers", "MatrixMemory"]

@@ -252,7 +252,7 @@ def attend(shape, qkv: torch.Tensor, out: torch.Tensor, ctx: StepContext, table:
     """Attention of the finished query rows in ``qkv`` over the paged cache into ``out``: a tensor-core kernel where one
     takes the sizes, else the plain kernel (a step of few tokens cuts their keys into spans so that the GPU has CTAs to
     run).  ``shape`` as for ``plan_decode_attention``, with ``plan_decode``, ``has_terms`` and the terms themselves
-    (``slopes``, ``sinks``) where it has any."""
+    (``slopes``, ``sinks``, ``softcap``) where it has any."""
     if fast.try_attention(qkv, out, ctx, table, cache, shape, gate):
         return
     rows = qkv.shape[0] * shape.n_heads
@@ -261,7 +261,7 @@ def attend(shape, qkv: torch.Tensor, out: torch.Tensor, ctx: StepContext, table:
     ops.attention_paged(qkv, qkv.shape[1], out, ctx.positions, ctx.seq_ids, table, cache.k, cache.v,
                         shape.n_heads, shape.n_kv_heads, shape.head_dim, shape.window or 0, n_splits=splits,
                         keep_first=shape.keep_first, chunk=getattr(shape, "chunk", None) or 0, slopes=getattr(shape, "slopes", None), sinks=getattr(shape, "sinks", None),
-                        gate=gate)
+                        gate=gate, softcap=getattr(shape, "softcap", None) or 0.0)
 
 
 VALUE_MIX_SOURCE = "value mix source"   # in a pass's ``ctx.extras``: the first value-mixing layer's own values [T, G dv]

@@ -119,8 +119,11 @@ class OpenEnded:
     """A mixer or feed-forward whose result is one last product over rows it makes: result = W rows (+ b).  Whoever
     arranges such parts side by side may take their last products over (``take_output``), let each write its rows into
     neighbouring columns of one buffer (``rows_into``) and multiply once; where a part is used alone, its own ``forward`` does
-    both.  Mixers that also start with one product over their input can give that away too (``take_input``) and be handed
-    its result (``rows_from``)."""
+    both.  Parts that also start with one product over their input can give that away too (``take_input``, where
+    ``gives_input`` says so) and be handed its result (``rows_from``).  A part of whose result some is no product over rows adds that
+    to the stream itself (``adds_itself``); where all of it is such, ``open_columns`` is 0 and there is no last product."""
+
+    gives_input: bool = False
 
     def open_columns(self) -> int:
         """Numbers per token of the rows before the last product."""
@@ -134,6 +137,9 @@ class OpenEnded:
         """The rows of input x (a tensor, or ScaledRows where ``takes_scaled_rows``) into ``rows`` [T, open_columns], columns of
         a wider buffer; ``mul``: a factor on them, applied in 32 bits before they are rounded."""
         raise NotImplementedError
+
+    def adds_itself(self, x, ctx: "StepContext", residual: torch.Tensor) -> None:
+        """Adds to ``residual`` what the last product does not make of input x (a tensor)."""
 
     def take_input(self) -> torch.Tensor:
         """The first product's weight [columns, hidden], columns a multiple of 8; the part keeps none."""
@@ -226,6 +232,10 @@ class Block(Part):
 
     def takes_scaled_rows(self, ctx: StepContext) -> bool:
         return False
+
+    def leaves_scaled_rows(self, ctx: StepContext) -> bool:
+        """Whether the block may be called with ``then_norm`` although it does not take ScaledRows itself (``x_in`` is None)."""
+        return self.takes_scaled_rows(ctx)
 
     def first_norm(self) -> Norm | None:
         """The norm the block applies to the residual stream before anything else, if it starts that way."""

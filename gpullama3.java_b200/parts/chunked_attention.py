@@ -47,6 +47,7 @@ class _KernelShape:
 
 class ChunkedAttention(Mixer, OpenEnded):
     graph_safe = True
+    gives_input = True
     pad_safe = True
 
     def __init__(self, hidden_size: int, n_heads: int, n_kv_heads: int, head_dim: int, value_dim: int, scale: float,

@@ -18,7 +18,10 @@ cosine and sine times the encoding's ``magnitude``) and the rotated row of W_dkv
 score = scale (q_plain . W_uk,h c + q_rot . k_rot).  The cache row is then [c | k_rot] as a key and [c | 0] as a value, and a
 query in the latent space is [W_uk,h^T q_plain | q_rot]: still one key/value head and the same attention kernels.  The
 per-head product that carries the queries has an identity block for the rotated part.  ``output_gate``: the
-concatenated heads are multiplied by sigmoid(W_g x) before the output product; its rows ride in the first product."""
+concatenated heads are multiplied by sigmoid(W_g x) before the output product; its rows ride in the first product.
+``head_gate``: one such number per head, sigmoid(W_g x)_h (the attention kernels apply it, since what follows is linear).
+``sink``: a learned number per head whose exponential joins the softmax's denominator.  The rotated parts may be turned in
+interleaved pairs or over their halves, as the position encoding says."""
 
 from __future__ import annotations
 
@@ -26,35 +29,41 @@ import torch
 
 from ..cache.sequence_cache import KVCacheNeed, KVView
 from ..config.base import ConfigError
-from ..kernels import fast, ops
+from ..kernels import ops
 from ..weights.loader import ParamSpec
-from .attention import kernel_head_dim
-from .base import Mixer, StepContext, register_mixer
+from .attention import attend, kernel_head_dim
+from .base import Mixer, OpenEnded, StepContext, register_mixer
 from .linear import Linear
+from .position import PAIRING_CODES
 
 
 def _pad8(n: int) -> int:
     return -(-n // 8) * 8
 
 
-class LatentAttention(Mixer):
+class LatentAttention(Mixer, OpenEnded):
     graph_safe = True
     pad_safe = True
+    gives_input = True
+    keep_first = 0
+    slopes = None
     DECODE_GROUP = 16   # query heads per key/value head that the decode attention kernel takes
 
     def __init__(self, hidden_size: int, n_heads: int, head_dim: int, value_dim: int, kv_rank: int, q_rank: int | None,
                  norm_eps: float, scale: float | None = None, window: int | None = None, rot_dim: int = 0,
-                 position=None, output_gate: bool = False):
+                 position=None, output_gate: bool = False, head_gate: bool = False, sink: bool = False):
+        if output_gate and head_gate:
+            raise ConfigError("latent attention: a gate per number or one per head, not both")
+        self.head_gate, self.sink, self.sinks = bool(head_gate), bool(sink), None
+        self.has_terms = self.head_gate or self.sink
         self.hidden_size, self.n_heads, self.key_dim, self.value_dim = hidden_size, n_heads, int(head_dim), int(value_dim)
         self.kv_rank, self.q_rank, self.norm_eps = int(kv_rank), (int(q_rank) if q_rank is not None else None), float(norm_eps)
         self.rot_dim, self.position, self.output_gate = int(rot_dim), position, bool(output_gate)
         self.scale = float(scale) if scale is not None else (self.key_dim + self.rot_dim) ** -0.5
         if min(self.kv_rank, self.q_rank or 1, self.key_dim, self.value_dim, n_heads) < 1 or self.rot_dim < 0:
             raise ConfigError("latent attention: every size must be positive")
-        if self.rot_dim and (position is None or position.rotary_dim != self.rot_dim or self.rot_dim % 2
-                             or position.pairing != 0):
-            raise ConfigError(f"latent attention: {self.rot_dim} rotated dimensions need a rotary position encoding of "
-                              "that size over interleaved pairs")
+        if self.rot_dim and (position is None or position.rotary_dim != self.rot_dim or self.rot_dim % 2):
+            raise ConfigError(f"latent attention: {self.rot_dim} rotated dimensions need a rotary position encoding of that size")
         if self.rot_dim and self.q_rank is not None:
             raise ConfigError("latent attention: rotated dimensions go with queries that come straight from a projection")
         # the sizes the attention kernels see: one key/value head as wide as the (widened) latent and the rotated part
@@ -80,6 +89,10 @@ class LatentAttention(Mixer):
             p["q"] = ParamSpec((H * (dk + dr), h))
         if self.output_gate:
             p["g"] = ParamSpec((H * dv, h))
+        if self.head_gate:
+            p["g"] = ParamSpec((H, h))
+        if self.sink:
+            p["sink"] = ParamSpec((H,), "normal", 0.0, 1.0)
         return p
 
     def cache_need(self):
@@ -97,7 +110,7 @@ class LatentAttention(Mixer):
         H, dk, dv, R, D, dr = self.n_heads, self.key_dim, self.value_dim, self.kv_rank, self.head_dim, self.rot_dim
         keep = lambda t: t.to(device).to(torch.float32 if dtype == torch.float32 else t.dtype)
         first = [keep(tensors["dq"] if self.q_rank is not None else tensors["q"]), keep(tensors["dkv"])]
-        if self.output_gate:
+        if self.output_gate or self.head_gate:
             first.append(keep(tensors["g"]))
         common = torch.float32 if any(t.dtype == torch.float32 for t in first) else first[0].dtype
         rows, self.first_offsets, at = [], [], 0
@@ -124,7 +137,9 @@ class LatentAttention(Mixer):
         f32 = lambda n: tensors[n].to(device=device, dtype=torch.float32)
         mul = self.scale * D ** 0.5   # the attention kernels divide every score by sqrt(their head size)
         q_at, c_at = self.first_offsets[0], self.first_offsets[1]
-        self.gate_at = self.first_offsets[2] if self.output_gate else None
+        self.gate_at = self.first_offsets[2] if self.output_gate or self.head_gate else None
+        self.sinks = f32("sink").contiguous() if self.sink else None
+        turn = {"half_pairs": dr // 2} if dr and self.position.pairing == PAIRING_CODES["half"] else {"rotate": True}
         magnitude = float(getattr(self.position, "magnitude", 1.0)) if dr else 1.0
         seg, TO_K, TO_V = ops.head_row_segment, ops.TO_CACHE_KEYS, ops.TO_CACHE_VALUES
         if self.q_rank is not None:
@@ -136,36 +151,54 @@ class LatentAttention(Mixer):
             self.norm_weights = f32("dkv_norm").contiguous()
             # every head's plain part times the scale, its rotated part turned by the position (and times the scale)
             plain = seg(q_at, H, dk, 0, dk, mul=mul, src_stride=dk + dr, dst_stride=dk + dr)
-            turned = seg(q_at + dk, H, dr, dk, dr, mul=mul * magnitude, rotate=True, src_stride=dk + dr, dst_stride=dk + dr)
+            turned = seg(q_at + dk, H, dr, dk, dr, mul=mul * magnitude, src_stride=dk + dr, dst_stride=dk + dr, **turn)
             self.query_segment = ops.head_row_segments(*([plain, turned] if dr else [plain]))
             latent_weight = 0
         # c, once as (part of) a key row and once as a value row of its cache page; the rotated key part behind it
         latent = [seg(c_at, 1, R, 0, R if dr else D, -1, True, latent_weight, target=TO_K, cache_dim=D if dr else -1),
                   seg(c_at, 1, R, 0, D, -1, True, latent_weight, target=TO_V)]
         if dr:
-            latent.append(seg(c_at + R, 1, dr, R, D - R, mul=magnitude, rotate=True, target=TO_K, cache_dim=D))
+            latent.append(seg(c_at + R, 1, dr, R, D - R, mul=magnitude, target=TO_K, cache_dim=D, **turn))
         self.latent_segments = ops.head_row_segments(*latent)
 
     def _rotary(self, ctx: StepContext):
         return (ctx.positions, self.position.inverse_frequencies(ctx.device)) if self.rot_dim else None
 
-    def forward(self, x, ctx: StepContext, cache: KVView, residual, writes_cache=True, then_norm=None):
-        H, dk, dv, D, T, dr = self.n_heads, self.key_dim, self.value_dim, self.head_dim, x.shape[0], self.rot_dim
+    def open_columns(self):
+        return self.n_heads * self.value_dim
+
+    def take_output(self):
+        weight, self.o = self.o.weight, None
+        return weight, None
+
+    def take_input(self):
+        weight, self.down = self.down.weight, None
+        return weight
+
+    def takes_scaled_rows(self, ctx: StepContext) -> bool:
+        return ctx.all_decode and self.down is not None and self.down.links_with(ctx.n_tokens, ctx.dtype)
+
+    def rows_into(self, x, ctx: StepContext, cache: KVView, rows, writes_cache=True, mul=1.0):
+        self.rows_from(self.down.store(x, ctx.dtype, ctx.empty), ctx, cache, rows, writes_cache, mul)
+
+    def rows_from(self, raw, ctx: StepContext, cache: KVView, rows, writes_cache=True, mul=1.0):
+        """``raw`` [T, queries (or q_rank) | kv_rank + rot_dim | gate]."""
+        assert mul == 1.0
+        H, dk, dv, D, T, dr = self.n_heads, self.key_dim, self.value_dim, self.head_dim, raw.shape[0], self.rot_dim
         table = ctx.page_tables[cache.group]
-        down = self.down.store(x, ctx.dtype, ctx.empty)                       # [T, queries (or q_rank) | kv_rank + rot_dim | gate]
         if writes_cache:
-            ops.head_rows(down, None, self.latent_segments, self.norm_eps, None, self.norm_weights,
+            ops.head_rows(raw, None, self.latent_segments, self.norm_eps, None, self.norm_weights,
                           cache=(ctx.positions, ctx.seq_ids, table, cache.k, cache.v), rotary=self._rotary(ctx))
         if self.q_rank is not None:
             c_q = ctx.empty((T, self.q_pad), ctx.dtype)
-            ops.head_rows(down, c_q, self.query_segment, self.norm_eps, None, self.norm_weights)
+            ops.head_rows(raw, c_q, self.query_segment, self.norm_eps, None, self.norm_weights)
             q = self.uq.store(c_q[:, :self.q_rank], ctx.dtype, ctx.empty)     # [T, H dk]
         else:
             q = ctx.empty((T, H * (dk + dr)), ctx.dtype)
-            ops.head_rows(down, q, self.query_segment, self.norm_eps, None, None, rotary=self._rotary(ctx))
+            ops.head_rows(raw, q, self.query_segment, self.norm_eps, None, None, rotary=self._rotary(ctx))
         carried = ctx.empty((T, H * D), ctx.dtype)                            # queries in the latent space
         ops.gemm_per_head(q, self.carry_in, carried)
-        heads = ctx.empty((T, H * dv), ctx.dtype)
+        gate = raw[:, self.gate_at:self.gate_at + H] if self.head_gate else None
         if ctx.all_decode and H > self.DECODE_GROUP and ops.attention_decode_supported(ctx.dtype, self.DECODE_GROUP, 1, D):
             # the decode kernel takes up to DECODE_GROUP query heads per key/value head: the heads go in groups, each
             # group over the same cached latents
@@ -174,19 +207,20 @@ class LatentAttention(Mixer):
                 n = min(self.DECODE_GROUP, H - g)
                 part = ctx.empty((T, n * D), ctx.dtype)
                 ops.attention_decode(carried[:, g * D:], carried.stride(0), part, ctx.kv_lens, table, cache.k, cache.v, n, 1,
-                                     D, self.window or 0, splits, early_start=early)
-                ops.gemm_per_head(part, self.carry_out[g:g + n], heads[:, g * dv:(g + n) * dv])
+                                     D, self.window or 0, splits, early_start=early,
+                                     sinks=self.sinks[g:g + n] if self.sink else None, gate=gate[:, g:] if self.head_gate else None)
+                ops.gemm_per_head(part, self.carry_out[g:g + n], rows[:, g * dv:(g + n) * dv])
         else:
             out = ctx.empty((T, H * D), ctx.dtype)
-            if not fast.try_attention(carried, out, ctx, table, cache, self):
-                n_rows = T * H
-                splits = 1 if n_rows >= 1024 else max(1, min(16, 1024 // n_rows, ctx.capacity(cache.group) // 512))
-                ops.attention_paged(carried, carried.stride(0), out, ctx.positions, ctx.seq_ids, table, cache.k, cache.v,
-                                    H, 1, D, self.window or 0, n_splits=splits)
-            ops.gemm_per_head(out, self.carry_out, heads)
+            attend(self, carried, out, ctx, table, cache, gate)
+            ops.gemm_per_head(out, self.carry_out, rows)
         if self.output_gate:
-            ops.gate_rows(heads, down[:, self.gate_at:], "sigmoid")
-        return self.o.add_to(heads, residual, then_norm)
+            ops.gate_rows(rows, raw[:, self.gate_at:], "sigmoid")
+
+    def forward(self, x, ctx: StepContext, cache: KVView, residual, writes_cache=True, then_norm=None):
+        rows = ctx.empty((x.shape[0], self.open_columns()), ctx.dtype)
+        self.rows_into(x, ctx, cache, rows, writes_cache)
+        return self.o.add_to(rows, residual, then_norm)
 
 
 register_mixer("latent_attention", LatentAttention)

@@ -1,5 +1,5 @@
 """Recurrent mixers whose memory is one matrix per head that decays and gains an outer product per token, without the
-delta rule's correction:  S_t = diag(g_t) S_(t-1) + k_t (b_t v_t)^T,  o_t = S_t^T q_t.  Three of them:
+delta rule's correction:  S_t = diag(g_t) S_(t-1) + k_t (b_t v_t)^T,  o_t = S_t^T q_t.  Four of them:
 
 ``GatedLinearAttention`` (``gla``): a decay per key channel from a low-rank projection,
 
@@ -20,10 +20,18 @@ delta rule's correction:  S_t = diag(g_t) S_(t-1) + k_t (b_t v_t)^T,  o_t = S_t^
     q and k turned by the token's position (halves; optional) ;  q times ``scale`` (it stands for a factor on the keys as well)
     y = W_o ( norm(o) * gate(W_g x) )      norm over each head's numbers or over all heads together, with a weight or none
 
+``MatrixMemory`` (``mlstm``): an exponential input gate and a forget gate per head and token, both soft-capped logarithms,
+
+    q = W_q x * d_k^(-1/2), k = W_k x  [heads, d_k] ;  v = W_v x  [heads, d_v]
+    i = cap tanh((W_i x + b_i) / cap),  f = log sigmoid(cap tanh((W_f x + b_f) / cap))  [heads]
+    m_t = max(f + m_(t-1), i) from m = 0 ;  g = e^(f + m_(t-1) - m_t), b = e^(i - m_t) ;  n_t = g n_(t-1) + b k_t
+    o = S^T q / (max(|n . q|, e^(-m)) + 1e-6) ;  y = W_o ( o / rms(o) per head * norm_weight * gate(W_g x) )
+
 All keep, per sequence, S of every head in 32 bits (and the convolution's last inputs) in one row of their cache slot,
 starting from zero.  Decays, step sizes, the recurrence and the output norms are 32-bit in both precisions; projections
 and the convolution are computed in the run's precision.  The scan is the kernel of the delta rule, told to leave out
-the correction; a decay fixed per head has kernels of its own, which take runs of tokens at once (``ops.fixed_decay``)."""
+the correction; a decay fixed per head and the matrix memory have kernels of their own, which take runs of tokens at once
+(``ops.fixed_decay``, ``ops.matrix_memory``)."""
 from __future__ import annotations
 
 import torch
@@ -173,6 +181,7 @@ class StateSpaceDuality(Mixer):
 
 class FixedDecayAttention(Mixer, OpenEnded):
     graph_safe = True
+    gives_input = True
     pad_safe = False
 
     def __init__(self, hidden_size: int, n_heads: int, head_dim: int, value_dim: int, decay, norm_eps: float, *,
@@ -274,6 +283,79 @@ class FixedDecayAttention(Mixer, OpenEnded):
         return self.o.add_to(rows, residual, then_norm)
 
 
+class MatrixMemory(Mixer, OpenEnded):
+    graph_safe = True
+    pad_safe = False
+    gives_input = True
+
+    def __init__(self, hidden_size: int, n_heads: int, head_dim: int, value_dim: int, gate_cap: float, norm_eps: float, *,
+                 gate: str = "sigmoid"):
+        """``gate_cap``: the soft cap on both gates' logits.  ``gate``: the activation of the output gate."""
+        if min(n_heads, head_dim, value_dim) < 1 or head_dim > ops.MAX_MEMORY_KEYS:
+            raise ConfigError(f"matrix memory: key size {head_dim} must be between 1 and {ops.MAX_MEMORY_KEYS}, heads and value size positive")
+        if not gate_cap > 0:
+            raise ConfigError(f"matrix memory: the gates' cap must be positive, got {gate_cap}")
+        if gate not in ops.GATE_ACTIVATIONS:
+            raise ConfigError(f"matrix memory: gate {gate!r}; known: {', '.join(sorted(ops.GATE_ACTIVATIONS))}")
+        self.hidden_size, self.n_heads, self.key_dim, self.value_dim = int(hidden_size), int(n_heads), int(head_dim), int(value_dim)
+        self.cap, self.norm_eps, self.gate, self.scale = float(gate_cap), float(norm_eps), gate, int(head_dim) ** -0.5
+        self.inputs: Linear | None = None
+        self.o: Linear | None = None
+
+    def parameters(self):
+        H, dk, dv, h = self.n_heads, self.key_dim, self.value_dim, self.hidden_size
+        return {"q": ParamSpec((H * dk, h)), "k": ParamSpec((H * dk, h)), "v": ParamSpec((H * dv, h)), "g": ParamSpec((H * dv, h)),
+                "o": ParamSpec((h, H * dv)), "norm": ParamSpec((H * dv,), "norm"), "i": ParamSpec((H, h)), "f": ParamSpec((H, h)),
+                "i_bias": ParamSpec((H,), "normal", -1.0, 1.0), "f_bias": ParamSpec((H,), "normal", 4.0, 1.0)}
+
+    def cache_need(self):
+        return StateNeed((ops.matrix_memory_state(self.n_heads, self.key_dim, self.value_dim),), torch.float32)
+
+    def load(self, tensors, dtype, device):
+        run = lambda t: t.to(device).to(torch.float32 if dtype == torch.float32 else t.dtype)
+        f32 = lambda n: tensors[n].to(device=device, dtype=torch.float32).contiguous()
+        self.inputs, (self.q_off, self.k_off, self.v_off, self.g_off, self.i_off, self.f_off) = _stacked(
+            [run(tensors[n]) for n in ("q", "k", "v", "g", "i", "f")], device)
+        self.o = Linear(run(tensors["o"]).contiguous())
+        self.weight, self.i_bias, self.f_bias = f32("norm"), f32("i_bias"), f32("f_bias")
+
+    def open_columns(self):
+        return self.n_heads * self.value_dim
+
+    def take_output(self):
+        weight, self.o = self.o.weight, None
+        return weight, None
+
+    def take_input(self):
+        weight, self.inputs = self.inputs.weight, None
+        return weight
+
+    def takes_scaled_rows(self, ctx: StepContext) -> bool:
+        return ctx.all_decode and self.inputs is not None and self.inputs.links_with(ctx.n_tokens, ctx.dtype)
+
+    def rows_into(self, x, ctx: StepContext, cache: StateView, rows, writes_cache=True, mul=1.0):
+        self.rows_from(self.inputs.store(x, ctx.dtype, ctx.empty), ctx, cache, rows, writes_cache, mul)
+
+    def rows_from(self, raw, ctx: StepContext, cache: StateView, rows, writes_cache=True, mul=1.0):
+        assert mul == 1.0
+        H, dk, dv, T = self.n_heads, self.key_dim, self.value_dim, raw.shape[0]
+        q, k, v, g, i, f = (raw[:, at:] for at in (self.q_off, self.k_off, self.v_off, self.g_off, self.i_off, self.f_off))
+        args = (q, k, v, (i, f, self.i_bias, self.f_bias), self.cap, cache.data, ctx.slots_dev, ctx.seq_ids, ctx.cu_seqlens, H, dk, dv,
+                ctx.max_q_len)
+        if ops.matrix_memory_finishes(ctx.dtype, ctx.all_decode, dk, dv):
+            ops.matrix_memory(*args, q_scale=self.scale, finish=(rows, g, self.gate, self.norm_eps, self.weight), alloc=ctx.empty)
+            return
+        o = ctx.empty((T, H * dv), torch.float32)
+        ops.matrix_memory(*args, q_scale=self.scale, out=o, alloc=ctx.empty)
+        ops.gated_rmsnorm(o, self.weight, g, rows, H, dv, self.norm_eps, self.gate)
+
+    def forward(self, x, ctx: StepContext, cache: StateView, residual, writes_cache=True, then_norm=None):
+        rows = ctx.empty((x.shape[0], self.open_columns()), ctx.dtype)
+        self.rows_into(x, ctx, cache, rows, writes_cache)
+        return self.o.add_to(rows, residual, then_norm)
+
+
+register_mixer("mlstm", MatrixMemory)
 register_mixer("fixed_decay", FixedDecayAttention)
 register_mixer("gla", GatedLinearAttention)
 register_mixer("ssd", StateSpaceDuality)

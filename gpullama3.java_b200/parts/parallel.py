@@ -3,13 +3,15 @@
 ``ParallelBlock``: the mixer and the feed-forward read the same residual stream, each through a norm of its own, and both
 results join it at once,
 
-    x <- x + mixer(norm_1(x)) + feed_forward(norm_2(x))                         (a layer may have no feed-forward)
+    x <- x + mixer(norm_1(x)) + feed_forward(norm_2(x))         (a layer may have no feed-forward, or one norm for both)
 
 ``ParallelMixers``: two mixers on the same input, each with a factor,  left_scale * left(h) + right_scale * right(h).
 
 Parts whose result is one last product over rows they make (``OpenEnded``) are multiplied together: the mixers and the
 feed-forward write their rows into neighbouring columns of one buffer and ONE product over the joined weights adds the
-layer's whole result into the stream; two mixers likewise start with one product over their joined input weights.  The
+layer's whole result into the stream; two mixers likewise start with one product over their joined input weights, and so do a
+mixer and a feed-forward that read the same norm and both give their first product away.  What a feed-forward adds to the stream
+itself (a mixture's routed experts) it adds before that last product.  The
 factors of ``ParallelMixers`` are applied to the rows in 32 bits.  The two norms differ in their weights alone, so a prompt
 makes both in one read of the stream, and in a decode step the product that completes the stream leaves both copies for
 the next block's products (``ScaledRows``), whose shared row factor they apply themselves.  In a decode step the
@@ -81,19 +83,30 @@ def _join(device) -> None:
 
 class ParallelBlock(Block):
     def __init__(self, mixer, mixer_norm, feed_forward=None, feed_forward_norm=None):
-        if (feed_forward is None) != (feed_forward_norm is None):
-            raise ConfigError("a feed-forward and the norm of its input come together")
+        """``feed_forward_norm`` None: mixer and feed-forward both read the rows of ``mixer_norm``."""
+        if feed_forward is None and feed_forward_norm is not None:
+            raise ConfigError("a norm of the feed-forward's input needs a feed-forward")
         given = {"mixer": mixer, "mixer_norm": mixer_norm, "feed_forward": feed_forward, "feed_forward_norm": feed_forward_norm}
         super().__init__(**{k: v for k, v in given.items() if v is not None})
         for k, v in given.items():
             setattr(self, k, v)
         self.out: Linear | None = None     # the joined last product, where every part gives its own away
+        self.inputs: Linear | None = None  # the joined first product, where both parts read one norm and give theirs away
 
     def after_load(self):
         sublayers = [p for p in (self.mixer, self.feed_forward) if p is not None]
         if all(isinstance(p, OpenEnded) for p in sublayers):
             self.columns = [p.open_columns() for p in sublayers]
-            self.out = _joined([p.take_output() for p in sublayers])
+            self.out = _joined([p.take_output() for p, n in zip(sublayers, self.columns) if n])
+            if self.shares_norm and all(p.gives_input for p in sublayers):
+                ins = [p.take_input() for p in sublayers]
+                common = torch.float32 if any(w.dtype == torch.float32 for w in ins) else ins[0].dtype
+                self.input_columns = ins[0].shape[0]
+                self.inputs = Linear(torch.cat([w.to(common) for w in ins], dim=0).contiguous())
+
+    @property
+    def shares_norm(self) -> bool:
+        return self.feed_forward is not None and self.feed_forward_norm is None
 
     @property
     def graph_safe(self):
@@ -104,7 +117,7 @@ class ParallelBlock(Block):
         return all(p.pad_safe for p in all_parts(self).values())
 
     def first_norm(self):
-        if self.feed_forward is None:
+        if self.feed_forward_norm is None:
             return self.mixer_norm
         return _as_pair(self.mixer_norm, self.feed_forward_norm)
 
@@ -113,10 +126,14 @@ class ParallelBlock(Block):
         return (self.out is not None and first is not None and first.row_factor_form() is not None
                 and all(p.takes_scaled_rows(ctx) for p in (self.mixer, self.feed_forward) if p is not None))
 
+    def leaves_scaled_rows(self, ctx: StepContext) -> bool:
+        return ctx.all_decode and self.out is not None
+
     def _normed(self, residual, ctx: StepContext):
         """The inputs of the mixer and the feed-forward (None without one)."""
-        if self.feed_forward is None:
-            return self.mixer_norm.forward(residual, ctx.dtype, alloc=ctx.empty), None
+        if self.feed_forward_norm is None:
+            h = self.mixer_norm.forward(residual, ctx.dtype, alloc=ctx.empty)
+            return h, h
         pair = _as_pair(self.mixer_norm, self.feed_forward_norm)
         if pair is not None and pair.second_form().dtype == torch.float32:
             weight, eps, _ = pair.row_factor_form()
@@ -130,7 +147,7 @@ class ParallelBlock(Block):
         if x_in is None:
             h, g = self._normed(residual, ctx)
         else:
-            h, g = x_in if isinstance(x_in, tuple) else (x_in, None)
+            h, g = x_in if isinstance(x_in, tuple) else (x_in, x_in)
         if self.out is None:    # (a part that keeps its last product to itself: one after the other, both inputs made before)
             self.mixer.forward(h, ctx, cache, residual, writes_cache)
             if self.feed_forward is not None:
@@ -140,14 +157,30 @@ class ParallelBlock(Block):
         n = self.columns[0]
         if self.feed_forward is None:
             self.mixer.rows_into(h, ctx, cache, rows, writes_cache)
-        elif ctx.all_decode:
-            with _beside(ctx.device):
+            return self.out.add_to(rows, residual, then_norm)
+        raw = self.inputs.store(h, ctx.dtype, ctx.empty) if self.inputs is not None else None
+
+        def mix():
+            if raw is not None:
+                self.mixer.rows_from(raw[:, :self.input_columns], ctx, cache, rows[:, :n], writes_cache)
+            else:
+                self.mixer.rows_into(h, ctx, cache, rows[:, :n], writes_cache)
+
+        def feed_forward():
+            if raw is not None:
+                self.feed_forward.rows_from(raw[:, self.input_columns:], ctx, None, rows[:, n:])
+            elif self.columns[1]:
                 self.feed_forward.rows_into(g, ctx, None, rows[:, n:])
-            self.mixer.rows_into(h, ctx, cache, rows[:, :n], writes_cache)
+            self.feed_forward.adds_itself(g, ctx, residual)
+
+        if ctx.all_decode:
+            with _beside(ctx.device):
+                feed_forward()
+            mix()
             _join(ctx.device)
         else:
-            self.mixer.rows_into(h, ctx, cache, rows[:, :n], writes_cache)
-            self.feed_forward.rows_into(g, ctx, None, rows[:, n:])
+            mix()
+            feed_forward()
         return self.out.add_to(rows, residual, then_norm)
 
 

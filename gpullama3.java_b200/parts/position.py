@@ -107,15 +107,18 @@ def yarn_inverse_frequencies(dims: int, base: float, factor: float, original: fl
 
 
 class YarnRotaryPositionEncoding(PositionEncoding):
-    """Rotary encoding over interleaved pairs with frequencies stretched for contexts longer than the ``original`` one
+    """Rotary encoding with frequencies stretched for contexts longer than the ``original`` one
     (``yarn_inverse_frequencies``); cosine and sine are multiplied by ``magnitude`` = magnitude_slope ln(factor) + 1.
     Without ``factor`` (or with 1) it is the plain rotary encoding of base ``base``."""
     graph_safe = True
     pad_safe = True
 
     def __init__(self, rotary_dim: int, base: float, factor: float | None = None, original: float | None = None,
-                 fast: float = 32.0, slow: float = 1.0, magnitude_slope: float = 0.1, min_ramp_width: float = 0.001):
-        self.rotary_dim, self.pairing, self.base = int(rotary_dim), PAIRING_CODES["interleaved"], float(base)
+                 fast: float = 32.0, slow: float = 1.0, magnitude_slope: float = 0.1, min_ramp_width: float = 0.001,
+                 pairing: str = "interleaved"):
+        if pairing not in PAIRING_CODES:
+            raise ValueError(f"pairing must be one of {sorted(PAIRING_CODES)}, got {pairing!r}")
+        self.rotary_dim, self.pairing, self.base = int(rotary_dim), PAIRING_CODES[pairing], float(base)
         if self.rotary_dim % 2 or self.rotary_dim < 2:
             raise ValueError(f"rotary_dim {rotary_dim} must be even and positive")
         self.factor = float(factor) if factor else 1.0

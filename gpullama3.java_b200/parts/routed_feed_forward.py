@@ -8,6 +8,11 @@
 With ``router_bias`` a learned vector joins the logits z.  With one group and ``weight_eps`` 0 the weights are the softmax
 over the chosen logits alone (s_e over the chosen s is exp(z_e) over the chosen exp(z)).
 
+With ``score="sigmoid"`` every expert's score is the sigmoid of its own logit.  With ``choice_correction`` a learned vector joins the
+scores for the choice alone: the experts are chosen by s + correction and weighed by s.  ``weight_scale``: a last factor on the
+weights.  ``activation`` may be one without a gate (``relu_squared``): expert e is then down_e( act(up_e h) ).  ``shared_size``: a
+further expert of that inner size that every token runs through, its result times sigmoid(w_sg h), one number per token.
+
 With ``router="table"`` there is no router product: row ``token id`` of an integer table [vocabulary, top] names the token's
 experts, and every one of them weighs 1 / top.
 
@@ -26,18 +31,23 @@ import torch
 from ..config.base import ConfigError
 from ..kernels import ops
 from ..weights.loader import ParamSpec
-from .base import FeedForward, StepContext, register_feed_forward
+from .base import FeedForward, OpenEnded, StepContext, register_feed_forward
 from .linear import Linear
 
 
-class RoutedFeedForward(FeedForward):
+def _pad8(n: int) -> int:
+    return -(-n // 8) * 8
+
+
+class RoutedFeedForward(FeedForward, OpenEnded):
     graph_safe = True    # (decode steps: the pair kernels read the routing from device memory)
     pad_safe = False     # a prompt pass may read the experts' row counts on the host
 
     def __init__(self, hidden_size: int, intermediate_size: int, n_experts: int, top: int, groups: int = 1,
                  keep_groups: int | None = None, activation: str = "silu", limit: float | None = None, slope: float = 1.0,
                  weight_eps: float = 1e-20, router: str = "learned", vocab_size: int | None = None,
-                 router_bias: bool = False):
+                 router_bias: bool = False, score: str = "softmax", choice_correction: bool = False, weight_scale: float = 1.0,
+                 shared_size: int | None = None):
         keep_groups = groups if keep_groups is None else keep_groups
         if router not in ("learned", "table"):
             raise ConfigError(f"routed feed-forward: router {router!r}; known: learned, table")
@@ -46,8 +56,19 @@ class RoutedFeedForward(FeedForward):
         if router_bias and router != "learned":
             raise ConfigError("routed feed-forward: only a learned router has logits a bias can join")
         self.routing, self.vocab_size, self.router_bias = router, int(vocab_size or 0), bool(router_bias)
-        if activation not in ops.ACTIVATION_CODES:
-            raise ConfigError(f"feed-forward activation {activation!r}; known: {', '.join(sorted(ops.ACTIVATION_CODES))}")
+        self.gated = activation not in ops.UNGATED_ACTIVATIONS
+        if self.gated and activation not in ops.ACTIVATION_CODES:
+            raise ConfigError(f"feed-forward activation {activation!r}; known: "
+                              f"{', '.join(sorted([*ops.ACTIVATION_CODES, *ops.UNGATED_ACTIVATIONS]))}")
+        if score not in ops.ROUTER_SCORES:
+            raise ConfigError(f"routed feed-forward: scores {score!r}; known: {', '.join(sorted(ops.ROUTER_SCORES))}")
+        if (choice_correction or score != "softmax" or weight_scale != 1.0) and router != "learned":
+            raise ConfigError("routed feed-forward: only a learned router has scores")
+        if shared_size is not None and (shared_size < 1 or self.gated):
+            raise ConfigError("routed feed-forward: a shared expert has a positive size and an activation without a gate")
+        self.score, self.choice_correction, self.weight_scale = score, bool(choice_correction), float(weight_scale)
+        self.shared_size = int(shared_size or 0)
+        self.gives_input = self.shared_size > 0
         if activation == "clamped_sigmoid" and (limit is None or not limit > 0):
             raise ConfigError(f"the clamped feed-forward needs a positive limit, got {limit!r}")
         if not (1 <= n_experts <= ops.MAX_EXPERTS) or not (1 <= top <= min(n_experts, ops.MAX_EXPERTS_PER_TOKEN)):
@@ -67,8 +88,14 @@ class RoutedFeedForward(FeedForward):
              {"table": ParamSpec((self.vocab_size, self.top), "int_table", float(self.n_experts))})
         if self.router_bias:
             p["router_bias"] = ParamSpec((self.n_experts,), "normal", 0.0, 0.02)
+        if self.choice_correction:
+            p["correction"] = ParamSpec((self.n_experts,), "normal", 0.0, 0.1)
+        if self.shared_size:
+            p.update({"shared.up": ParamSpec((self.shared_size, self.hidden_size)),
+                      "shared.down": ParamSpec((self.hidden_size, self.shared_size)), "shared.sg": ParamSpec((1, self.hidden_size))})
         for e in range(self.n_experts):
-            p[f"e{e}.gate"] = ParamSpec((self.intermediate_size, self.hidden_size))
+            if self.gated:
+                p[f"e{e}.gate"] = ParamSpec((self.intermediate_size, self.hidden_size))
             p[f"e{e}.up"] = ParamSpec((self.intermediate_size, self.hidden_size))
             p[f"e{e}.down"] = ParamSpec((self.hidden_size, self.intermediate_size))
         return p
@@ -81,14 +108,25 @@ class RoutedFeedForward(FeedForward):
             self.bias = tensors["router_bias"].to(device=device, dtype=torch.float32).contiguous() if self.router_bias else None
         else:
             self.table = tensors["table"].to(device=device, dtype=torch.int32).contiguous()
-        self.w_gate_up = torch.empty((E, 2 * ff, h), dtype=run, device=device)   # gate and up rows interleaved
+        self.correction = tensors["correction"].to(device=device, dtype=torch.float32).contiguous() if self.choice_correction else None
+        self.w_up = torch.empty((E, (2 if self.gated else 1) * ff, h), dtype=run, device=device)   # gated: gate and up rows interleaved
         self.w_down = torch.empty((E, h, ff), dtype=run, device=device)
         for e in range(E):
-            self.w_gate_up[e, 0::2] = tensors[f"e{e}.gate"].to(device=device, dtype=run)
-            self.w_gate_up[e, 1::2] = tensors[f"e{e}.up"].to(device=device, dtype=run)
+            if self.gated:
+                self.w_up[e, 0::2] = tensors[f"e{e}.gate"].to(device=device, dtype=run)
+                self.w_up[e, 1::2] = tensors[f"e{e}.up"].to(device=device, dtype=run)
+            else:
+                self.w_up[e] = tensors[f"e{e}.up"].to(device=device, dtype=run)
             self.w_down[e] = tensors[f"e{e}.down"].to(device=device, dtype=run)
-        self.gate_up = [Linear(self.w_gate_up[e]) for e in range(E)]
+        self.up = [Linear(self.w_up[e]) for e in range(E)]
         self.down = [Linear(self.w_down[e]) for e in range(E)]
+        self.shared_up = self.shared_down = None
+        if self.shared_size:      # one product for the shared expert's rows and its gate's, each group padded to a multiple of 8 rows
+            self.shared_gate_at = _pad8(self.shared_size)
+            w = torch.zeros((self.shared_gate_at + 8, h), dtype=run, device=device)
+            w[:self.shared_size] = tensors["shared.up"].to(device=device, dtype=run)
+            w[self.shared_gate_at] = tensors["shared.sg"].to(device=device, dtype=run)[0]
+            self.shared_up, self.shared_down = Linear(w), Linear(tensors["shared.down"].to(device=device, dtype=run).contiguous())
         # a decode step's launches depend on device memory alone when the streaming kernel takes the rows, or else when
         # the grouped product does (the per-expert products need the runs' lengths on the host)
         grouped = run == torch.bfloat16 and E <= ops.MAX_GEMM_GROUPS and h % 8 == 0 and ff % 8 == 0
@@ -101,7 +139,8 @@ class RoutedFeedForward(FeedForward):
         if self.routing == "table":
             ops.moe_table_route(ctx.tokens, self.table, chosen, weights, self.n_experts)
             return chosen, weights
-        ops.moe_route(x, self.router, chosen, weights, self.groups, self.keep_groups, self.weight_eps, scores, self.bias)
+        ops.moe_route(x, self.router, chosen, weights, self.groups, self.keep_groups, self.weight_eps, scores, self.bias,
+                      score=self.score, correction=self.correction, scale=self.weight_scale)
         return chosen, weights
 
     def as_prompt(self, ctx: StepContext, n_tokens: int) -> bool:
@@ -111,7 +150,8 @@ class RoutedFeedForward(FeedForward):
             return True     # (rows too long to stage for the streaming kernel)
         return (not ctx.all_decode) and n_tokens > 64 and n_tokens * self.top >= 16 * self.n_experts
 
-    def forward(self, x, ctx: StepContext, residual, then_norm=None):
+    def adds_itself(self, x, ctx: StepContext, residual):
+        """The routed experts' weighted sum."""
         T = x.shape[0]
         chosen, weights = self.route(x, ctx)
         pairs = T * self.top
@@ -121,7 +161,7 @@ class RoutedFeedForward(FeedForward):
         y = ctx.empty((pairs, self.intermediate_size), ctx.dtype)
         o = ctx.empty((pairs, self.hidden_size), torch.float32)
         if not self.as_prompt(ctx, T):
-            ops.moe_rows(x, self.w_gate_up, offsets, y, order=order, top=self.top, activation=self.activation,
+            ops.moe_rows(x, self.w_up, offsets, y, order=order, top=self.top, activation=self.activation,
                          gate_args=self.gate_args)
             ops.moe_rows(y, self.w_down, offsets, o)
         else:
@@ -129,15 +169,47 @@ class RoutedFeedForward(FeedForward):
             ops.moe_gather(x, order, xs, self.top)
             # one launch over all experts' tiles, the runs read on the device; where that kernel does not take the operands
             # (the float32 run, odd sizes) one product per expert, for which the runs' lengths come back to the host
-            if not (ops.gemm_tcgen05_grouped(xs, self.w_gate_up, offsets, y, ops.GATED_EPILOGUE_OF[self.activation], self.gate_args)
+            epilogue = ops.GATED_EPILOGUE_OF[self.activation] if self.gated else ops.EPILOGUE_SQUARED_RELU
+            if not (ops.gemm_tcgen05_grouped(xs, self.w_up, offsets, y, epilogue, self.gate_args)
                     and ops.gemm_tcgen05_grouped(y, self.w_down, offsets, o)):
                 bounds = offsets.tolist()
-                for e in range(self.n_experts):
-                    lo, hi = bounds[e], bounds[e + 1]
-                    if hi > lo:
-                        self.gate_up[e].gated_into(xs[lo:hi], y[lo:hi], self.activation, self.gate_args)
-                        self.down[e].into(y[lo:hi], o[lo:hi])
+                runs = [(e, bounds[e], bounds[e + 1]) for e in range(self.n_experts) if bounds[e + 1] > bounds[e]]
+                for e, lo, hi in runs:
+                    if self.gated:
+                        self.up[e].gated_into(xs[lo:hi], y[lo:hi], self.activation, self.gate_args)
+                    else:
+                        self.up[e].into(xs[lo:hi], y[lo:hi])
+                if not self.gated:
+                    ops.bias_act_rows(y, None, self.activation)
+                for e, lo, hi in runs:
+                    self.down[e].into(y[lo:hi], o[lo:hi])
         ops.moe_combine(o, place, weights, residual)
+
+    # ---- the shared expert: rows before a last product
+    def open_columns(self):
+        return self.shared_size
+
+    def take_output(self):
+        weight, self.shared_down = self.shared_down.weight, None
+        return weight, None
+
+    def take_input(self):
+        weight, self.shared_up = self.shared_up.weight, None
+        return weight
+
+    def rows_into(self, x, ctx: StepContext, cache, rows, writes_cache=True, mul=1.0):
+        self.rows_from(self.shared_up.store(x, ctx.dtype, ctx.empty), ctx, cache, rows, writes_cache, mul)
+
+    def rows_from(self, raw, ctx: StepContext, cache, rows, writes_cache=True, mul=1.0):
+        assert mul == 1.0
+        ops.bias_act_rows(raw[:, :self.shared_size], None, self.activation, out=rows, gate=raw[:, self.shared_gate_at:])
+
+    def forward(self, x, ctx: StepContext, residual, then_norm=None):
+        self.adds_itself(x, ctx, residual)
+        if self.shared_size:
+            rows = ctx.empty((x.shape[0], self.shared_size), ctx.dtype)
+            self.rows_into(x, ctx, None, rows)
+            self.shared_down.add_to(rows, residual)
         return None
 
 
