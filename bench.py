@@ -501,6 +501,25 @@ def fazezen_config(z):
     return {"architecture": "Fazezen", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-6}, "layers": layers}
 
 
+def zanezen_config(z):
+    """Layers in the order differential attention (half the heads, two maps of `dim` each over values of twice `dim`), matrix memory
+    (half the heads, values of twice `dim`), latent attention (96 latent + 32 rotated dimensions: one key/value head of 128),
+    repeated; feed-forwards dense and routed in turn (8 experts without gate of half the dense width, 2 per token, and a shared one of
+    the same width: the same products per token as the dense one)."""
+    H, G, d = z["heads"] // 2, max(1, z["kv_heads"] // 2), z["dim"]
+    att = {"heads": H, "kv_heads": G, "dim": d, "vdim": 2 * d, "scale": d ** -0.5, "diff": 0.35, "conv": 4, "softcap": 30.0,
+           "rot": {"base": 50000.0, "dims": d // 2, "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+    mem = {"heads": H, "dim": d, "vdim": 2 * d, "gate_cap": 15.0}
+    lat = {"heads": z["heads"], "dim": d, "rot_dim": 32, "vdim": d, "kv_rank": z["kv_rank"] - 32, "scale": (d + 32) ** -0.5,
+           "rot": {"base": 10000.0, "dims": 32}}
+    dense = {"kind": "dense", "ff": z["ff"]}
+    moe = {"kind": "moe", "expert": {"ff": z["ff"] // 2}, "router": {"experts": 8, "top": 2, "scale": 1.0}, "shared": {"ff": z["ff"] // 2}}
+    kinds = (("attention", att), ("mlstm", mem), ("latent_attention", lat))
+    layers = [{"type": kinds[i % 3][0], "mixer": dict(kinds[i % 3][1]), "mlp": dense if i % 2 == 0 else moe} for i in range(z["layers"])]
+    return {"architecture": "Zanezen", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0},
+            "residual_mult": 0.8, "layers": layers}
+
+
 def llama_like(z):
     return {"architectures": ["LlamaForCausalLM"], "num_hidden_layers": z["layers"], "hidden_size": z["width"],
             "num_attention_heads": z["heads"], "num_key_value_heads": z["kv_heads"], "head_dim": z["dim"],
@@ -588,6 +607,9 @@ DESIGNS = {
                                 "token)", ("pekerax", "llama")),
     "fazezen": (fazezen_config, "Fazezen, layers attention within runs of positions beside retention / lightning attention / "
                                 "lightning attention, dense feed-forwards beside the mixers", ("guduzen", "gatuzen", "llama")),
+    "zanezen": (zanezen_config, "Zanezen, layers differential attention with convolution and soft cap / matrix memory / latent "
+                                "attention with sink and head gates, feed-forwards beside the mixers, dense and routed in turn (8 "
+                                "experts, 2 per token, one shared)", ("bisudra", "fazezen", "gatuzen")),
 }
 
 
@@ -599,7 +621,8 @@ def run_design(args, peaks, peak_source, clocks) -> int:
     sizes = {}
     name = args.design
     make, what, beside = DESIGNS[name]
-    others = {"guduzen": guduzen_config, "pekerax": pekerax_config, "gatuzen": gatuzen_config, "llama": llama_like}
+    others = {"guduzen": guduzen_config, "pekerax": pekerax_config, "gatuzen": gatuzen_config, "bisudra": bisudra_config,
+              "fazezen": fazezen_config, "llama": llama_like}
     for key in (args.design_sizes.split(",") if args.design_sizes else sorted(DESIGN_SIZES, reverse=True)):
         z = DESIGN_SIZES[key]
         sizes[key] = {"sizes": z, name: run_design_arm(make(z), f"{name} {key}", args, peaks)}

@@ -213,18 +213,19 @@ def expert(h, W, p):
     return product(squared_relu(product(h, W[p + "up"])), W[p + "down"])
 
 
-MARGINS = []    # while a list is put here, every routed layer appends its margins [T]
+_MARGINS = [None]    # a list that every routed layer appends its margins [T] to while ``forward(..., margins=list)`` runs
 
 
 def mixture(h, W, p, mlp):
     f = _ROUNDING[0]
     chosen, weights, margin = route(h if f is None else f(h), W, p, mlp["router"])
-    if MARGINS:
-        MARGINS[0].append(margin)
+    if _MARGINS[0] is not None:
+        _MARGINS[0].append(margin)
     y = torch.zeros_like(h)
-    for t in range(h.shape[0]):
-        for e, w in zip(chosen[t].tolist(), weights[t]):
-            y[t] += w * expert(h[t:t + 1], W, p + f"e{e}.")[0]
+    for e in range(mlp["router"]["experts"]):
+        t, place = (chosen == e).nonzero(as_tuple=True)
+        if t.numel():
+            y[t] += weights[t, place][:, None] * expert(h[t], W, p + f"e{e}.")
     if mlp.get("shared") is not None:
         y = y + expert(h, W, p + "shared.") * torch.sigmoid(product(h, W[p + "shared.sg"]))
     return y
@@ -242,13 +243,13 @@ def layer(x, W, config, i):
     return x + float(config["residual_mult"]) * y
 
 
-def forward(config, weights, tokens, return_layers=False, reads=None):
+def forward(config, weights, tokens, return_layers=False, reads=None, margins=None):
     """Logits [T, vocab] of one sequence (float64); with ``return_layers`` also the stream after every layer.  ``reads``:
     a rounding applied to what every product reads and to what it returns (to see how far roundings alone move the
-    result)."""
+    result).  ``margins``: a list every routed layer appends its margins to (see ``route``)."""
     W = {k: (v.to(F) if v.is_floating_point() else v) for k, v in weights.items()}
     tokens = torch.as_tensor(tokens, dtype=torch.long)
-    _ROUNDING[0] = reads
+    _ROUNDING[0], _MARGINS[0] = reads, margins
     x = W["embed"][tokens] * float(config["embedding"]["scale"])
     layers = []
     for i in range(len(config["layers"])):
@@ -256,5 +257,5 @@ def forward(config, weights, tokens, return_layers=False, reads=None):
         layers.append(x)
     last = rms_norm(x, W["final.norm"], float(config["norm"]["eps"]))
     logits = (reads(last) if reads else last) @ W["head"].T
-    _ROUNDING[0] = None
+    _ROUNDING[0] = _MARGINS[0] = None
     return (logits, layers) if return_layers else logits
