@@ -505,8 +505,9 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_row_stride, _
         }
         const int head = kvh * group + row;
         if (n_splits == 1) {
-            if (terms.gate) acc *= 1.0f / (1.0f + expf(-__bfloat162float(terms.gate[(size_t)seq * terms.ld_gate + head])));
-            out[((size_t)seq * n_heads + head) * D + d] = __float2bfloat16_rn(acc / l);
+            // (the quotient before the gate, as the merge kernel has it: a result does not depend on the number of spans)
+            const float gate = terms.gate ? 1.0f / (1.0f + expf(-__bfloat162float(terms.gate[(size_t)seq * terms.ld_gate + head]))) : 1.f;
+            out[((size_t)seq * n_heads + head) * D + d] = __float2bfloat16_rn(acc / l * gate);
         } else {
             const size_t p = (size_t)(span_first + split) * n_heads + head;
             part_o[p * D + d] = acc;

@@ -518,18 +518,21 @@ fixed_decay_outputs_kernel(FixedDecayArgs a) {
             const __nv_bfloat16* gate = (const __nv_bfloat16*)a.gate + t * a.ld_gate + (size_t)h * a.d_v;
             __nv_bfloat16* dst = (__nv_bfloat16*)a.rows + t * a.ld_rows + (size_t)h * a.d_v;
             const bool pairs = (((uintptr_t)gate | (uintptr_t)dst) & 3) == 0;
+            uint32_t g2[NS / 8];      // (all asked for before the first result is stored)
+#pragma unroll
+            for (int j = 0; j < NS / 8; ++j)
+                g2[j] = pairs && j * 8 + 2 * tq + 1 < a.d_v ? __ldg(reinterpret_cast<const uint32_t*>(gate + j * 8 + 2 * tq)) : 0u;
 #pragma unroll
             for (int j = 0; j < NS / 8; ++j) {
                 const int c = j * 8 + 2 * tq;
                 if (c + 1 < a.d_v && pairs) {
-                    const uint32_t g2 = *reinterpret_cast<const uint32_t*>(gate + c);
                     *reinterpret_cast<uint32_t*>(dst + c) =
-                        pack_pair(o[j][2 * hh] * scale * gate_32(__uint_as_float(g2 << 16), a.gate_act),
-                                  o[j][2 * hh + 1] * scale * gate_32(__uint_as_float(g2 & 0xffff0000u), a.gate_act));
+                        pack_pair(o[j][2 * hh] * scale * gate_16(__uint_as_float(g2[j] << 16), a.gate_act),
+                                  o[j][2 * hh + 1] * scale * gate_16(__uint_as_float(g2[j] & 0xffff0000u), a.gate_act));
                 } else {
                     for (int e = 0; e < 2; ++e)
                         if (c + e < a.d_v)
-                            dst[c + e] = __float2bfloat16_rn(o[j][2 * hh + e] * scale * gate_32(__bfloat162float(gate[c + e]), a.gate_act));
+                            dst[c + e] = __float2bfloat16_rn(o[j][2 * hh + e] * scale * gate_16(__bfloat162float(gate[c + e]), a.gate_act));
                 }
             }
         } else {

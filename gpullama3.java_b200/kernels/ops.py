@@ -46,6 +46,7 @@ _SIGNATURES = {
     "b200_gemm_generic_batched": ("gemm_generic", [c_void_p, c_int, c_int, ctypes.c_longlong, c_void_p, c_int, c_int,
                                                    ctypes.c_longlong, c_void_p, c_int, c_int, ctypes.c_longlong, c_int, c_int,
                                                    c_int, c_int]),
+    "b200_gemm_heads": ("gemm_heads", [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int]),
     "b200_gemm_decode": ("gemm_decode", [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int,
                                          c_int, c_float, c_float, c_void_p, c_int]),
     "b200_gemm_decode_linked": ("gemm_decode", [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int,
@@ -398,12 +399,18 @@ def gemm_generic(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, epilogue: in
 
 def gemm_per_head(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor) -> None:
     """c[:, h n : (h + 1) n] = a[:, h k : (h + 1) k] @ w[h].T for every head h: a [T, H k], w [H, n, k], c [T, H n].
-    One launch of the plain kernel (32-bit FMA accumulation) for all heads."""
+    One launch for all heads: of a tensor-core kernel for bfloat16 operands that it takes, else of the plain kernel (32-bit FMA
+    accumulation)."""
     _dev(a, w, c)
     H, n, k = w.shape
     T = a.shape[0]
     assert w.is_contiguous() and a.stride(1) == 1 and c.stride(1) == 1
     assert tuple(a.shape) == (T, H * k) and tuple(c.shape) == (T, H * n)
+    if a.dtype == w.dtype == c.dtype == torch.bfloat16 and k % 8 == 0:
+        status = _fn("b200_gemm_heads")(a.data_ptr(), a.stride(0), w.data_ptr(), c.data_ptr(), c.stride(0), T, n, k, H, _stream())
+        if status != _UNSUPPORTED:
+            _check(status, "gemm_heads")
+            return
     _check(_fn("b200_gemm_generic_batched")(a.data_ptr(), dtype_code(a.dtype), a.stride(0), k, w.data_ptr(),
                                             dtype_code(w.dtype), k, n * k, c.data_ptr(), dtype_code(c.dtype), c.stride(0), n,
                                             T, n, k, H, _stream()), "gemm_per_head")

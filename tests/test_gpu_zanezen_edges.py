@@ -39,6 +39,14 @@ def _slow(tensors):
             tensors[n] = t * 2.0
 
 
+def _closed(tensors):
+    for n, t in tensors.items():
+        if n.endswith("mix.i.b"):
+            tensors[n] = torch.linspace(-7.5, -6.0, t.numel())
+        if n.endswith("mix.f.b"):
+            tensors[n] = torch.linspace(1.0, 5.0, t.numel())
+
+
 def _wide_gates(tensors):
     for n, t in tensors.items():
         if n.endswith(("mix.f", "mix.i")):
@@ -155,16 +163,6 @@ def test_every_constant_and_mechanism(session_tmp, dtype):
         differs(name, P.forward(cfg, {**weights, name: kept}, tokens))
     sinkless = {**weights, "l2.mix.sink": torch.full_like(weights["l2.mix.sink"], -1e4)}
     differs("the sink", P.forward(cfg, sinkless, tokens), 0.6)
-    memory = P.matrix_memory
-
-    def without_floor(q, k, v, li, lf):
-        return memory(q, k, v, li + 100.0, lf)       # (gates so large that the divisor never is e^(-m))
-
-    P.matrix_memory = without_floor
-    try:
-        differs("the divisor's floor", P.forward(cfg, weights, tokens), 0.3)
-    finally:
-        P.matrix_memory = memory
     for cut in ((150, None), (90, 31), (149, 3)):
         assert_logits(_run(d, dtype, tokens, *cut), _settled(cfg, weights, tokens, ref), dtype, f"mechanisms, {cut}")
 
@@ -175,6 +173,26 @@ def _settled(cfg, weights, tokens, ref):
     r = reference(cfg, weights, tokens)
     assert torch.equal(r.logits, ref)
     return r
+
+
+@DTYPES
+def test_the_divisors_floor(session_tmp, dtype):
+    """Input gates far below zero: what a memory returns is then so small that the eps of its head's norm counts, and with it the
+    divisor, which is e^(-m) here."""
+    d = make_zanezen_dir(session_tmp, SLOW, seed=3, edit=_closed)
+    cfg, weights = plain_inputs(d)
+    tokens = random_prompts(cfg["vocab"], [80], seed=4)[0]
+    ref = P.forward(cfg, weights, tokens)
+    scale = float(ref.abs().max())
+    memory = P.matrix_memory
+    P.matrix_memory = lambda q, k, v, li, lf: memory(q, k, v, li + 100.0, lf)       # (a divisor that never is e^(-m))
+    try:
+        moved = _moved(P.forward(cfg, weights, tokens), ref, scale)
+    finally:
+        P.matrix_memory = memory
+    assert float((moved > 20).float().mean()) > 0.8, moved.median()
+    for cut in ((80, None), (70, 9), (2, None)):
+        assert_logits(_run(d, dtype, tokens, *cut), ref, dtype, f"floor, {cut}")
 
 
 @DTYPES

@@ -283,3 +283,17 @@ def test_activated_rows_times_a_gate_of_one_number(dtype, T, n):
         want = P.squared_relu(u[:, :n].cpu().to(F)) * torch.sigmoid(u[:, n:n + 1].cpu().to(F))
         _close(wide[:, off:off + n], want, 2e-6 if dtype == torch.float32 else 5e-3)
         assert float(wide[:, :off].abs().sum()) == 0.0 and float(wide[:, off + n:].abs().sum()) == 0.0
+
+
+@DTYPES
+@pytest.mark.parametrize("T, H, n, k", [(1, 3, 128, 96), (8, 20, 32, 128), (70, 2, 40, 24), (200, 4, 130, 56), (65, 5, 11, 8), (300, 1, 300, 512), (40, 3, 9, 14)])
+def test_products_per_head(dtype, T, H, n, k):
+    """Every kernel behind ``gemm_per_head``: sizes on and off the tensor-core kernel's grid, results in columns of a wider buffer."""
+    torch.manual_seed(n)
+    a, w = torch.randn(T, H * k, device="cuda").to(dtype), (torch.randn(H, n, k, device="cuda") / k ** 0.5).to(dtype)
+    want = torch.einsum("thk,hnk->thn", a.cpu().to(F).view(T, H, k), w.cpu().to(F)).reshape(T, H * n)
+    for off in (0, 8, 3):
+        wide = torch.zeros(T, H * n + 16, dtype=dtype, device="cuda")
+        ops.gemm_per_head(a, w, wide[:, off:off + H * n])
+        _close(wide[:, off:off + H * n], want, 3e-6 if dtype == torch.float32 else 6e-3)
+        assert float(wide[:, :off].abs().sum()) == 0.0 and float(wide[:, off + H * n:].abs().sum()) == 0.0
