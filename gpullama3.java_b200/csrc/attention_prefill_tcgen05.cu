@@ -106,6 +106,60 @@ __device__ __forceinline__ void zero_values_beyond_end(__nv_bfloat16* v0, __nv_b
     }
 }
 
+// arithmetic on pairs of floats in one instruction, and the maximum of three
+__device__ __forceinline__ unsigned long long pack2(float a, float b) {
+    unsigned long long v;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(v) : "f"(a), "f"(b));
+    return v;
+}
+__device__ __forceinline__ void unpack2(unsigned long long v, float& a, float& b) {
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(v));
+}
+__device__ __forceinline__ unsigned long long fma2(unsigned long long a, unsigned long long b, unsigned long long c) {
+    unsigned long long d;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+    return d;
+}
+__device__ __forceinline__ unsigned long long add2(unsigned long long a, unsigned long long b) {
+    unsigned long long d;
+    asm("add.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+    return d;
+}
+__device__ __forceinline__ float max3(float a, float b, float c) {
+    float d;
+    asm("max.f32 %0, %1, %2, %3;" : "=f"(d) : "f"(a), "f"(b), "f"(c));
+    return d;
+}
+__device__ __forceinline__ float max3_abs(float a, float b, float c) {
+    float d;
+    asm("max.abs.f32 %0, %1, %2, %3;" : "=f"(d) : "f"(a), "f"(b), "f"(c));
+    return d;
+}
+
+// 32 scores of a row under the soft cap, in units of q.k.  Three special-function results per score (the cap's exponential and
+// reciprocal, the softmax's exponential) would bind the kernel; while no score of the warp is beyond 0.6 of the cap,
+// tanh(x) = x (1 + t (c1 + t (c2 + t (c3 + t c4)))), t = x^2, runs on the multiply-add pipe instead, two scores at a time.  The four
+// numbers are fitted to tanh(x) / x on that range (largest relative error 1e-7, less than the exponential's).
+__device__ __forceinline__ void soft_cap32(float (&v)[32], float cap, float cap_log2) {
+    float m = 0.f;
+#pragma unroll
+    for (int j = 0; j < 32; j += 2) m = max3_abs(m, v[j], v[j + 1]);
+    if (__any_sync(0xffffffffu, m > 0.6f * cap)) {
+#pragma unroll
+        for (int j = 0; j < 32; ++j) v[j] = soft_capped_fast(v[j], cap, cap_log2);
+        return;
+    }
+    const float inv = 1.f / cap;
+    const unsigned long long inv2 = pack2(inv, inv), zero2 = pack2(0.f, 0.f), one2 = pack2(1.f, 1.f);
+    const unsigned long long c1 = pack2(-0.33332622f, -0.33332622f), c2 = pack2(0.13313521f, 0.13313521f);
+    const unsigned long long c3 = pack2(-0.05223111f, -0.05223111f), c4 = pack2(0.01564048f, 0.01564048f);
+#pragma unroll
+    for (int j = 0; j < 32; j += 2) {
+        const unsigned long long z = pack2(v[j], v[j + 1]), x = fma2(z, inv2, zero2), t = fma2(x, x, zero2);
+        unpack2(fma2(fma2(fma2(fma2(fma2(c4, t, c3), t, c2), t, c1), t, one2), z, zero2), v[j], v[j + 1]);
+    }
+}
+
 template <int D, bool TERMS>
 __global__ void __launch_bounds__(kFaThreads, D == 64 ? 2 : 1)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
@@ -290,10 +344,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             for (int c = 0; c < 2; ++c) {
                 float v[32];
                 tmem_ld32(tmem_s + lane_base + half * 64 + c * 32, v);
-                if (TERMS && cap_qk > 0.f) {
-#pragma unroll
-                    for (int j = 0; j < 32; ++j) v[j] = soft_capped_fast(v[j], cap_qk, cap_log2);
-                }
+                if (TERMS && cap_qk > 0.f) soft_cap32(v, cap_qk, cap_log2);
                 uint32_t pk[16];
                 float l0 = 0.f, l1 = 0.f;
 #pragma unroll
@@ -426,31 +477,6 @@ __device__ __forceinline__ void tie32(uint32_t (&r)[32]) {
                       "+r"(r[16]), "+r"(r[17]), "+r"(r[18]), "+r"(r[19]), "+r"(r[20]), "+r"(r[21]), "+r"(r[22]), "+r"(r[23]),
                       "+r"(r[24]), "+r"(r[25]), "+r"(r[26]), "+r"(r[27]), "+r"(r[28]), "+r"(r[29]), "+r"(r[30]), "+r"(r[31])
                  :: "memory");
-}
-
-// arithmetic on pairs of floats in one instruction, and the maximum of three
-__device__ __forceinline__ unsigned long long pack2(float a, float b) {
-    unsigned long long v;
-    asm("mov.b64 %0, {%1, %2};" : "=l"(v) : "f"(a), "f"(b));
-    return v;
-}
-__device__ __forceinline__ void unpack2(unsigned long long v, float& a, float& b) {
-    asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(v));
-}
-__device__ __forceinline__ unsigned long long fma2(unsigned long long a, unsigned long long b, unsigned long long c) {
-    unsigned long long d;
-    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
-    return d;
-}
-__device__ __forceinline__ unsigned long long add2(unsigned long long a, unsigned long long b) {
-    unsigned long long d;
-    asm("add.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
-    return d;
-}
-__device__ __forceinline__ float max3(float a, float b, float c) {
-    float d;
-    asm("max.f32 %0, %1, %2, %3;" : "=f"(d) : "f"(a), "f"(b), "f"(c));
-    return d;
 }
 
 // 16 registers (32 bfloat16) of this thread's row into 16 consecutive columns of tensor memory
@@ -735,9 +761,14 @@ attention_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const _
                     if (!ok) break;
                     if (TERMS && cap_qk > 0.f) {
 #pragma unroll
-                        for (int c = 0; c < 4; ++c)
+                        for (int c = 0; c < 4; ++c) {
+                            float v[32];
 #pragma unroll
-                            for (int i = 0; i < 32; ++i) sr[c][i] = __float_as_uint(soft_capped_fast(__uint_as_float(sr[c][i]), cap_qk, cap_log2));
+                            for (int i = 0; i < 32; ++i) v[i] = __uint_as_float(sr[c][i]);
+                            soft_cap32(v, cap_qk, cap_log2);
+#pragma unroll
+                            for (int i = 0; i < 32; ++i) sr[c][i] = __float_as_uint(v[i]);
+                        }
                     }
                     // probabilities as bfloat16 pairs into this row's lane of P: key k of the block in column k / 2
                     float l4[4] = {0.f, 0.f, 0.f, 0.f};
