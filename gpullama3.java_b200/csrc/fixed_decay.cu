@@ -389,25 +389,7 @@ fixed_decay_outputs_kernel(FixedDecayArgs a) {
         load_tile(ks + p * kRun * ld, ld, a.kt[p] + (size_t)first * a.ld_kt + (size_t)h * a.head_qk, a.ld_kt, n, d_pad, d_pad);
     }
     load_tile(vs, ldv, a.vt + (size_t)first * a.ld_vt + (size_t)h * a.head_v + col0, a.ld_vt, n, NS, (a.d_v - col0 + 7) / 8 * 8);
-    {   // the state before the run, (hi, lo) pairs: four numbers per thread and access where the rows allow it
-        const uint32_t* S = reinterpret_cast<const uint32_t*>(a.runs) + ((size_t)(first_run(a.cu_seqlens, seq) + run) * a.heads + h) * a.d_k * a.d_v;
-        const bool vec = a.d_v % 4 == 0;
-        for (int i = threadIdx.x; i < d_pad * (NS / 4); i += kRunThreads) {
-            const int r = i / (NS / 4), c = (i % (NS / 4)) * 4;
-            uint32_t w[4] = {0, 0, 0, 0};
-            if (r < a.d_k && col0 + c < a.d_v) {
-                if (vec) {
-                    const uint4 x = *reinterpret_cast<const uint4*>(S + (size_t)r * a.d_v + col0 + c);
-                    w[0] = x.x; w[1] = x.y; w[2] = x.z; w[3] = x.w;
-                } else {
-#pragma unroll
-                    for (int e = 0; e < 4; ++e) w[e] = col0 + c + e < a.d_v ? S[(size_t)r * a.d_v + col0 + c + e] : 0u;
-                }
-            }
-            *reinterpret_cast<uint2*>(shi + (size_t)r * ldv + c) = make_uint2(__byte_perm(w[0], w[1], 0x5410), __byte_perm(w[2], w[3], 0x5410));
-            *reinterpret_cast<uint2*>(slo + (size_t)r * ldv + c) = make_uint2(__byte_perm(w[0], w[1], 0x7632), __byte_perm(w[2], w[3], 0x7632));
-        }
-    }
+    load_state_parts<NS>(shi, slo, ldv, reinterpret_cast<const uint32_t*>(a.runs) + ((size_t)(first_run(a.cu_seqlens, seq) + run) * a.heads + h) * a.d_k * a.d_v, a.d_k, a.d_v, col0, d_pad);
     copies_done();
     __syncthreads();
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, mi = lane >> 3, mr = lane & 7, gq = lane >> 2, tq = lane & 3;

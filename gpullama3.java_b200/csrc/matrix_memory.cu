@@ -457,35 +457,17 @@ memory_outputs_kernel(MemoryArgs a) {
     load_tile(ks, ld, a.kt + (size_t)first * a.ld_kt + (size_t)h * a.head_qk, a.ld_kt, n, d_pad, d_pad);
     load_tile(vs, ldv, a.vt + (size_t)first * a.ld_vt + (size_t)h * a.head_v + col0, a.ld_vt, n, NS, (a.d_v - col0 + 7) / 8 * 8);
     const float* U = run_at(a, seq, run, h);
-    if (threadIdx.x < kRun) {
-        const float* F = a.gates + (size_t)h * a.n_tokens + first;
-        const size_t plane = (size_t)a.heads * a.n_tokens;
-        const int i = min((int)threadIdx.x, n - 1);
-        const float f = F[i], m = F[2 * plane + i];
-        w_i[threadIdx.x] = f - m;
-        w_j[threadIdx.x] = F[plane + i] - f;
-        before[threadIdx.x] = expf(f + (m_before(a, seq, seq0, run, h) - m));
-        least[threadIdx.x] = expf(-m);
-    }
+    const float* F = a.gates + (size_t)h * a.n_tokens + first;
+    const size_t plane = (size_t)a.heads * a.n_tokens;
+    const int mine = min((int)threadIdx.x % kRun, n - 1);      // (asked for before the memory's tiles, used behind them)
+    const float f = F[mine], log_in = F[plane + mine], m = F[2 * plane + mine], m_first = m_before(a, seq, seq0, run, h);
+    load_state_parts<NS>(shi, slo, ldv, reinterpret_cast<const uint32_t*>(U), a.d_k, a.d_v, col0, d_pad);
     for (int i = threadIdx.x; i < d_pad; i += kRunThreads) n_s[i] = i < a.d_k ? U[(size_t)a.d_k * a.d_v + i] : 0.f;
-    {   // the memory before the run, (hi, lo) pairs: four numbers per thread and access where the rows allow it
-        const uint32_t* S = reinterpret_cast<const uint32_t*>(U);
-        const bool vec = a.d_v % 4 == 0;
-        for (int i = threadIdx.x; i < d_pad * (NS / 4); i += kRunThreads) {
-            const int r = i / (NS / 4), c = (i % (NS / 4)) * 4;
-            uint32_t w[4] = {0, 0, 0, 0};
-            if (r < a.d_k && col0 + c < a.d_v) {
-                if (vec) {
-                    const uint4 x = *reinterpret_cast<const uint4*>(S + (size_t)r * a.d_v + col0 + c);
-                    w[0] = x.x; w[1] = x.y; w[2] = x.z; w[3] = x.w;
-                } else {
-#pragma unroll
-                    for (int e = 0; e < 4; ++e) w[e] = col0 + c + e < a.d_v ? S[(size_t)r * a.d_v + col0 + c + e] : 0u;
-                }
-            }
-            *reinterpret_cast<uint2*>(shi + (size_t)r * ldv + c) = make_uint2(__byte_perm(w[0], w[1], 0x5410), __byte_perm(w[2], w[3], 0x5410));
-            *reinterpret_cast<uint2*>(slo + (size_t)r * ldv + c) = make_uint2(__byte_perm(w[0], w[1], 0x7632), __byte_perm(w[2], w[3], 0x7632));
-        }
+    if (threadIdx.x < kRun) {
+        w_i[threadIdx.x] = f - m;
+        w_j[threadIdx.x] = log_in - f;
+        before[threadIdx.x] = expf(f + (m_first - m));
+        least[threadIdx.x] = expf(-m);
     }
     copies_done();
     __syncthreads();

@@ -75,6 +75,42 @@ __device__ __forceinline__ void load_tile(__nv_bfloat16* dst, int ld, const __nv
     }
 }
 
+// columns col0 .. col0 + NS of a state [d_k][d_v] kept as (hi, lo) pairs of bfloat16 (one 32-bit word per number) as two tiles [d_pad][ldv]
+// of its hi and lo parts, zeros beyond its edges: four numbers per thread and access where the rows allow it, eight accesses of a thread
+// on their way at once
+template <int NS>
+__device__ __forceinline__ void load_state_parts(__nv_bfloat16* shi, __nv_bfloat16* slo, int ldv, const uint32_t* S, int d_k, int d_v, int col0, int d_pad) {
+    const bool vec = d_v % 4 == 0;
+    const int total = d_pad * (NS / 4);
+    for (int base = threadIdx.x; base < total; base += 8 * kRunThreads) {
+        uint4 x[8];
+#pragma unroll
+        for (int u = 0; u < 8; ++u) {
+            const int i = base + u * kRunThreads, r = i / (NS / 4), c = (i % (NS / 4)) * 4;
+            x[u] = make_uint4(0, 0, 0, 0);
+            if (i < total && r < d_k && col0 + c < d_v) {
+                const uint32_t* p = S + (size_t)r * d_v + col0 + c;
+                if (vec) {
+                    x[u] = *reinterpret_cast<const uint4*>(p);
+                } else {
+                    x[u].x = p[0];
+                    x[u].y = col0 + c + 1 < d_v ? p[1] : 0u;
+                    x[u].z = col0 + c + 2 < d_v ? p[2] : 0u;
+                    x[u].w = col0 + c + 3 < d_v ? p[3] : 0u;
+                }
+            }
+        }
+#pragma unroll
+        for (int u = 0; u < 8; ++u) {
+            const int i = base + u * kRunThreads, r = i / (NS / 4), c = (i % (NS / 4)) * 4;
+            if (i < total) {
+                *reinterpret_cast<uint2*>(shi + (size_t)r * ldv + c) = make_uint2(__byte_perm(x[u].x, x[u].y, 0x5410), __byte_perm(x[u].z, x[u].w, 0x5410));
+                *reinterpret_cast<uint2*>(slo + (size_t)r * ldv + c) = make_uint2(__byte_perm(x[u].x, x[u].y, 0x7632), __byte_perm(x[u].z, x[u].w, 0x7632));
+            }
+        }
+    }
+}
+
 // where a sequence's runs start in the scratch: a bound on the runs of the sequences before it that needs no sum over them
 __device__ __forceinline__ int first_run(const int* cu_seqlens, int seq) { return cu_seqlens[seq] / kRun + seq; }
 
